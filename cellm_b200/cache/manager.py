@@ -3,7 +3,7 @@ need, and (through the native runtime) the pages and the state slot each live
 request holds.
 
 Paged groups: keys and values of all order items with the same
-(kv heads, head size, window, value size), pool [items, pages, kv heads, page size, head
+(kv heads, head size, window or chunk, value size), pool [items, pages, kv heads, page size, head
 size] each for K and V (V with rows of the value size where that differs) (K alone for a group whose rows are keys and values at once); one page id of a group means that page in every item
 of the group. The reference sizes one pool for all layers, convolution layers
 included (tools/infer/src/main.rs:386-392); here only items that keep keys
@@ -81,7 +81,7 @@ class CacheManager:
         windows = [k.window for k in self.paged_keys]
         keeps = [k.keep_first if k.window else 0 for k in self.paged_keys]
         self._h = lib().cellm_cache_create(self.page_size, n_paged, int_array(self.group_pages), int_array(windows),
-                                           int_array(keeps), self.num_slots)
+                                           int_array(keeps), int_array([k.chunk for k in self.paged_keys]), self.num_slots)
         if not self._h:
             raise CacheError(last_error())
 

@@ -7,7 +7,7 @@
 // 16 rows per warp; keys are walked in blocks of 64 through the request's
 // block table, with K and V blocks brought in by cp.async, double-buffered.
 // Scores q.k * scale, causal mask (key <= the token's position), optional
-// window, online softmax in 32-bit with the running maximum taken off
+// window or chunk of positions, online softmax in 32-bit with the running maximum taken off
 // (crates/cellm-cache/src/kvcache.rs:753-787, :1206-1227 is the reference's
 // single-token loop). Probabilities are rounded to bfloat16 for the P.V
 // product; sums and outputs stay 32-bit until the final store.
@@ -27,13 +27,20 @@
 
 namespace {
 
-// What the general form adds to a row: the sequence's first `keep_first` keys stay visible behind the window, and a head's
-// output is multiplied by the sigmoid of one number per (token, head) (`gate` [T, gate_ld] 32-bit; null: none).
+// What the general form adds to a row: the sequence's first `keep_first` keys stay visible behind the window, a head's
+// output is multiplied by the sigmoid of one number per (token, head) (`gate` [T, gate_ld] 32-bit; null: none), and with
+// `chunk` > 0 (instead of a window) a token reads the keys of its own run of that many positions, counted from position 0.
 struct FlashExtras {
     int keep_first = 0;
     const float* gate = nullptr;
     long long gate_ld = 0;
+    int chunk = 0;
 };
+
+// The first key a token at position pos reads (may be negative: every earlier key).
+__device__ __forceinline__ int first_key(int pos, int window, int chunk) {
+    return chunk > 0 ? pos / chunk * chunk : window > 0 ? pos - window + 1 : 0;
+}
 
 __device__ __forceinline__ float gate_factor(const FlashExtras& ex, int token, int head) {
     return ex.gate ? 1.f / (1.f + __expf(-ex.gate[(size_t)token * ex.gate_ld + head])) : 1.f;
@@ -74,7 +81,7 @@ attention_flash_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ part
     const int r0 = (tile - base) * BM;
     const int t_lo = r0 / G, t_hi = min(r0 + BM - 1, rows - 1) / G;
     const int key_end = ctx + t_hi + 1;
-    const int key_begin = window > 0 ? max(0, ctx + t_lo - window + 1) : 0;
+    const int key_begin = max(0, first_key(ctx + t_lo, window, ex.chunk));
     const int kb_begin = key_begin / BN, kb_end = (key_end + BN - 1) / BN;
     // the blocks this tile walks: those that hold kept first keys and lie wholly before the window's first block, then
     // the window's; a CTA's piece is a run of this list
@@ -127,7 +134,7 @@ attention_flash_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ part
     // per-thread rows: g = lane / 4 and g + 8 of this warp's 16
     const int row_a = r0 + warp * 16 + (lane >> 2), row_b = row_a + 8;
     const int pos_a = row_a < rows ? ctx + row_a / G : -1, pos_b = row_b < rows ? ctx + row_b / G : -1;
-    const int lo_a = window > 0 ? pos_a - window + 1 : 0, lo_b = window > 0 ? pos_b - window + 1 : 0;
+    const int lo_a = first_key(pos_a, window, ex.chunk), lo_b = first_key(pos_b, window, ex.chunk);
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
     float o[NT][4];
 #pragma unroll
@@ -169,7 +176,7 @@ attention_flash_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ part
         float mx_a = -INFINITY, mx_b = -INFINITY;
         const int w_row0 = r0 + warp * 16, w_row1 = min(w_row0 + 15, rows - 1);
         const bool open_block = w_row0 + 15 < rows && kb * BN + BN - 1 <= ctx + w_row0 / G &&
-                                (window <= 0 || kb * BN >= ctx + w_row1 / G - window + 1);
+                                kb * BN >= first_key(ctx + w_row1 / G, window, ex.chunk);
         if (open_block) {
 #pragma unroll
             for (int n = 0; n < BN / 8; ++n) {
@@ -391,7 +398,7 @@ int launch_flash(__nv_bfloat16* out, float* part_o, float* part_ml, const __nv_b
 }  // namespace
 
 // Head sizes the tensor-core kernel is built for.
-CELLM_API int cellm_attention_flash_supports(int hd) { return hd == 32 || hd == 64 || hd == 128; }
+CELLM_API int cellm_attention_flash_supports(int hd) { return hd == 32 || hd == 64 || hd == 96 || hd == 128; }
 
 // out, q: [T, nh*hd] bf16. n_tiles: sum over requests of ceil(q_len * (nh/nkv) / rows_per_cta),
 // rows_per_cta = 64 (wide = 1) or 16 (wide = 0). nsplit > 1 needs part_o
@@ -420,6 +427,7 @@ static int attention_flash_impl(void* out, float* part_o, float* part_ml, const 
                                      nkv, scale, window, nsplit, err, stream, sinks, unrot, interleaved, ex)
     if (hd == 32) GO(32);
     else if (hd == 64) GO(64);
+    else if (hd == 96) GO(96);
     else if (hd == 128) GO(128);
     else return CELLM_ERR_SIZE;
 #undef GO
@@ -472,6 +480,21 @@ CELLM_API int cellm_attention_flash_masked(void* out, float* part_o, float* part
     ex.gate_ld = gate_ld;
     return attention_flash_impl(out, part_o, part_ml, q, k_pool, v_pool, cu_seqlens, ctx_lens, block_table, bt_stride, B, T,
                                 n_tiles, num_pages, page_size, nh, nkv, hd, scale, window, wide, nsplit, err, stream, sinks,
+                                nullptr, 0, nullptr, ex);
+}
+
+// Chunked: position i reads the keys j <= i of its own run of `chunk` positions (floor(i / chunk) = floor(j / chunk), runs
+// counted from position 0 of the sequence); chunk 0: every earlier key.
+CELLM_API int cellm_attention_flash_chunked(void* out, float* part_o, float* part_ml, const void* q, const void* k_pool,
+                                            const void* v_pool, const int* cu_seqlens, const int* ctx_lens,
+                                            const int* block_table, int bt_stride, int B, int T, int n_tiles, int num_pages,
+                                            int page_size, int nh, int nkv, int hd, float scale, int chunk, int wide, int nsplit,
+                                            int* err, cudaStream_t stream) {
+    if (chunk < 0) return CELLM_ERR_SIZE;
+    FlashExtras ex;
+    ex.chunk = chunk;
+    return attention_flash_impl(out, part_o, part_ml, q, k_pool, v_pool, cu_seqlens, ctx_lens, block_table, bt_stride, B, T,
+                                n_tiles, num_pages, page_size, nh, nkv, hd, scale, 0, wide, nsplit, err, stream, nullptr,
                                 nullptr, 0, nullptr, ex);
 }
 

@@ -24,7 +24,7 @@ attention_plain_kernel(TA* __restrict__ out, const TA* __restrict__ q, const TA*
                        int bt_stride, int num_pages, int page_size, int nh, int nkv, int hd, int hdv, int v_row, float scale,
                        int window, const float* __restrict__ sinks, const float* __restrict__ unrot, int interleaved,
                        int keep_first, float fixed_sink, int has_fixed_sink, const float* __restrict__ gate, long long gate_ld,
-                       int* __restrict__ err) {
+                       int chunk, int* __restrict__ err) {
     constexpr int CH = ATTN_PLAIN_THREADS;
     extern __shared__ float smem[];
     float* qs = smem;             // [hd]
@@ -37,7 +37,8 @@ attention_plain_kernel(TA* __restrict__ out, const TA* __restrict__ q, const TA*
     const int kvh = h / (nh / nkv);
     const int pos = positions[t];
     const int b = seq_of_token[t];
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    // the first key this token reads: its window's, or the first of its own run of `chunk` positions
+    const int lo = chunk > 0 ? pos / chunk * chunk : (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int i = threadIdx.x; i < hd; i += CH) qs[i] = to_float(q[(size_t)t * nh * hd + (size_t)h * hd + i]) * scale;
     float m = -INFINITY, l = 0.f;
@@ -154,10 +155,10 @@ static int attention_plain_impl(void* out, const void* q, const void* k_pool, co
                                 int hd, int hdv, int v_row, float scale, int window, int dtype, int* err,
                                 cudaStream_t stream, const float* sinks = nullptr, const float* unrot = nullptr,
                                 int interleaved = 0, int keep_first = 0, float fixed_sink = 0.f, int has_fixed_sink = 0,
-                                const float* gate = nullptr, long long gate_ld = 0) {
+                                const float* gate = nullptr, long long gate_ld = 0, int chunk = 0) {
     if (T <= 0) return CELLM_OK;
     if (unrot && hdv % 2) return CELLM_ERR_SIZE;
-    if (keep_first < 0) return CELLM_ERR_SIZE;
+    if (keep_first < 0 || chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return CELLM_ERR_SIZE;
     if (hd > ATTN_PLAIN_MAX_HD || hd <= 0 || hdv <= 0 || hdv > v_row || hdv > ATTN_PLAIN_MAX_HD || nkv <= 0 || nh % nkv) return CELLM_ERR_SIZE;
     // the first hd floats hold the query; the output is turned back in the same place (hdv floats)
     const size_t smem = (size_t)((hd > hdv ? hd : hdv) + 2 * ATTN_PLAIN_THREADS) * sizeof(float);
@@ -165,12 +166,12 @@ static int attention_plain_impl(void* out, const void* q, const void* k_pool, co
     if (dtype == CELLM_F32)
         CELLM_RUN(attention_plain_kernel<float>, grid, ATTN_PLAIN_THREADS, smem, stream,
             (float*)out, (const float*)q, (const float*)k_pool, (const float*)v_pool, positions, seq_of_token,
-            block_table, bt_stride, num_pages, page_size, nh, nkv, hd, hdv, v_row, scale, window, sinks, unrot, interleaved, keep_first, fixed_sink, has_fixed_sink, gate, gate_ld, err);
+            block_table, bt_stride, num_pages, page_size, nh, nkv, hd, hdv, v_row, scale, window, sinks, unrot, interleaved, keep_first, fixed_sink, has_fixed_sink, gate, gate_ld, chunk, err);
     else if (dtype == CELLM_BF16)
         CELLM_RUN(attention_plain_kernel<__nv_bfloat16>, grid, ATTN_PLAIN_THREADS, smem, stream,
             (__nv_bfloat16*)out, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool,
             (const __nv_bfloat16*)v_pool, positions, seq_of_token, block_table, bt_stride, num_pages,
-            page_size, nh, nkv, hd, hdv, v_row, scale, window, sinks, unrot, interleaved, keep_first, fixed_sink, has_fixed_sink, gate, gate_ld, err);
+            page_size, nh, nkv, hd, hdv, v_row, scale, window, sinks, unrot, interleaved, keep_first, fixed_sink, has_fixed_sink, gate, gate_ld, chunk, err);
     else return CELLM_ERR_DTYPE;
     return CELLM_OK;
 }
@@ -223,4 +224,14 @@ CELLM_API int cellm_attention_plain_masked(void* out, const void* q, const void*
     return attention_plain_impl(out, q, k_pool, v_pool, positions, seq_of_token, block_table, bt_stride, num_pages, page_size, T, nh, nkv,
                                 hd, hdv, v_row, scale, window, dtype, err, stream, sinks, nullptr, 0, keep_first, fixed_sink, has_fixed_sink,
                                 gate, gate_ld);
+}
+
+// Chunked: position i reads the keys j <= i of its own run of `chunk` positions (floor(i / chunk) = floor(j / chunk), runs
+// counted from position 0 of the sequence); chunk 0: every earlier key. A pool of values with rows of hdv entries.
+CELLM_API int cellm_attention_plain_chunked(void* out, const void* q, const void* k_pool, const void* v_pool,
+                                            const int* positions, const int* seq_of_token, const int* block_table,
+                                            int bt_stride, int num_pages, int page_size, int T, int nh, int nkv,
+                                            int hd, int hdv, float scale, int chunk, int dtype, int* err, cudaStream_t stream) {
+    return attention_plain_impl(out, q, k_pool, v_pool, positions, seq_of_token, block_table, bt_stride, num_pages, page_size, T, nh, nkv,
+                                hd, hdv, hdv, scale, 0, dtype, err, stream, nullptr, nullptr, 0, 0, 0.f, 0, nullptr, 0, chunk);
 }

@@ -215,6 +215,12 @@ struct TileRange {
     bool has;        // the tile holds at least one token
 };
 
+// The first key a token at position pos reads: its window's, or the first of its own run of `chunk` positions (counted from
+// position 0); it may be negative or 0 (every earlier key).
+__device__ __forceinline__ int first_key(int pos, int window, int chunk) {
+    return chunk > 0 ? pos / chunk * chunk : window > 0 ? pos - window + 1 : 0;
+}
+
 // Launched with 320 threads. A scheduler holds three of the ten warps and 16384 registers: 168 a thread at
 // most, which the bound of 384 threads makes the compiler keep.
 __global__ void __launch_bounds__(384, 1)
@@ -223,7 +229,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     const int* __restrict__ cu_seqlens, const int* __restrict__ ctx_lens,
                     const int* __restrict__ block_table, int bt_stride, int B, int num_pages, int page_size, int nh,
                     int nkv, float scale_log2e, int window, const float* __restrict__ sinks, const float* __restrict__ gate,
-                    long long gate_ld, int* __restrict__ err) {
+                    long long gate_ld, int chunk, int* __restrict__ err) {
     extern __shared__ __align__(1024) uint8_t smem_raw[];
     TcSmem& sm = *reinterpret_cast<TcSmem*>(smem_raw);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -286,7 +292,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             tr[t].has = tr[t].tok0 < q_len;
             if (tr[t].has) {
                 const int tok1 = min(tr[t].tok0 + tok_per_tile, q_len) - 1;
-                const int kb = window > 0 ? max(0, ctx + tr[t].tok0 - window + 1) : 0;
+                const int kb = max(0, first_key(ctx + tr[t].tok0, window, chunk));
                 tr[t].lo = kb / TN;
                 tr[t].hi = (ctx + tok1 + 1 + TN - 1) / TN;
                 if (t == 0) key_begin = kb;
@@ -397,7 +403,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const int tok = tr[t].tok0 + r / G;                           // token within the portion
         const bool row_ok = tok < q_len;
         const int pos = row_ok ? ctx + tok : -1;
-        const int lo = window > 0 ? pos - window + 1 : 0;
+        const int lo = first_key(pos, window, chunk);
         const uint32_t lane_base = tmem + ((uint32_t)(qt * 32) << 16);
         const uint32_t s_col = (uint32_t)(t * TN);
         const uint32_t o_col = (uint32_t)(O_COL + t * HD);
@@ -416,7 +422,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             tc_fence_before();
             mbar_arrive(&sm.s_empty[t]);                              // the scores are in registers now
             const int jbase = (tr[t].lo + it) * TN;
-            const bool open_block = row_ok && jbase + TN - 1 <= pos && (window <= 0 || jbase >= lo);
+            const bool open_block = row_ok && jbase + TN - 1 <= pos && jbase >= lo;
             if (!open_block) {
 #pragma unroll
                 for (int i = 0; i < TN; ++i) {
@@ -555,7 +561,7 @@ static int attention_tc_impl(void* out, const void* q, const void* k_pool, const
                              const int* cu_seqlens, const int* ctx_lens, const int* block_table, int bt_stride,
                              int B, int T, int n_tiles, int num_pages, int page_size, int nh, int nkv, int hd,
                              float scale, int window, const float* sinks, const float* gate, long long gate_ld, int* err,
-                             cudaStream_t stream) {
+                             cudaStream_t stream, int chunk = 0) {
     if (T <= 0 || n_tiles <= 0) return CELLM_OK;
     if (!cellm_attention_tc_supports(hd, nh, nkv, page_size) || scale <= 0.f) return CELLM_ERR_SIZE;
     if (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15) return CELLM_ERR_ALIGN;
@@ -583,7 +589,7 @@ static int attention_tc_impl(void* out, const void* q, const void* k_pool, const
     dim3 grid((unsigned)n_tiles, (unsigned)nkv);
     CELLM_RUN(attention_tc_kernel, grid, THREADS, smem, stream, mq, mk, mv, (__nv_bfloat16*)out, cu_seqlens,
               ctx_lens, block_table, bt_stride, B, num_pages, page_size, nh, nkv, scale * 1.4426950408889634f, window, sinks,
-              gate, gate_ld, err);
+              gate, gate_ld, chunk, err);
     return CELLM_OK;
 }
 
@@ -604,4 +610,15 @@ CELLM_API int cellm_attention_tc_gated(void* out, const void* q, const void* k_p
                                        int* err, cudaStream_t stream) {
     return attention_tc_impl(out, q, k_pool, v_pool, cu_seqlens, ctx_lens, block_table, bt_stride, B, T, n_tiles, num_pages,
                              page_size, nh, nkv, hd, scale, window, sinks, gate, gate_ld, err, stream);
+}
+
+// Chunked: position i reads the keys j <= i of its own run of `chunk` positions (runs counted from position 0 of the
+// sequence); chunk 0: every earlier key.
+CELLM_API int cellm_attention_tc_chunked(void* out, const void* q, const void* k_pool, const void* v_pool,
+                                         const int* cu_seqlens, const int* ctx_lens, const int* block_table, int bt_stride,
+                                         int B, int T, int n_tiles, int num_pages, int page_size, int nh, int nkv, int hd,
+                                         float scale, int chunk, int* err, cudaStream_t stream) {
+    if (chunk < 0) return CELLM_ERR_SIZE;
+    return attention_tc_impl(out, q, k_pool, v_pool, cu_seqlens, ctx_lens, block_table, bt_stride, B, T, n_tiles, num_pages,
+                             page_size, nh, nkv, hd, scale, 0, nullptr, nullptr, 0, err, stream, chunk);
 }

@@ -64,6 +64,19 @@ __device__ __forceinline__ float cellm_activate(float z, int act) {
     }
 }
 
+// The clamped gate: with g' = min(g, limit) and u' = clamp(u, -limit, limit), g' sigmoid(slope g') (u' + 1). The quick form
+// takes the exponential by the fast instruction, for results that are rounded to bfloat16 at once.
+__device__ __forceinline__ float cellm_clamped_gate(float g, float u, float limit, float slope) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + expf(-slope * g)) * (u + 1.f);
+}
+__device__ __forceinline__ float cellm_clamped_gate_rounded(float g, float u, float limit, float slope) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return __fdividef(g, 1.f + __expf(-slope * g)) * (u + 1.f);
+}
+
 // xIELU with its two factors already formed (ap = softplus(p), aq = 1/2 + softplus(q)): z > 0: ap z^2 + z / 2; otherwise
 // aq (exp(z) - 1 - z) + z / 2.
 __device__ __forceinline__ float cellm_softplus(float v) { return v > 20.f ? v : log1pf(expf(v)); }

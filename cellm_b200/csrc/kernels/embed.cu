@@ -140,3 +140,49 @@ CELLM_API int cellm_embed_pairs(float* out, const void* table, int table_dtype, 
         return CELLM_ERR_DTYPE;
     return CELLM_OK;
 }
+
+// With a norm: out[t, :] = r / sqrt(mean(r^2) + eps) * w, r = float(table[ids[t], :]) * scale; the row waits in shared memory.
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_norm_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ ids, const float* __restrict__ w, int H, int V,
+                  float scale, float eps, int* __restrict__ err) {
+    extern __shared__ float row_s[];
+    __shared__ float scratch[32];
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x, id = ids[t];
+    const bool ok = id >= 0 && id < V;
+    if (!ok && threadIdx.x == 0) atomicOr(err, CELLM_DEV_BAD_TOKEN);
+    const T* row = table + (size_t)(ok ? id : 0) * H;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float v = ok ? to_float(row[i]) * scale : 0.f;
+        row_s[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.f / sqrtf(ss / (float)H + eps);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)t * H + i] = row_s[i] * inv * w[i];
+}
+
+// w [H] 32-bit.
+CELLM_API int cellm_embed_norm(float* out, const void* table, int table_dtype, const int* ids, const float* w, int T, int H, int V, float scale,
+                               float eps, int* err, cudaStream_t stream) {
+    if (T <= 0) return CELLM_OK;
+    if (!w) return CELLM_ERR_ARG;
+    const size_t smem = (size_t)H * sizeof(float);
+    if (H <= 0 || smem > 200 * 1024) return CELLM_ERR_SIZE;
+#define EN_RUN(T_)                                                                                                              \
+    do {                                                                                                                        \
+        if (smem > 48 * 1024) {                                                                                                 \
+            cudaError_t e = cudaFuncSetAttribute(embed_norm_kernel<T_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return (int)e;                                                                                \
+        }                                                                                                                       \
+        CELLM_RUN_SERIAL(embed_norm_kernel<T_>, T, 256, smem, stream, out, (const T_*)table, ids, w, H, V, scale, eps, err);     \
+    } while (0)
+    if (table_dtype == CELLM_F32) EN_RUN(float);
+    else if (table_dtype == CELLM_BF16) EN_RUN(__nv_bfloat16);
+    else return CELLM_ERR_DTYPE;
+#undef EN_RUN
+    return CELLM_OK;
+}

@@ -26,7 +26,7 @@
 // and the slice that finishes last sums them in a fixed order (see the kernel).
 //
 // Epilogues (template parameter EPI of gemm_tcgen05_kernel; each is described where it is defined):
-//   0  C = A.W^T                      1  SwiGLU over interleaved gate and up blocks
+//   0  C = A.W^T                      1  SwiGLU (or the clamped gate) over interleaved gate and up blocks
 //   2  in_proj + gated short convolution of a decode step (cellm_gemm_conv_tcgen05)
 //   3  q/k/v product + head norms + rotation + cache write of a decode step (cellm_gemm_rope_tcgen05)
 // 2 and 3 exist for swapped tiles whose K split is summed inside a cluster.
@@ -133,7 +133,7 @@ template <int BN, int STAGES, bool SWAP, int EPI, bool CLUSTER, typename TO>
 __global__ void __launch_bounds__(192, SWAP ? 2 : 1)      // swapped tiles: two CTAs an SM, so the next product's can move in early
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_constant__ CUtensorMap map_cols,
                     TO* __restrict__ C, float* __restrict__ ws, int* __restrict__ counters, int M, int N, int K,
-                    long long ldc, int kblocks_per_split, int w_is_static, int* __restrict__ err, const ConvEpi conv, const RopeEpi rope) {
+                    long long ldc, int kblocks_per_split, int w_is_static, int* __restrict__ err, const ConvEpi conv, const RopeEpi rope, const GateEpi gate_epi) {
     static_assert(!CLUSTER || SWAP, "the cluster reduction serves swapped tiles");
     static_assert(EPI < 2 || CLUSTER, "the convolution and rotation epilogues are written for the cluster's reduction");
     extern __shared__ uint8_t smem_raw[];
@@ -338,7 +338,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                         tmem_ld32(lane_addr + (uint32_t)(j * 128 + h * 32), g);
                         tmem_ld32(lane_addr + (uint32_t)(j * 128 + 64 + h * 32), u);
 #pragma unroll
-                        for (int i = 0; i < 32; ++i) g[i] = __float_as_uint(silu_mul(__uint_as_float(g[i]), __uint_as_float(u[i])));
+                        for (int i = 0; i < 32; ++i) g[i] = __float_as_uint(gate_up(__uint_as_float(g[i]), __uint_as_float(u[i]), gate_epi));
                         const int o = o0 + j * 64 + h * 32;
                         if (p < P && o < Q / 2) store_row<TO>(C + (size_t)p * ldc + o, g, Q / 2 - o, aligned);
                     }
@@ -415,7 +415,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
 #pragma unroll
                             for (int j = 0; j < 8; ++j) {
                                 if (q + j < q_end) {
-                                    if (gate) C[(size_t)(q + j) * ldc + (p0 / 2 + pl)] = from_float<TO>(silu_mul(g[j], u[j]));
+                                    if (gate) C[(size_t)(q + j) * ldc + (p0 / 2 + pl)] = from_float<TO>(gate_up(g[j], u[j], gate_epi));
                                     else C[(size_t)(q + j) * ldc + p] = from_float<TO>(g[j]);
                                 }
                             }
@@ -454,7 +454,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                                 }
 #pragma unroll
                                 for (int j = 0; j < 8; ++j)
-                                    if (q + 64 + i + j < q_end) C[(size_t)p * ldc + (q / 2 + i + j)] = from_float<TO>(silu_mul(g[j], u[j]));
+                                    if (q + 64 + i + j < q_end) C[(size_t)p * ldc + (q / 2 + i + j)] = from_float<TO>(gate_up(g[j], u[j], gate_epi));
                             }
                     }
                 }
@@ -583,7 +583,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
 #pragma unroll
                     for (int r = 0; r < 8; ++r)
                         if (r < splits) { g += mine[r * plane]; u += mine[r * plane + 64]; }
-                    if (p0 + row + 64 < P) C[(size_t)q * ldc + (p0 / 2 + row)] = from_float<TO>(silu_mul(g, u));
+                    if (p0 + row + 64 < P) C[(size_t)q * ldc + (p0 / 2 + row)] = from_float<TO>(gate_up(g, u, gate_epi));
                 }
             }
         }
@@ -596,7 +596,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
 // Sum of the K-split pieces of a product with plain tiles, ws[split][M][N], in the order of the splits; one
 // thread for four neighbouring outputs. EPI as in the product's kernel (1: gate and up blocks of 64 columns).
 template <int EPI, typename TO>
-__global__ void splitk_sum_kernel(const float* __restrict__ ws, TO* __restrict__ C, int M, int N, long long ldc, int splits) {
+__global__ void splitk_sum_kernel(const float* __restrict__ ws, TO* __restrict__ C, int M, int N, long long ldc, int splits,
+                                  const GateEpi gate_epi) {
     pdl_trigger();
     pdl_wait();
     const int NO = EPI == 1 ? N / 2 : N;                       // output columns
@@ -626,7 +627,7 @@ __global__ void splitk_sum_kernel(const float* __restrict__ ws, TO* __restrict__
         }
     }
     for (int j = 0; j < 4 && o0 + j < NO; ++j)
-        C[(size_t)m * ldc + o0 + j] = from_float<TO>(EPI == 1 ? silu_mul(a[j], b[j]) : a[j]);
+        C[(size_t)m * ldc + o0 + j] = from_float<TO>(EPI == 1 ? gate_up(a[j], b[j], gate_epi) : a[j]);
 }
 
 // Sixteen values of a row (the last chunk of a tile whose width is an odd multiple of 16).
@@ -678,7 +679,7 @@ __global__ void __launch_bounds__(192)
 gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                                TO* __restrict__ C, int M, int N, int K, long long ldc, int w_is_static,
                                int* __restrict__ err, int bn, const int* __restrict__ tile_group, int act,
-                               const float* __restrict__ act_numbers) {
+                               const float* __restrict__ act_numbers, const GateEpi gate_epi) {
     // bn: the width of a tile in columns, a multiple of 16 (of 128 with the SwiGLU epilogue) and at most BN, which
     // sizes the stages and the accumulators. Widths between the powers of two let the number of tiles come close
     // to a multiple of the SMs, so that the last wave is not half empty.
@@ -833,7 +834,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
                         tmem_ld32(lane_addr + (uint32_t)(j * 128 + 64 + h * 32), u);
                         if (j == bn / 128 - 1 && h == 1) { tc_fence_before(); mbar_arrive(&sm.acc_empty2[buf]); }
 #pragma unroll
-                        for (int i = 0; i < 32; ++i) g[i] = __float_as_uint(silu_mul(__uint_as_float(g[i]), __uint_as_float(u[i])));
+                        for (int i = 0; i < 32; ++i) g[i] = __float_as_uint(gate_up(__uint_as_float(g[i]), __uint_as_float(u[i]), gate_epi));
                         const int o = o0 + j * 64 + h * 32;
                         if (p < M && o < N / 2) store_row<TO>(C + (size_t)p * ldc + o, g, N / 2 - o, aligned);
                     }
@@ -851,7 +852,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
 template <int BN, int STAGES, bool SWAP, int EPI, bool CLUSTER, typename TO>
 int launch(const CUtensorMap& m_rows, const CUtensorMap& m_cols, TO* C, float* ws, int* counters, int M, int N, int K,
            long long ldc, int split_k, int kblocks_per_split, int w_is_static, int* err, cudaStream_t stream,
-           const ConvEpi& conv, const RopeEpi& rope) {
+           const ConvEpi& conv, const RopeEpi& rope, const GateEpi& gate_epi) {
     const size_t smem = sizeof(GemmSmem<BN, STAGES, CLUSTER ? (BN + 8) * BM : 0>) + 1024;
     static bool configured = false;
     auto kernel = gemm_tcgen05_kernel<BN, STAGES, SWAP, EPI, CLUSTER, TO>;
@@ -880,14 +881,14 @@ int launch(const CUtensorMap& m_rows, const CUtensorMap& m_cols, TO* C, float* w
         cfg.numAttrs = 2;
     }
     cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, m_rows, m_cols, C, ws, counters, M, N, K, ldc, kblocks_per_split,
-                                       w_is_static, err, conv, rope);
+                                       w_is_static, err, conv, rope, gate_epi);
     return e == cudaSuccess ? CELLM_OK : (int)e;
 }
 
 template <int BN, int STAGES, int EPI, typename TO>
 int launch_persistent(const CUtensorMap& m_a, const CUtensorMap& m_w, TO* C, int M, int N, int K, long long ldc,
                       int w_is_static, int* err, cudaStream_t stream, int bn, const int* tile_group = nullptr, int act = -1,
-                      const float* act_numbers = nullptr) {
+                      const float* act_numbers = nullptr, const GateEpi& gate_epi = GateEpi()) {
     const size_t smem = sizeof(GemmSmem<BN, STAGES>) + 1024;
     static int sms = 0;
     if (sms == 0) {
@@ -901,7 +902,7 @@ int launch_persistent(const CUtensorMap& m_a, const CUtensorMap& m_w, TO* C, int
     const int tiles = ((N + bn - 1) / bn) * ((M + BM - 1) / BM);
     dim3 grid((unsigned)(tiles < sms ? tiles : sms));
     cudaError_t e = cellm_launch(gemm_tcgen05_persistent_kernel<BN, STAGES, EPI, TO>, grid, dim3(192), smem, stream, m_a,
-                                 m_w, C, M, N, K, ldc, w_is_static, err, bn, tile_group, act, act_numbers);
+                                 m_w, C, M, N, K, ldc, w_is_static, err, bn, tile_group, act, act_numbers, gate_epi);
     return e == cudaSuccess ? CELLM_OK : (int)e;
 }
 
@@ -938,7 +939,7 @@ CELLM_API int cellm_gemm_tcgen05_plan(int M, int N, int K, int bn, int split_k, 
 static int gemm_impl(void* C, const void* A, const void* W, int M, int N, int K, long long lda,
                      long long ldw, long long ldc, int out_dtype, int bn, int split_k, int epilogue,
                      int w_is_static, float* workspace, int* counters, int* err, cudaStream_t stream,
-                     const ConvEpi& conv, const RopeEpi& rope) {
+                     const ConvEpi& conv, const RopeEpi& rope, const GateEpi& gate_epi = GateEpi()) {
     if (M <= 0 || N <= 0) return CELLM_OK;
     if (K <= 0 || (K & 7)) return CELLM_ERR_SIZE;
     if (((uintptr_t)A & 15) || ((uintptr_t)W & 15) || ((lda * 2) & 15) || ((ldw * 2) & 15)) return CELLM_ERR_ALIGN;
@@ -982,8 +983,8 @@ static int gemm_impl(void* C, const void* A, const void* W, int M, int N, int K,
     if (!swap && split == 1 && narrow >= 128) {
 #define GOP(BN_, ST_, EP_)                                                                                          \
     do {                                                                                                            \
-        if (out_dtype == CELLM_F32) rc = launch_persistent<BN_, ST_, EP_, float>(map_a, map_w, (float*)C, M, N, K, ldc, w_is_static, err, stream, narrow); \
-        else rc = launch_persistent<BN_, ST_, EP_, __nv_bfloat16>(map_a, map_w, (__nv_bfloat16*)C, M, N, K, ldc, w_is_static, err, stream, narrow); \
+        if (out_dtype == CELLM_F32) rc = launch_persistent<BN_, ST_, EP_, float>(map_a, map_w, (float*)C, M, N, K, ldc, w_is_static, err, stream, narrow, nullptr, -1, nullptr, gate_epi); \
+        else rc = launch_persistent<BN_, ST_, EP_, __nv_bfloat16>(map_a, map_w, (__nv_bfloat16*)C, M, N, K, ldc, w_is_static, err, stream, narrow, nullptr, -1, nullptr, gate_epi); \
     } while (0)
         if (narrow == 128) { if (epilogue == 0) GOP(128, 6, 0); else GOP(128, 6, 1); }
         else { if (epilogue == 0) GOP(256, 4, 0); else GOP(256, 4, 1); }       // 144 to 256 columns
@@ -992,8 +993,8 @@ static int gemm_impl(void* C, const void* A, const void* W, int M, int N, int K,
     }
 #define GO3(BN_, ST_, SW_, EP_, CL_)                                                                                  \
     do {                                                                                                              \
-        if (out_dtype == CELLM_F32) rc = launch<BN_, ST_, SW_, EP_, CL_, float>(m_rows, m_cols, (float*)C, workspace, counters, M, N, K, ldc, split, per, w_is_static, err, stream, conv, rope); \
-        else rc = launch<BN_, ST_, SW_, EP_, CL_, __nv_bfloat16>(m_rows, m_cols, (__nv_bfloat16*)C, workspace, counters, M, N, K, ldc, split, per, w_is_static, err, stream, conv, rope); \
+        if (out_dtype == CELLM_F32) rc = launch<BN_, ST_, SW_, EP_, CL_, float>(m_rows, m_cols, (float*)C, workspace, counters, M, N, K, ldc, split, per, w_is_static, err, stream, conv, rope, gate_epi); \
+        else rc = launch<BN_, ST_, SW_, EP_, CL_, __nv_bfloat16>(m_rows, m_cols, (__nv_bfloat16*)C, workspace, counters, M, N, K, ldc, split, per, w_is_static, err, stream, conv, rope, gate_epi); \
     } while (0)
 #define GO2(BN_, ST_, SW_, EP_) GO3(BN_, ST_, SW_, EP_, false)
     // swapped: ST_ stages without, CST_ stages with the cluster's reduction buffer (two CTAs must still fit an SM); the
@@ -1025,10 +1026,10 @@ static int gemm_impl(void* C, const void* A, const void* W, int M, int N, int K,
         const int NO = epilogue == 1 ? N / 2 : N;
         const long long groups = (long long)M * ((NO + 3) / 4);
         const unsigned blocks = (unsigned)((groups + 255) / 256);
-        if (epilogue == 0 && out_dtype == CELLM_F32) CELLM_RUN((splitk_sum_kernel<0, float>), blocks, 256, 0, stream, workspace, (float*)C, M, N, ldc, split);
-        else if (epilogue == 0) CELLM_RUN((splitk_sum_kernel<0, __nv_bfloat16>), blocks, 256, 0, stream, workspace, (__nv_bfloat16*)C, M, N, ldc, split);
-        else if (out_dtype == CELLM_F32) CELLM_RUN((splitk_sum_kernel<1, float>), blocks, 256, 0, stream, workspace, (float*)C, M, N, ldc, split);
-        else CELLM_RUN((splitk_sum_kernel<1, __nv_bfloat16>), blocks, 256, 0, stream, workspace, (__nv_bfloat16*)C, M, N, ldc, split);
+        if (epilogue == 0 && out_dtype == CELLM_F32) CELLM_RUN((splitk_sum_kernel<0, float>), blocks, 256, 0, stream, workspace, (float*)C, M, N, ldc, split, gate_epi);
+        else if (epilogue == 0) CELLM_RUN((splitk_sum_kernel<0, __nv_bfloat16>), blocks, 256, 0, stream, workspace, (__nv_bfloat16*)C, M, N, ldc, split, gate_epi);
+        else if (out_dtype == CELLM_F32) CELLM_RUN((splitk_sum_kernel<1, float>), blocks, 256, 0, stream, workspace, (float*)C, M, N, ldc, split, gate_epi);
+        else CELLM_RUN((splitk_sum_kernel<1, __nv_bfloat16>), blocks, 256, 0, stream, workspace, (__nv_bfloat16*)C, M, N, ldc, split, gate_epi);
     }
     return rc;
 }
@@ -1054,6 +1055,31 @@ CELLM_API int cellm_gemm_grouped_tcgen05(void* C, const void* A, const void* W, 
     }
     if (out_dtype == CELLM_F32) return launch_persistent<256, 4, 0, float>(map_a, map_w, (float*)C, M, N, K, ldc, 0, err, stream, bn, tile_group, act);
     return launch_persistent<256, 4, 0, __nv_bfloat16>(map_a, map_w, (__nv_bfloat16*)C, M, N, K, ldc, 0, err, stream, bn, tile_group, act);
+}
+
+// The grouped product over gate and up (epilogue 1): W holds `groups` matrices of N rows (N a multiple of 128) in blocks of
+// 64 gate rows followed by their 64 up rows, and C [M, N / 2] gets the two joined as `gate_kind` says (0 silu(g) * u; 1 the
+// clamped gate with `limit` and `slope`). tile_group null (groups = 1): an ordinary product of any M.
+CELLM_API int cellm_gemm_grouped_gated_tcgen05(void* C, const void* A, const void* W, int M, int N, int K, int groups, long long lda,
+                                               long long ldw, long long ldc, int out_dtype, const int* tile_group, int gate_kind, float limit,
+                                               float slope, int* err, cudaStream_t stream) {
+    if (M <= 0 || N <= 0) return CELLM_OK;
+    if (K <= 0 || (K & 7) || (N & 127) || groups < 1 || (tile_group && (M % BM)) || (!tile_group && groups != 1)) return CELLM_ERR_SIZE;
+    if (((uintptr_t)A & 15) || ((uintptr_t)W & 15) || ((lda * 2) & 15) || ((ldw * 2) & 15)) return CELLM_ERR_ALIGN;
+    if (out_dtype != CELLM_F32 && out_dtype != CELLM_BF16) return CELLM_ERR_DTYPE;
+    if (gate_kind < 0 || gate_kind > 1) return CELLM_ERR_ARG;
+    GateEpi gate_epi;
+    gate_epi.kind = gate_kind, gate_epi.limit = limit, gate_epi.slope = slope;
+    const int bn = (N & 255) == 0 ? 256 : 128;      // a tile of 256 columns must not reach into the next matrix's rows
+    CUtensorMap map_a, map_w;
+    if (!tensor_map(&map_a, A, (uint64_t)M, (uint64_t)K, (uint64_t)lda * 2, (uint32_t)BM)) return CELLM_ERR_ARG;
+    if (!tensor_map(&map_w, W, (uint64_t)groups * (uint64_t)N, (uint64_t)K, (uint64_t)ldw * 2, (uint32_t)bn)) return CELLM_ERR_ARG;
+    if (bn == 128) {
+        if (out_dtype == CELLM_F32) return launch_persistent<128, 6, 1, float>(map_a, map_w, (float*)C, M, N, K, ldc, 0, err, stream, bn, tile_group, -1, nullptr, gate_epi);
+        return launch_persistent<128, 6, 1, __nv_bfloat16>(map_a, map_w, (__nv_bfloat16*)C, M, N, K, ldc, 0, err, stream, bn, tile_group, -1, nullptr, gate_epi);
+    }
+    if (out_dtype == CELLM_F32) return launch_persistent<256, 4, 1, float>(map_a, map_w, (float*)C, M, N, K, ldc, 0, err, stream, bn, tile_group, -1, nullptr, gate_epi);
+    return launch_persistent<256, 4, 1, __nv_bfloat16>(map_a, map_w, (__nv_bfloat16*)C, M, N, K, ldc, 0, err, stream, bn, tile_group, -1, nullptr, gate_epi);
 }
 
 // An ordinary product of any M with xIELU in its epilogue: C [M, N] = xielu(A [M, K] . W [N, K]^T) with the two learned
@@ -1086,6 +1112,20 @@ CELLM_API int cellm_gemm_tcgen05(void* C, const void* A, const void* W, int M, i
     const RopeEpi none3{};
     return gemm_impl(C, A, W, M, N, K, lda, ldw, ldc, out_dtype, bn, split_k, epilogue, w_is_static, workspace, counters,
                      err, stream, none, none3);
+}
+
+// The product over blocks of gate and up rows (epilogue 1 of the product described above gemm_impl), the two joined as
+// `gate_kind` says: 0 silu(g) * u, 1 the clamped gate with `limit` and `slope`.
+CELLM_API int cellm_gemm_gated_tcgen05(void* C, const void* A, const void* W, int M, int N, int K, long long lda,
+                                       long long ldw, long long ldc, int out_dtype, int bn, int split_k, int gate_kind, float limit,
+                                       float slope, int w_is_static, float* workspace, int* counters, int* err, cudaStream_t stream) {
+    if (gate_kind < 0 || gate_kind > 1) return CELLM_ERR_ARG;
+    const ConvEpi none{};
+    const RopeEpi none3{};
+    GateEpi gate_epi;
+    gate_epi.kind = gate_kind, gate_epi.limit = limit, gate_epi.slope = slope;
+    return gemm_impl(C, A, W, M, N, K, lda, ldw, ldc, out_dtype, bn, split_k, 1, w_is_static, workspace, counters,
+                     err, stream, none, none3, gate_epi);
 }
 
 // in_proj and the gated short convolution of a decode step in one kernel (the kernel's EPI = 2).

@@ -48,7 +48,8 @@ template <int HD>
 __device__ __forceinline__ int tile_offset(int row, int chunk) {
     constexpr int CH = HD / 8;
     int sw;
-    if constexpr (CH >= 8) sw = chunk ^ (row & 7);
+    if constexpr (CH == 12) sw = chunk ^ ((row >> 1) & 3);      // rows of 192 bytes: neighbours lie 64 bytes apart modulo 128
+    else if constexpr (CH >= 8) sw = chunk ^ (row & 7);
     else if constexpr (CH == 4) sw = chunk ^ ((row >> 1) & 3);
     else sw = chunk ^ ((row >> 2) & 1);
     return (row * CH + sw) * 16;

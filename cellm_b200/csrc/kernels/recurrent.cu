@@ -3,8 +3,10 @@
 //   HGRN2            S <- diag(f) S + (1 - f) v^T                      o = S^T q
 //   gated delta rule S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //   generalized delta rule   S <- diag(d) S - (a * u)(u^T S) + k v^T (the old S on the right)   o = S^T r
+//   scalar decay     S <- d S + (w v) k^T, one decay d and one writing factor w per head (retention: constants of the
+//                    head; Mamba-2's state-space duality: formed from the token's step size)       o = S^T q
 //
-// In both, column j of S needs only v_j (and the token's vectors over the rows), so the columns are independent: a
+// In all, column j of S needs only v_j (and the token's vectors over the rows), so the columns are independent: a
 // block walks some neighbouring columns of one (request, head) through the request's tokens of the step in order,
 // from the state the step before left. The walk and the order of every sum depend on the head's sizes alone, not on
 // how the sequence was cut, so the state after a token is bit-identical. Everything that enters the recurrence is
@@ -12,7 +14,8 @@
 // (`*_scan_kernel`); the others live in registers (`state_walk_kernel`).
 //
 // Also here: the update of a short convolution's state (conv_taps.cuh), the preparation of the delta rule's
-// inputs (convolution + silu, unit vectors, beta, decays), and the norm over a head's output with an optional gate.
+// inputs (convolution + silu, unit vectors, beta, decays), of Mamba-2's (convolution + silu, step sizes and decays), the
+// rotation of projected heads in place, and the norms over a head's or a group's output with an optional gate.
 #include <algorithm>
 
 #include "conv_taps.cuh"
@@ -58,16 +61,20 @@ __device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.com
 template <int N> __device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // Where the vectors over a head's rows lie: array a of token t and head h starts at p[a] + t * ld[a] + (h / heads_per[a]) * dim.
-// Delta rule: q, k, decay. HGRN2: q, f. Generalized delta rule: r, k, decay, unit key, removal rate times unit key.
+// Delta rule: q, k, decay. HGRN2: q, f. Generalized delta rule: r, k, decay, unit key, removal rate times unit key. Scalar
+// decay: q, k; and two numbers a token and head, the decay at num[0] + t * num_ld[0] + h and the writing factor at num[1]
+// likewise (pitch 0: constants of the head; num[1] null: 1).
 struct WalkVectors {
     const float* p[5];
     long long ld[5];
     int heads_per[5];
+    const float* num[2];
+    long long num_ld[2];
     int vec16;          // every start is a multiple of 16 bytes: copies of four values
 };
 
 // MODE 0: HGRN2; 1: the gated delta rule; 2: the generalized delta rule (five vectors a token: chunks of four tokens for
-// heads of 128 rows, so that three stages stay within the static shared memory).
+// heads of 128 rows, so that three stages stay within the static shared memory); 3: scalar decay.
 template <int DIM, int ROWS, int MODE>
 __global__ void __launch_bounds__(WALK_THREADS)
 state_walk_kernel(float* __restrict__ o_out, float* __restrict__ state, long long slot_stride, int n_slots, const WalkVectors vec,
@@ -119,6 +126,10 @@ state_walk_kernel(float* __restrict__ o_out, float* __restrict__ state, long lon
             if (col0 + c_ < vd) copy_async4(dst + tt * TOK + NV * DIM + c_, v_in + (size_t)(t0 + tt) * ld_v + h * vd + col0 + c_);
         }
         if (DELTA && tid < nt) copy_async4(dst + tid * TOK + NV * DIM + CPB, beta + (size_t)(t0 + tid) * heads + h);
+        if constexpr (MODE == 3) {
+            if (tid < 2 * nt && vec.num[tid & 1])
+                copy_async4(dst + (tid >> 1) * TOK + NV * DIM + CPB + (tid & 1), vec.num[tid & 1] + (size_t)(t0 + (tid >> 1)) * vec.num_ld[tid & 1] + h);
+        }
     };
 #pragma unroll
     for (int c = 0; c < WALK_STAGES - 1; ++c) {
@@ -181,6 +192,17 @@ state_walk_kernel(float* __restrict__ o_out, float* __restrict__ state, long lon
                 const float4 q = q4[g * RG + r];
                 S[4 * g + 0] = fmaf(kk[g].x, u, S[4 * g + 0]), S[4 * g + 1] = fmaf(kk[g].y, u, S[4 * g + 1]);
                 S[4 * g + 2] = fmaf(kk[g].z, u, S[4 * g + 2]), S[4 * g + 3] = fmaf(kk[g].w, u, S[4 * g + 3]);
+                o0 = fmaf(S[4 * g + 0], q.x, o0), o1 = fmaf(S[4 * g + 1], q.y, o1);
+                o0 = fmaf(S[4 * g + 2], q.z, o0), o1 = fmaf(S[4 * g + 3], q.w, o1);
+            }
+        } else if constexpr (MODE == 3) {
+            const float4* k4 = reinterpret_cast<const float4*>(tok + DIM);
+            const float d = tok[NV * DIM + CPB], wv = vec.num[1] ? tok[NV * DIM + CPB + 1] * v : v;
+#pragma unroll
+            for (int g = 0; g < NG; ++g) {
+                const float4 q = q4[g * RG + r], k = k4[g * RG + r];
+                S[4 * g + 0] = fmaf(d, S[4 * g + 0], k.x * wv), S[4 * g + 1] = fmaf(d, S[4 * g + 1], k.y * wv);
+                S[4 * g + 2] = fmaf(d, S[4 * g + 2], k.z * wv), S[4 * g + 3] = fmaf(d, S[4 * g + 3], k.w * wv);
                 o0 = fmaf(S[4 * g + 0], q.x, o0), o1 = fmaf(S[4 * g + 1], q.y, o1);
                 o0 = fmaf(S[4 * g + 2], q.z, o0), o1 = fmaf(S[4 * g + 3], q.w, o1);
             }
@@ -677,13 +699,273 @@ CELLM_API int cellm_gdelta_scan(float* o_out, float* state, long long slot_strid
     return CELLM_OK;
 }
 
+// ------------------------------------------------------------------------------------------------ scalar decay
+// The walk for heads of more than 128 rows: a warp a (request, head, 32 columns of S), the columns in shared memory, one
+// lane a column.
+__global__ void __launch_bounds__(32)
+decay_scan_kernel(float* __restrict__ o_out, float* __restrict__ state, long long slot_stride, int n_slots, const WalkVectors vec,
+                  const float* __restrict__ v_in, long long ld_v, const int* __restrict__ cu_seqlens,
+                  const int* __restrict__ slot_ids, int heads, int dim, int vd, int* __restrict__ err) {
+    extern __shared__ float sm[];
+    float* qs = sm;                 // [dim]
+    float* ks = sm + dim;           // [dim]
+    float* Ssh = sm + 2 * dim;      // [dim][32]: the warp's columns of S
+    const int b = blockIdx.x, h = blockIdx.y, lane = threadIdx.x, j = blockIdx.z * 32 + lane;
+    auto S = [&](int i) -> float& { return Ssh[i * 32 + lane]; };
+    pdl_trigger();
+    pdl_wait();
+    const int slot = slot_ids[b];
+    if (slot < 0 || slot >= n_slots) { if (lane == 0) atomicOr(err, CELLM_DEV_BAD_SLOT); return; }
+    const int start = cu_seqlens[b], end = cu_seqlens[b + 1];
+    float* st = state + (size_t)slot * slot_stride + (size_t)h * dim * vd;
+    const bool live = j < vd;
+    for (int i = 0; i < dim; ++i) S(i) = live ? st[(size_t)i * vd + j] : 0.f;
+    for (int t = start; t < end; ++t) {
+        const float* q = vec.p[0] + (size_t)t * vec.ld[0] + (h / vec.heads_per[0]) * dim;
+        const float* k = vec.p[1] + (size_t)t * vec.ld[1] + (h / vec.heads_per[1]) * dim;
+        for (int i = lane; i < dim; i += 32) { qs[i] = q[i]; ks[i] = k[i]; }
+        const float d = vec.num[0][(size_t)t * vec.num_ld[0] + h], w = vec.num[1] ? vec.num[1][(size_t)t * vec.num_ld[1] + h] : 1.f;
+        const float v = (live ? v_in[(size_t)t * ld_v + h * vd + j] : 0.f) * w;
+        __syncwarp();
+        float o = 0.f;
+        for (int i = 0; i < dim; ++i) {
+            const float s = fmaf(d, S(i), ks[i] * v);
+            S(i) = s;
+            o = fmaf(s, qs[i], o);
+        }
+        if (live) o_out[(size_t)t * heads * vd + (size_t)h * vd + j] = o;
+        __syncwarp();
+    }
+    if (live)
+        for (int i = 0; i < dim; ++i) st[(size_t)i * vd + j] = S(i);
+}
+
+// q, k: rows of `dim` values per head group, [T, ld_q] and [T, ld_k] 32-bit; head h reads group h / (heads / groups).
+// v [T, ld_v]: heads x vd. decay [T (or one row), heads] at pitch ld_d (0: one row of constants), write likewise (null:
+// 1). state [slots][heads][dim][vd] is moved on; o_out [T, heads * vd] gets S^T q.
+CELLM_API int cellm_decay_scan(float* o_out, float* state, long long slot_stride, int n_slots, const float* q, long long ld_q,
+                               const float* k, long long ld_k, const float* v, long long ld_v, const float* decay, long long ld_d,
+                               const float* write, long long ld_w, const int* cu_seqlens, const int* slot_ids, int B, int heads,
+                               int groups, int dim, int vd, int* err, cudaStream_t stream) {
+    if (B <= 0) return CELLM_OK;
+    if (heads <= 0 || groups <= 0 || heads % groups || dim <= 0 || vd <= 0 || dim > RECURRENT_MAX_DIM) return CELLM_ERR_SIZE;
+    if (!decay) return CELLM_ERR_ARG;
+    WalkVectors vec;
+    for (int a = 0; a < 5; ++a) vec.p[a] = nullptr, vec.ld[a] = 0, vec.heads_per[a] = heads / groups;
+    vec.p[0] = q, vec.p[1] = k, vec.ld[0] = ld_q, vec.ld[1] = ld_k;
+    vec.num[0] = decay, vec.num[1] = write, vec.num_ld[0] = ld_d, vec.num_ld[1] = ld_w;
+    vec.vec16 = dim % 4 == 0 && ld_q % 4 == 0 && ld_k % 4 == 0 && aligned16(q) && aligned16(k);
+#define DECAY_WALK(D, R)                                                                                           \
+    CELLM_RUN((state_walk_kernel<D, R, 3>), dim3(B, heads, (vd + WalkShape<D, R>::CPB - 1) / WalkShape<D, R>::CPB), WALK_THREADS, 0, stream, \
+              o_out, state, slot_stride, n_slots, vec, v, ld_v, (const float*)nullptr, cu_seqlens, slot_ids, heads, dim, vd, err)
+    if (dim <= 16) DECAY_WALK(16, 4);
+    else if (dim <= 32) DECAY_WALK(32, 4);
+    else if (dim <= 64) DECAY_WALK(64, 8);
+    else if (dim <= 128) DECAY_WALK(128, 8);
+    else {
+        const size_t big = (size_t)(2 + 32) * dim * sizeof(float);
+        if (big > 48 * 1024) {
+            cudaError_t e = cudaFuncSetAttribute(decay_scan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)big);
+            if (e != cudaSuccess) return (int)e;
+        }
+        CELLM_RUN(decay_scan_kernel, dim3(B, heads, (vd + 31) / 32), 32, big, stream, o_out, state, slot_stride, n_slots, vec, v, ld_v,
+                  cu_seqlens, slot_ids, heads, dim, vd, err);
+    }
+#undef DECAY_WALK
+    return CELLM_OK;
+}
+
+// Rotation in place: the first `rot` entries of each of n_heads heads (hd wide, side by side from column col0 of x [T, ld]
+// on) turn by pos * f_i, times `amp`. One block a token; pairs (2i, 2i + 1) or (i, i + rot / 2).
+__global__ void __launch_bounds__(256)
+rotate_heads_kernel(float* __restrict__ x, long long ld, int col0, int n_heads, int hd, int rot, int interleaved,
+                    const float* __restrict__ freq, float amp, const int* __restrict__ positions) {
+    extern __shared__ float sm[];
+    float* cs = sm;                 // [rot / 2]
+    float* sn = sm + rot / 2;
+    const int half = rot / 2;
+    pdl_trigger();
+    const float pos = (float)positions[blockIdx.x];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float c, s;
+        split_sincos(pos, freq[2 * i], freq[2 * i + 1], &c, &s);
+        cs[i] = c * amp;
+        sn[i] = s * amp;
+    }
+    pdl_wait();
+    __syncthreads();
+    float* row = x + (size_t)blockIdx.x * ld + col0;
+    for (int idx = threadIdx.x; idx < n_heads * half; idx += blockDim.x) {
+        const int i = idx % half;
+        float* h = row + (idx / half) * hd;
+        const int i0 = interleaved ? 2 * i : i, i1 = interleaved ? 2 * i + 1 : i + half;
+        const float u = h[i0], v = h[i1];
+        h[i0] = u * cs[i] - v * sn[i];
+        h[i1] = v * cs[i] + u * sn[i];
+    }
+}
+
+CELLM_API int cellm_rotate_heads(float* x, long long ld, int col0, int n_heads, int hd, int rot, int interleaved, const float* freq,
+                                 float amp, const int* positions, int T, cudaStream_t stream) {
+    if (T <= 0 || n_heads <= 0 || rot <= 0) return CELLM_OK;
+    if (rot > hd || rot % 2 || rot > 8192) return CELLM_ERR_SIZE;
+    if (!freq) return CELLM_ERR_ARG;
+    CELLM_RUN(rotate_heads_kernel, T, 256, (size_t)rot * sizeof(float), stream, x, ld, col0, n_heads, hd, rot, interleaved, freq, amp, positions);
+    return CELLM_OK;
+}
+
+// Mamba-2's inputs. Channels col0 .. col0 + C of proj (x | B | C side by side) pass a causal convolution over time with a
+// bias and silu into xbc [T, C]; the step sizes dt = softplus(proj[col_dt + h] + dt_bias_h) go to step [T, heads] and the
+// decays exp(-exp(A_log_h) dt) to decay [T, heads]. A thread a channel walks `run` tokens with the taps' inputs in
+// registers (TAPS > 0), or reads them anew for every token (TAPS 0: any number of taps). The last row of blocks forms the
+// step sizes.
+template <int TAPS>
+__global__ void __launch_bounds__(256)
+ssd_prep_kernel(float* __restrict__ xbc, float* __restrict__ step, float* __restrict__ decay, ConvTaps cv, const float* __restrict__ conv_bias,
+                const float* __restrict__ state_base, long long slot_stride, int n_slots, int col_dt, const float* __restrict__ dt_bias,
+                const float* __restrict__ A_log, const int* __restrict__ seq_of_token, const int* __restrict__ cu_seqlens,
+                const int* __restrict__ slot_ids, int T, int heads, int run, int* __restrict__ err) {
+    const int t0 = blockIdx.x * run, t1 = min(T, t0 + run);
+    pdl_trigger();
+    if (blockIdx.y == gridDim.y - 1) {
+        pdl_wait();
+        for (int i = threadIdx.x; i < (t1 - t0) * heads; i += blockDim.x) {
+            const int t = t0 + i / heads, h = i % heads;
+            const float dt = cellm_softplus(cv.proj[(size_t)t * cv.ld + col_dt + h] + dt_bias[h]);
+            step[(size_t)t * heads + h] = dt;
+            decay[(size_t)t * heads + h] = expf(-expf(A_log[h]) * dt);
+        }
+        return;
+    }
+    const int c = blockIdx.y * blockDim.x + threadIdx.x;
+    if (c >= cv.C) return;
+    const float bias = conv_bias[c];
+    float w[TAPS > 0 ? TAPS : 1], u[TAPS > 0 ? TAPS : 1];
+    if constexpr (TAPS > 0) {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[j] = cv.taps[(size_t)c * TAPS + j];
+    }
+    pdl_wait();
+    int end = -1, start = 0;
+    for (int t = t0; t < t1; ++t) {
+        bool fresh = t == t0;
+        if (t >= end) {         // another request's portion begins
+            const int b = seq_of_token[t];
+            start = cu_seqlens[b], end = cu_seqlens[b + 1];
+            int slot = slot_ids[b];
+            if (slot < 0 || slot >= n_slots) { atomicOr(err, CELLM_DEV_BAD_SLOT); slot = 0; }
+            cv.state = state_base ? state_base + (size_t)slot * slot_stride : nullptr;
+            fresh = true;
+        }
+        float y;
+        if constexpr (TAPS > 0) {
+            if (fresh) {
+#pragma unroll
+                for (int j = 0; j < TAPS - 1; ++j) {
+                    const int tt = t - (TAPS - 1) + j;
+                    u[j] = tt >= start ? cv.proj[(size_t)tt * cv.ld + cv.col0 + c] : cv.state[(size_t)(tt - start + TAPS - 1) * cv.C + c];
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < TAPS - 1; ++j) u[j] = u[j + 1];
+            }
+            u[TAPS - 1] = cv.proj[(size_t)t * cv.ld + cv.col0 + c];
+            y = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) y = fmaf(w[j], u[j], y);
+        } else {
+            y = conv_taps_at(cv, t, start, c);
+        }
+        y += bias;
+        xbc[(size_t)t * cv.C + c] = y * sigmoidf_(y);
+    }
+}
+
+CELLM_API int cellm_ssd_prep(float* xbc, float* step, float* decay, const float* proj, long long ld, int col0, int C, int col_dt,
+                             const float* taps, int n_taps, const float* conv_bias, const float* state, long long slot_stride,
+                             int n_slots, const float* dt_bias, const float* A_log, const int* seq_of_token, const int* cu_seqlens,
+                             const int* slot_ids, int T, int heads, int* err, cudaStream_t stream) {
+    if (T <= 0) return CELLM_OK;
+    if (C <= 0 || heads <= 0 || n_taps < 1 || n_taps > CONV_TAPS_MAX) return CELLM_ERR_SIZE;
+    if (n_taps > 1 && !state) return CELLM_ERR_ARG;
+    ConvTaps cv;
+    cv.proj = proj; cv.ld = ld; cv.col0 = col0; cv.bias = nullptr; cv.taps = taps; cv.state = nullptr; cv.n_taps = n_taps; cv.C = C;
+    const int run = T >= 512 ? 8 : 1;
+    const dim3 grid((unsigned)((T + run - 1) / run), (unsigned)((C + 255) / 256 + 1));
+#define SSD_PREP(N) CELLM_RUN(ssd_prep_kernel<N>, grid, 256, 0, stream, xbc, step, decay, cv, conv_bias, state, slot_stride, n_slots, col_dt, \
+                              dt_bias, A_log, seq_of_token, cu_seqlens, slot_ids, T, heads, run, err)
+    if (n_taps == 4) SSD_PREP(4);
+    else if (n_taps == 3) SSD_PREP(3);
+    else if (n_taps == 2) SSD_PREP(2);
+    else SSD_PREP(0);
+#undef SSD_PREP
+    return CELLM_OK;
+}
+
+// Mamba-2's way out of the recurrence: v = (o + D_h x) * silu(z), then v in `groups` equal parts, each divided by its own
+// root mean square, times w. A block a (token, group); the part's values wait in shared memory.
+template <typename TA>
+__global__ void __launch_bounds__(256)
+gated_group_norm_kernel(TA* __restrict__ out, const float* __restrict__ o, const float* __restrict__ x, long long ld_x,
+                        const float* __restrict__ D, const float* __restrict__ z, long long ld_z, const float* __restrict__ w, int inner,
+                        int vd, int Hg, float eps) {
+    extern __shared__ float vals[];      // [Hg]
+    __shared__ float scratch[32];
+    pdl_trigger();
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    const int lo = blockIdx.y * Hg;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < Hg; i += blockDim.x) {
+        const int c = lo + i;
+        const float g = z[t * ld_z + c];
+        float v = o[t * inner + c];
+        if (D) v = fmaf(D[c / vd], x[t * ld_x + c], v);
+        v *= g * sigmoidf_(g);
+        vals[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.f / sqrtf(ss / (float)Hg + eps);
+    for (int i = threadIdx.x; i < Hg; i += blockDim.x) out[t * inner + lo + i] = from_float<TA>(vals[i] * inv * w[lo + i]);
+}
+
+// o [T, inner] 32-bit (heads of vd side by side), x at pitch ld_x and z at pitch ld_z likewise; D [heads] (null: no term in
+// x); w [inner].
+CELLM_API int cellm_gated_group_norm(void* out, const float* o, const float* x, long long ld_x, const float* D, const float* z, long long ld_z,
+                                     const float* w, int T, int inner, int vd, int groups, float eps, int dtype, cudaStream_t stream) {
+    if (T <= 0) return CELLM_OK;
+    if (inner <= 0 || vd <= 0 || inner % vd || groups < 1 || inner % groups || groups > 65535) return CELLM_ERR_SIZE;
+    if (!z || !w || (D && !x)) return CELLM_ERR_ARG;
+    const int Hg = inner / groups;
+    const size_t smem = (size_t)Hg * sizeof(float);
+    if (smem > 200 * 1024) return CELLM_ERR_SIZE;
+    const int threads = Hg >= 256 ? 256 : Hg >= 128 ? 128 : 64;
+#define GGN_RUN(TA)                                                                                                          \
+    do {                                                                                                                      \
+        if (smem > 48 * 1024) {                                                                                               \
+            cudaError_t e = cudaFuncSetAttribute(gated_group_norm_kernel<TA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return (int)e;                                                                              \
+        }                                                                                                                     \
+        CELLM_RUN(gated_group_norm_kernel<TA>, dim3((unsigned)T, (unsigned)groups), threads, smem, stream, (TA*)out, o, x, ld_x, D, z, ld_z, w, \
+                  inner, vd, Hg, eps);                                                                                        \
+    } while (0)
+    if (dtype == CELLM_F32) GGN_RUN(float);
+    else if (dtype == CELLM_BF16) GGN_RUN(__nv_bfloat16);
+    else return CELLM_ERR_DTYPE;
+#undef GGN_RUN
+    return CELLM_OK;
+}
+
 // ------------------------------------------------------------------------------------------------ norm over a head's output
 // out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * w[:] (* sigmoid(gate[t, h, :])): a warp a (token, head). w is one row
-// of vd values for all heads, or (w_per_head) a row for every head.
+// of vd values for all heads, or (w_per_head) a row for every head, or null (no weight). gate_silu: the gate's factor is
+// silu(gate) instead.
 template <typename TA>
 __global__ void __launch_bounds__(256)
 head_norm_gate_kernel(TA* __restrict__ out, const float* __restrict__ o, const float* __restrict__ w,
-                      const float* __restrict__ gate, long long gate_ld, int n_rows, int heads, int vd, float eps, int w_per_head) {
+                      const float* __restrict__ gate, long long gate_ld, int n_rows, int heads, int vd, float eps, int w_per_head,
+                      int gate_silu) {
     pdl_trigger();
     pdl_wait();
     const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -696,22 +978,39 @@ head_norm_gate_kernel(TA* __restrict__ out, const float* __restrict__ o, const f
     const int t = r / heads, h = r % heads;
     const float* wr = w + (w_per_head ? (size_t)h * vd : 0);
     for (int j = lane; j < vd; j += 32) {
-        float y = x[j] * inv * wr[j];
-        if (gate) y *= sigmoidf_(gate[(size_t)t * gate_ld + (size_t)h * vd + j]);
+        float y = w ? x[j] * inv * wr[j] : x[j] * inv;
+        if (gate) {
+            const float g = gate[(size_t)t * gate_ld + (size_t)h * vd + j];
+            y *= gate_silu ? g * sigmoidf_(g) : sigmoidf_(g);
+        }
         out[(size_t)r * vd + j] = from_float<TA>(y);
     }
 }
 
-CELLM_API int cellm_head_norm_gate(void* out, const float* o, const float* w, const float* gate, long long gate_ld, int T,
-                                   int heads, int vd, float eps, int w_per_head, int dtype, cudaStream_t stream) {
+static int head_norm_impl(void* out, const float* o, const float* w, const float* gate, long long gate_ld, int T, int heads, int vd, float eps,
+                          int w_per_head, int gate_silu, int dtype, cudaStream_t stream) {
     if (T <= 0) return CELLM_OK;
     if (heads <= 0 || vd <= 0) return CELLM_ERR_SIZE;
     const int n_rows = T * heads;
     const unsigned blocks = (unsigned)((n_rows + 7) / 8);
     if (dtype == CELLM_F32)
-        CELLM_RUN(head_norm_gate_kernel<float>, blocks, 256, 0, stream, (float*)out, o, w, gate, gate_ld, n_rows, heads, vd, eps, w_per_head);
+        CELLM_RUN(head_norm_gate_kernel<float>, blocks, 256, 0, stream, (float*)out, o, w, gate, gate_ld, n_rows, heads, vd, eps, w_per_head, gate_silu);
     else if (dtype == CELLM_BF16)
-        CELLM_RUN(head_norm_gate_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)out, o, w, gate, gate_ld, n_rows, heads, vd, eps, w_per_head);
+        CELLM_RUN(head_norm_gate_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)out, o, w, gate, gate_ld, n_rows, heads, vd, eps, w_per_head,
+                  gate_silu);
     else return CELLM_ERR_DTYPE;
     return CELLM_OK;
+}
+
+CELLM_API int cellm_head_norm_gate(void* out, const float* o, const float* w, const float* gate, long long gate_ld, int T,
+                                   int heads, int vd, float eps, int w_per_head, int dtype, cudaStream_t stream) {
+    if (!w) return CELLM_ERR_ARG;
+    return head_norm_impl(out, o, w, gate, gate_ld, T, heads, vd, eps, w_per_head, 0, dtype, stream);
+}
+
+// The norm without a weight, times silu of the gate.
+CELLM_API int cellm_head_norm_silu(void* out, const float* o, const float* gate, long long gate_ld, int T, int heads, int vd, float eps,
+                                   int dtype, cudaStream_t stream) {
+    if (!gate) return CELLM_ERR_ARG;
+    return head_norm_impl(out, o, nullptr, gate, gate_ld, T, heads, vd, eps, 0, 1, dtype, stream);
 }

@@ -9,6 +9,10 @@
 //   the `top` experts with the largest c are chosen; their weights are s / (sum of the chosen s + 1e-20) * scale
 //   out = sum_k weight_k * D_k act(U_k h)  [+ sigmoid(g . h) * shared(h)]
 //
+// Two other forms share the parts around them: a router whose `top` experts are those with the largest z + bias and whose
+// weights are the softmax over the chosen of these sums (route_kernel<., 1>), and gated experts, D_k (silu(G_k h) * (U_k h)),
+// whose gate and up rows lie in blocks of 64 (expert_gate_up_kernel).
+//
 // Ties go to the lower index. The chosen experts are listed by descending c, and every sum runs in an order
 // that depends on the sizes alone, so a token's result does not depend on what else is in the batch.
 #include "common.cuh"
@@ -59,13 +63,12 @@ __device__ __forceinline__ void lane_dot4(float (&a)[4], float f, const TW* __re
     for (int j = 0; j < 4; ++j) a[j] += f * p[j];
 }
 
-// One output row of up to four experts at once (expert j: row w[j] against its own vector v[j], factor f[j]): the sum of
-// f[j] * (w[j] . v[j]) in the order of j, a lane's share. The experts' loads are issued together.
+// A lane's shares of up to four dot products w[j] . v[j]; the rows' loads are issued together.
 template <typename TW>
-__device__ __forceinline__ float lane_dot_experts(const TW* const (&w)[4], const float* const (&v)[4], const float (&f)[4], int count, int n, int lane,
-                                                  bool vec) {
+__device__ __forceinline__ void lane_dots(float (&p)[4], const TW* const (&w)[4], const float* const (&v)[4], int count, int n, int lane, bool vec) {
     constexpr int PER = 16 / (int)sizeof(TW);
-    float p[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) p[j] = 0.f;
     if (vec) {
 #pragma unroll 2
         for (int i = lane * PER; i < n; i += 32 * PER) {
@@ -93,6 +96,15 @@ __device__ __forceinline__ float lane_dot_experts(const TW* const (&w)[4], const
             for (int j = 0; j < 4; ++j)
                 if (j < count) p[j] += to_float(w[j][i]) * v[j][i];
     }
+}
+
+// One output row of up to four experts at once (expert j: row w[j] against its own vector v[j], factor f[j]): the sum of
+// f[j] * (w[j] . v[j]) in the order of j, a lane's share.
+template <typename TW>
+__device__ __forceinline__ float lane_dot_experts(const TW* const (&w)[4], const float* const (&v)[4], const float (&f)[4], int count, int n, int lane,
+                                                  bool vec) {
+    float p[4];
+    lane_dots<TW>(p, w, v, count, n, lane, vec);
     float a = 0.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j)
@@ -105,7 +117,8 @@ __device__ __forceinline__ float lane_dot_experts(const TW* const (&w)[4], const
 // warp a token, its scores in shared memory.
 #define ROUTE_THREADS 128
 
-template <typename TC>
+// MODE 0: sigmoid scores, a correction for the choice; MODE 1: the softmax over the chosen z + bias (`correction` the bias).
+template <typename TC, int MODE>
 __global__ void __launch_bounds__(ROUTE_THREADS)
 route_kernel(int* __restrict__ idx, float* __restrict__ wts, float* __restrict__ gate_out, const float* __restrict__ z_all, long long ldz,
              const TC* __restrict__ correction, int T, int E, int top, int n_groups, int keep, float scale, int has_gate) {
@@ -124,9 +137,13 @@ route_kernel(int* __restrict__ idx, float* __restrict__ wts, float* __restrict__
     const float* zr = z_all + (size_t)t * ldz;
     const int gsz = E / n_groups;
     for (int e = lane; e < E; e += 32) {
-        const float s = 1.f / (1.f + expf(-zr[e]));
-        z[e] = s;
-        c[e] = s + to_float(correction[e]);
+        if constexpr (MODE == 1) {
+            z[e] = c[e] = zr[e] + (correction ? to_float(correction[e]) : 0.f);
+        } else {
+            const float s = 1.f / (1.f + expf(-zr[e]));
+            z[e] = s;
+            c[e] = s + to_float(correction[e]);
+        }
     }
     if (has_gate && lane == 0) gate_out[t] = 1.f / (1.f + expf(-zr[E]));
     __syncwarp();
@@ -163,6 +180,12 @@ route_kernel(int* __restrict__ idx, float* __restrict__ wts, float* __restrict__
     }
     __syncwarp();
     float sum = 0.f;
+    if constexpr (MODE == 1) {      // chosen[0] is the largest
+        const float m = chosen[0];
+        for (int r = 0; r < top; ++r) sum += expf(chosen[r] - m);
+        for (int r = lane; r < top; r += 32) wts[(size_t)t * top + r] = expf(chosen[r] - m) / sum * scale;
+        return;
+    }
     for (int r = 0; r < top; ++r) sum += chosen[r];
     for (int r = lane; r < top; r += 32) wts[(size_t)t * top + r] = chosen[r] / (sum + 1e-20f) * scale;
 }
@@ -178,11 +201,31 @@ CELLM_API int cellm_route(int* idx, float* wts, float* gate_out, const float* z,
     if (smem > 48 * 1024) return CELLM_ERR_SIZE;
     const unsigned blocks = (unsigned)((T + ROUTE_THREADS / 32 - 1) / (ROUTE_THREADS / 32));
     if (c_dtype == CELLM_F32)
-        CELLM_RUN(route_kernel<float>, blocks, ROUTE_THREADS, smem, stream, idx, wts, gate_out, z, ldz, (const float*)correction, T, E, top,
+        CELLM_RUN((route_kernel<float, 0>), blocks, ROUTE_THREADS, smem, stream, idx, wts, gate_out, z, ldz, (const float*)correction, T, E, top,
                   n_groups, keep, scale, has_gate);
     else if (c_dtype == CELLM_BF16)
-        CELLM_RUN(route_kernel<__nv_bfloat16>, blocks, ROUTE_THREADS, smem, stream, idx, wts, gate_out, z, ldz, (const __nv_bfloat16*)correction,
+        CELLM_RUN((route_kernel<__nv_bfloat16, 0>), blocks, ROUTE_THREADS, smem, stream, idx, wts, gate_out, z, ldz, (const __nv_bfloat16*)correction,
                   T, E, top, n_groups, keep, scale, has_gate);
+    else return CELLM_ERR_DTYPE;
+    return CELLM_OK;
+}
+
+// The same for a router without sigmoids: the `top` largest z + bias are chosen (bias null: none) and weighed by the softmax
+// over them, times `scale`.
+CELLM_API int cellm_route_softmax(int* idx, float* wts, float* gate_out, const float* z, long long ldz, const void* bias, int b_dtype, int T,
+                                  int E, int top, float scale, int has_gate, cudaStream_t stream) {
+    if (T <= 0) return CELLM_OK;
+    if (E < 1 || top < 1 || top > E) return CELLM_ERR_SIZE;
+    if (has_gate && !gate_out) return CELLM_ERR_ARG;
+    const size_t smem = (size_t)(ROUTE_THREADS / 32) * (2 * E + 2 + top) * sizeof(float);
+    if (smem > 48 * 1024) return CELLM_ERR_SIZE;
+    const unsigned blocks = (unsigned)((T + ROUTE_THREADS / 32 - 1) / (ROUTE_THREADS / 32));
+    if (b_dtype == CELLM_F32)
+        CELLM_RUN((route_kernel<float, 1>), blocks, ROUTE_THREADS, smem, stream, idx, wts, gate_out, z, ldz, (const float*)bias, T, E, top, 1, 1,
+                  scale, has_gate);
+    else if (b_dtype == CELLM_BF16)
+        CELLM_RUN((route_kernel<__nv_bfloat16, 1>), blocks, ROUTE_THREADS, smem, stream, idx, wts, gate_out, z, ldz, (const __nv_bfloat16*)bias, T, E,
+                  top, 1, 1, scale, has_gate);
     else return CELLM_ERR_DTYPE;
     return CELLM_OK;
 }
@@ -236,10 +279,61 @@ expert_up_kernel(TA* __restrict__ mid, TA* __restrict__ smid, const TA* __restri
     }
 }
 
-// out[t, r] = sum_k wts[t, k] * (D_e mid[t * top + k])[r] (+ gate[t] * (D_s smid[t])[r]); down: [E * H, ff], D_s: [H, sff]
+// Gated experts: mid[t * top + k, j] = silu(G_e y[t])[j] * (U_e y[t])[j]. gu: [E * 2 ff, H] in blocks of 64 gate rows followed by
+// their 64 up rows (ff a multiple of 64); the shared expert's sgu [2 sff, H] likewise. A warp forms `rpw` (1 or 2)
+// neighbouring outputs, their gate and up rows in flight together.
 template <typename TA>
+__global__ void __launch_bounds__(EXPERT_THREADS)
+expert_gate_up_kernel(TA* __restrict__ mid, TA* __restrict__ smid, const TA* __restrict__ y, long long ldy, const TA* __restrict__ gu,
+                      const TA* __restrict__ sgu, const int* __restrict__ idx, int T, int H, int ff, int sff, int top, int E, int rpw) {
+    extern __shared__ __align__(16) float smem[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const bool is_shared = (int)blockIdx.x >= T * top;
+    const int slot = is_shared ? (int)blockIdx.x - T * top : (int)blockIdx.x;
+    const int t = is_shared ? slot : slot / top;
+    const int rows = is_shared ? sff : ff;
+    if ((int)blockIdx.y * EXPERT_WARPS * rpw >= rows) return;
+    const bool vec = rows_vectorise(is_shared ? sgu : gu, H, H);
+    pdl_trigger();
+    pdl_wait();
+    {
+        constexpr int PER = 16 / (int)sizeof(TA);
+        const TA* src = y + (size_t)t * ldy;
+        if (H % PER == 0 && (((uintptr_t)src) & 15) == 0) {
+            for (int i = threadIdx.x * PER; i < H; i += EXPERT_THREADS * PER) {
+                const uint4 x = *reinterpret_cast<const uint4*>(src + i);
+                const TA* xp = reinterpret_cast<const TA*>(&x);
+#pragma unroll
+                for (int k = 0; k < PER; ++k) smem[i + k] = to_float(xp[k]);
+            }
+        } else {
+            for (int i = threadIdx.x; i < H; i += EXPERT_THREADS) smem[i] = to_float(src[i]);
+        }
+    }
+    const TA* base = sgu;
+    if (!is_shared) base = gu + (size_t)min(max(idx[slot], 0), E - 1) * 2 * ff * H;
+    __syncthreads();
+    const int r0 = (blockIdx.y * EXPERT_WARPS + warp) * rpw, nr = min(rpw, rows - r0);
+    if (nr <= 0) return;
+    // output j's gate row lies in its block of 64 at (j / 64) * 128 + j % 64, its up row 64 further on; two neighbours that
+    // start at an even j share a block. Rows of the four slots: gate j, up j, gate j + 1, up j + 1.
+    const TA* w0 = base + ((size_t)(r0 / 64) * 128 + r0 % 64) * H;
+    const TA* w[4] = {w0, w0 + (size_t)64 * H, w0 + H, w0 + (size_t)65 * H};
+    const float* v[4] = {smem, smem, smem, smem};
+    const int count = 2 * nr;
+    float p[4];
+    lane_dots<TA>(p, w, v, count, H, lane, vec);
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+        const float g = warp_sum(p[2 * j]), u = warp_sum(p[2 * j + 1]);
+        if (lane == 0 && j < nr) (is_shared ? smid : mid)[(size_t)slot * rows + r0 + j] = from_float<TA>(g / (1.f + expf(-g)) * u);
+    }
+}
+
+// out[t, r] = sum_k wts[t, k] * (D_e mid[t * top + k])[r] (+ gate[t] * (D_s smid[t])[r]); down: [E * H, ff], D_s: [H, sff]
+template <typename TA, typename TO>
 __global__ void __launch_bounds__(EXPERT_DOWN_WARPS * 32)
-expert_down_kernel(TA* __restrict__ out, const TA* __restrict__ mid, const TA* __restrict__ smid, const TA* __restrict__ down,
+expert_down_kernel(TO* __restrict__ out, const TA* __restrict__ mid, const TA* __restrict__ smid, const TA* __restrict__ down,
                    const TA* __restrict__ sdown, const int* __restrict__ idx, const float* __restrict__ wts, const float* __restrict__ gate,
                    int H, int ff, int sff, int top, int E, int rpw) {
     extern __shared__ __align__(16) float smem[];   // [top * ff] the token's middles, [sff] the shared expert's, then [top] weights and experts
@@ -310,8 +404,65 @@ expert_down_kernel(TA* __restrict__ out, const TA* __restrict__ mid, const TA* _
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
         const float v = warp_sum(a[j]);
-        if (lane == 0 && j < nr) out[(size_t)t * H + r0 + j] = from_float<TA>(v);
+        if (lane == 0 && j < nr) out[(size_t)t * H + r0 + j] = from_float<TO>(v);
     }
+}
+
+// rows a warp forms: `most` where that still leaves some 600 blocks (four an SM) at work, else half as many, and so on
+static int expert_rows_a_warp(long long rows_in_all, int warps, int most, long long blocks_an_sm) {
+    static int sms = 0;
+    if (sms == 0) {
+        int dev = 0;
+        if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) sms = 148;
+    }
+    for (int r = most; r > 1; r /= 2)
+        if (rows_in_all / (warps * r) >= blocks_an_sm * sms) return r;
+    return 1;
+}
+
+// Both forms of the experts, row by row; `gated`: up and sup hold gate and up in blocks of 64.
+static int experts_rowwise_impl(void* out, void* mid, void* smid, const void* y, long long ldy, const void* up, const void* down,
+                                const void* sup, const void* sdown, const int* idx, const float* wts, const float* gate, int T, int H,
+                                int ff, int sff, int top, int E, int act, bool gated, int out_dtype, int dtype, cudaStream_t stream) {
+    if (T <= 0) return CELLM_OK;
+    if (H < 1 || ff < 1 || top < 1 || E < 1 || sff < 0) return CELLM_ERR_SIZE;
+    if ((sup == nullptr) != (sdown == nullptr) || (sup && (sff < 1 || !smid))) return CELLM_ERR_ARG;
+    if (!sup) sff = 0;
+    if (gated && (ff % 64 || sff % 64)) return CELLM_ERR_SIZE;
+    if (out_dtype != dtype && !(out_dtype == CELLM_F32 && dtype == CELLM_BF16)) return CELLM_ERR_DTYPE;
+    const size_t smem_up = (size_t)H * sizeof(float), smem_down = ((size_t)top * ff + sff + 2 * top) * sizeof(float);
+    if (smem_up > 200 * 1024 || smem_down > 200 * 1024) return CELLM_ERR_SIZE;
+    const int up_rows = ff > sff ? ff : sff;
+    const int rpw_up = expert_rows_a_warp((long long)T * top * ff + (sup ? (long long)T * sff : 0), EXPERT_WARPS, gated ? 2 : 4, 4);
+    const int rpw_down = expert_rows_a_warp((long long)T * H, EXPERT_DOWN_WARPS, 4, 2);
+    const dim3 grid_up((unsigned)(T * top + (sup ? T : 0)), (unsigned)((up_rows + EXPERT_WARPS * rpw_up - 1) / (EXPERT_WARPS * rpw_up)));
+    const dim3 grid_down((unsigned)T, (unsigned)((H + EXPERT_DOWN_WARPS * rpw_down - 1) / (EXPERT_DOWN_WARPS * rpw_down)));
+    if (grid_up.y > 65535 || grid_down.y > 65535) return CELLM_ERR_SIZE;
+#define GO(TA, TO)                                                                                                                \
+    do {                                                                                                                          \
+        static bool configured = false;                                                                                           \
+        if (!configured && (smem_up > 48 * 1024 || smem_down > 48 * 1024)) {                                                      \
+            cudaError_t e = cudaFuncSetAttribute(expert_up_kernel<TA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);  \
+            if (e == cudaSuccess) e = cudaFuncSetAttribute(expert_gate_up_kernel<TA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
+            if (e == cudaSuccess) e = cudaFuncSetAttribute(expert_down_kernel<TA, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
+            if (e != cudaSuccess) return (int)e;                                                                                  \
+            configured = true;                                                                                                    \
+        }                                                                                                                         \
+        if (gated)                                                                                                                \
+            CELLM_RUN(expert_gate_up_kernel<TA>, grid_up, EXPERT_THREADS, smem_up, stream, (TA*)mid, (TA*)smid, (const TA*)y, ldy, \
+                      (const TA*)up, (const TA*)sup, idx, T, H, ff, sff, top, E, rpw_up);                                         \
+        else                                                                                                                      \
+            CELLM_RUN(expert_up_kernel<TA>, grid_up, EXPERT_THREADS, smem_up, stream, (TA*)mid, (TA*)smid, (const TA*)y, ldy, (const TA*)up,  \
+                      (const TA*)sup, idx, T, H, ff, sff, top, E, act, rpw_up);                                                   \
+        CELLM_RUN((expert_down_kernel<TA, TO>), grid_down, EXPERT_DOWN_WARPS * 32, smem_down, stream, (TO*)out, (const TA*)mid, (const TA*)smid, \
+                  (const TA*)down, (const TA*)sdown, idx, wts, gate, H, ff, sff, top, E, rpw_down);                                \
+    } while (0)
+    if (dtype == CELLM_F32) GO(float, float);
+    else if (dtype == CELLM_BF16 && out_dtype == CELLM_F32) GO(__nv_bfloat16, float);
+    else if (dtype == CELLM_BF16) GO(__nv_bfloat16, __nv_bfloat16);
+    else return CELLM_ERR_DTYPE;
+#undef GO
+    return CELLM_OK;
 }
 
 // The chosen experts of every token, and the shared expert (sup null: none), walked row by row. mid: [T * top, ff] and
@@ -319,50 +470,15 @@ expert_down_kernel(TA* __restrict__ out, const TA* __restrict__ mid, const TA* _
 CELLM_API int cellm_experts_rowwise(void* out, void* mid, void* smid, const void* y, long long ldy, const void* up, const void* down,
                                     const void* sup, const void* sdown, const int* idx, const float* wts, const float* gate, int T, int H,
                                     int ff, int sff, int top, int E, int act, int dtype, cudaStream_t stream) {
-    if (T <= 0) return CELLM_OK;
-    if (H < 1 || ff < 1 || top < 1 || E < 1 || sff < 0) return CELLM_ERR_SIZE;
-    if ((sup == nullptr) != (sdown == nullptr) || (sup && (sff < 1 || !smid))) return CELLM_ERR_ARG;
-    if (!sup) sff = 0;
-    const size_t smem_up = (size_t)H * sizeof(float), smem_down = ((size_t)top * ff + sff + 2 * top) * sizeof(float);
-    if (smem_up > 200 * 1024 || smem_down > 200 * 1024) return CELLM_ERR_SIZE;
-    const int up_rows = ff > sff ? ff : sff;
-    // rows a warp: four where that still leaves some 600 blocks (four an SM) at work, else two, else one
-    static int sms = 0;
-    if (sms == 0) {
-        int dev = 0;
-        if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) sms = 148;
-    }
-    auto rows_a_warp = [&](long long rows_in_all) {
-        for (int r = 4; r > 1; r /= 2)
-            if (rows_in_all / (EXPERT_WARPS * r) >= 4LL * sms) return r;
-        return 1;
-    };
-    const int rpw_up = rows_a_warp((long long)T * top * ff + (sup ? (long long)T * sff : 0));
-    int rpw_down = 1;
-    for (int r = 4; r > 1; r /= 2)
-        if ((long long)T * H / (EXPERT_DOWN_WARPS * r) >= 2LL * sms) { rpw_down = r; break; }
-    const dim3 grid_up((unsigned)(T * top + (sup ? T : 0)), (unsigned)((up_rows + EXPERT_WARPS * rpw_up - 1) / (EXPERT_WARPS * rpw_up)));
-    const dim3 grid_down((unsigned)T, (unsigned)((H + EXPERT_DOWN_WARPS * rpw_down - 1) / (EXPERT_DOWN_WARPS * rpw_down)));
-    if (grid_up.y > 65535 || grid_down.y > 65535) return CELLM_ERR_SIZE;
-#define GO(TA)                                                                                                                    \
-    do {                                                                                                                          \
-        static bool configured = false;                                                                                           \
-        if (!configured && (smem_up > 48 * 1024 || smem_down > 48 * 1024)) {                                                      \
-            cudaError_t e = cudaFuncSetAttribute(expert_up_kernel<TA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);  \
-            if (e == cudaSuccess) e = cudaFuncSetAttribute(expert_down_kernel<TA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
-            if (e != cudaSuccess) return (int)e;                                                                                  \
-            configured = true;                                                                                                    \
-        }                                                                                                                         \
-        CELLM_RUN(expert_up_kernel<TA>, grid_up, EXPERT_THREADS, smem_up, stream, (TA*)mid, (TA*)smid, (const TA*)y, ldy, (const TA*)up,  \
-                  (const TA*)sup, idx, T, H, ff, sff, top, E, act, rpw_up);                                                               \
-        CELLM_RUN(expert_down_kernel<TA>, grid_down, EXPERT_DOWN_WARPS * 32, smem_down, stream, (TA*)out, (const TA*)mid, (const TA*)smid, \
-                  (const TA*)down, (const TA*)sdown, idx, wts, gate, H, ff, sff, top, E, rpw_down);                                         \
-    } while (0)
-    if (dtype == CELLM_F32) GO(float);
-    else if (dtype == CELLM_BF16) GO(__nv_bfloat16);
-    else return CELLM_ERR_DTYPE;
-#undef GO
-    return CELLM_OK;
+    return experts_rowwise_impl(out, mid, smid, y, ldy, up, down, sup, sdown, idx, wts, gate, T, H, ff, sff, top, E, act, false, dtype, dtype, stream);
+}
+
+// Gated experts (see expert_gate_up_kernel): gu [E * 2 ff, H], down [E * H, ff], sgu [2 sff, H], sdown [H, sff]; ff and sff
+// multiples of 64. out of element type out_dtype (the activations' or 32-bit).
+CELLM_API int cellm_experts_gated_rowwise(void* out, void* mid, void* smid, const void* y, long long ldy, const void* gu, const void* down,
+                                          const void* sgu, const void* sdown, const int* idx, const float* wts, const float* gate, int T, int H,
+                                          int ff, int sff, int top, int E, int out_dtype, int dtype, cudaStream_t stream) {
+    return experts_rowwise_impl(out, mid, smid, y, ldy, gu, down, sgu, sdown, idx, wts, gate, T, H, ff, sff, top, E, 0, true, out_dtype, dtype, stream);
 }
 
 // ---- a plain activation: h = act(u) for 32-bit sums u [T, n] (row pitch ld) ----------------------------------------------
@@ -476,7 +592,11 @@ CELLM_API int cellm_moe_gather(void* xs, const void* y, long long ldy, const int
 }
 
 // out[t, :] = sum_k wts[t, k] * Y[slot_row[t * top + k], :] (+ gate[t] * shared[t, :]), the sum in the order of k, 32-bit.
-__global__ void moe_combine_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ Y, const int* __restrict__ slot_row,
+__device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+__device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+
+template <typename TO>
+__global__ void moe_combine_kernel(TO* __restrict__ out, const __nv_bfloat16* __restrict__ Y, const int* __restrict__ slot_row,
                                    const float* __restrict__ wts, const float* __restrict__ shared, const float* __restrict__ gate, int H,
                                    int top) {
     pdl_trigger();
@@ -495,7 +615,7 @@ __global__ void moe_combine_kernel(__nv_bfloat16* __restrict__ out, const __nv_b
             a0 += g * shared[(size_t)t * H + c];
             a1 += g * shared[(size_t)t * H + c + 1];
         }
-        *reinterpret_cast<__nv_bfloat162*>(out + (size_t)t * H + c) = __floats2bfloat162_rn(a0, a1);
+        store_pair(out + (size_t)t * H + c, a0, a1);
     }
 }
 
@@ -503,6 +623,15 @@ CELLM_API int cellm_moe_combine(void* out, const void* Y, const int* slot_row, c
                                 int H, int top, cudaStream_t stream) {
     if (T <= 0) return CELLM_OK;
     if ((H & 1) || top < 1) return CELLM_ERR_SIZE;
-    CELLM_RUN(moe_combine_kernel, T, 256, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)Y, slot_row, wts, shared, gate, H, top);
+    CELLM_RUN(moe_combine_kernel<__nv_bfloat16>, T, 256, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)Y, slot_row, wts, shared, gate, H, top);
+    return CELLM_OK;
+}
+
+// The same with a 32-bit result.
+CELLM_API int cellm_moe_combine32(float* out, const void* Y, const int* slot_row, const float* wts, const float* shared, const float* gate, int T,
+                                  int H, int top, cudaStream_t stream) {
+    if (T <= 0) return CELLM_OK;
+    if ((H & 1) || top < 1) return CELLM_ERR_SIZE;
+    CELLM_RUN(moe_combine_kernel<float>, T, 256, 0, stream, out, (const __nv_bfloat16*)Y, slot_row, wts, shared, gate, H, top);
     return CELLM_OK;
 }

@@ -10,6 +10,8 @@
 //   token_gate_mul    out[t] = act(g[t]) * table[ids[t]][col0 .. col0 + n]     (a token's own row gated by the stream)
 //   scaled_rms_add    x[t] += m * y[t] / sqrt(mean(y[t]^2) + eps) * w
 //   weighted_sum2     out = ca * a + cb * b
+//   post_norm         x = r / sqrt(mean(r^2) + eps) * w with r = alpha * x + a;  y = x in the activations' type: a layer's
+//                     norm behind the sum (the stream itself is normed)
 //
 // Means, variances, factors and the stream are 32-bit. The variance is the mean of the squared deviations from the mean
 // (two passes over a row held in shared memory). A block's sums have a fixed order that depends on the width alone.
@@ -321,5 +323,93 @@ CELLM_API int cellm_head_gate_mul(void* o, const float* gate, long long gate_ld,
     if (dtype == CELLM_F32) CELLM_RUN(head_gate_mul_kernel<float>, blocks, 256, 0, stream, (float*)o, gate, gate_ld, heads, vd, total);
     else if (dtype == CELLM_BF16) CELLM_RUN(head_gate_mul_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)o, gate, gate_ld, heads, vd, total);
     else return CELLM_ERR_DTYPE;
+    return CELLM_OK;
+}
+
+// ---- the norm behind the sum -----------------------------------------------------------------------------------------
+// One block a row; the row's sums wait in registers (PER values of a thread in pieces of four; H at most PER * 4 * the
+// block's threads) or, for any other width, in shared memory.
+template <typename TA, typename TD, int PER>
+__global__ void __launch_bounds__(512)
+post_norm_kernel(TA* __restrict__ y, float* __restrict__ x, const TD* __restrict__ a, float alpha, const float* __restrict__ w, int H, float eps) {
+    extern __shared__ __align__(16) float row_s[];
+    __shared__ float scratch[32];
+    pdl_trigger();
+    pdl_wait();
+    const size_t base = (size_t)blockIdx.x * H;
+    float ss = 0.f;
+    if constexpr (PER > 0) {
+        float4 r[PER];
+#pragma unroll
+        for (int p = 0; p < PER; ++p) {
+            const int i = (threadIdx.x + p * blockDim.x) * 4;
+            r[p] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < H) {
+                const float4 v = ld4(x + base + i), u = ld4(a + base + i);
+                r[p] = make_float4(fmaf(alpha, v.x, u.x), fmaf(alpha, v.y, u.y), fmaf(alpha, v.z, u.z), fmaf(alpha, v.w, u.w));
+            }
+            ss = fmaf(r[p].x, r[p].x, ss), ss = fmaf(r[p].y, r[p].y, ss), ss = fmaf(r[p].z, r[p].z, ss), ss = fmaf(r[p].w, r[p].w, ss);
+        }
+        ss = block_sum(ss, scratch);
+        const float inv = 1.f / sqrtf(ss / (float)H + eps);
+#pragma unroll
+        for (int p = 0; p < PER; ++p) {
+            const int i = (threadIdx.x + p * blockDim.x) * 4;
+            if (i < H) {
+                const float4 g = ld4(w + i);
+                const float4 o = make_float4(r[p].x * inv * g.x, r[p].y * inv * g.y, r[p].z * inv * g.z, r[p].w * inv * g.w);
+                st4(x + base + i, o);
+                if (y) st4(y + base + i, o);
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < H; i += blockDim.x) {
+            const float v = fmaf(alpha, x[base + i], to_float(a[base + i]));
+            row_s[i] = v;
+            ss = fmaf(v, v, ss);
+        }
+        ss = block_sum(ss, scratch);
+        const float inv = 1.f / sqrtf(ss / (float)H + eps);
+        for (int i = threadIdx.x; i < H; i += blockDim.x) {
+            const float v = row_s[i] * inv * w[i];
+            x[base + i] = v;
+            if (y) y[base + i] = from_float<TA>(v);
+        }
+    }
+}
+
+// x [T, H] 32-bit, replaced; a [T, H] of element type add_dtype; w [H] 32-bit; y [T, H] of element type dtype (null: the
+// stream only).
+CELLM_API int cellm_post_norm(void* y, float* x, const void* a, int add_dtype, float alpha, const float* w, int T, int H, float eps, int dtype,
+                              cudaStream_t stream) {
+    if (T <= 0) return CELLM_OK;
+    if (H <= 0) return CELLM_ERR_SIZE;
+    if (!x || !a || !w) return CELLM_ERR_ARG;
+    const bool vec = H % 4 == 0 && H <= 8192 && on16(x) && on16(y) && on16(a) && on16(w);
+    const size_t smem = vec ? 0 : (size_t)H * sizeof(float);
+    if (smem > 200 * 1024) return CELLM_ERR_SIZE;
+#define PN_LAUNCH(TA, TD, PER, threads)                                                                                         \
+    do {                                                                                                                        \
+        if (smem > 48 * 1024) {                                                                                                 \
+            cudaError_t e = cudaFuncSetAttribute(post_norm_kernel<TA, TD, PER>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return (int)e;                                                                                \
+        }                                                                                                                       \
+        CELLM_RUN((post_norm_kernel<TA, TD, PER>), T, threads, smem, stream, (TA*)y, x, (const TD*)a, alpha, w, H, eps);         \
+    } while (0)
+#define PN_RUN(TA, TD)                                                                                                          \
+    do {                                                                                                                        \
+        if (!vec) PN_LAUNCH(TA, TD, 0, 256);                                                                                     \
+        else if (H <= 512) PN_LAUNCH(TA, TD, 1, 128);                                                                           \
+        else if (H <= 1024) PN_LAUNCH(TA, TD, 1, 256);                                                                          \
+        else if (H <= 2048) PN_LAUNCH(TA, TD, 1, 512);                                                                          \
+        else if (H <= 4096) PN_LAUNCH(TA, TD, 2, 512);                                                                          \
+        else PN_LAUNCH(TA, TD, 4, 512);                                                                                         \
+    } while (0)
+    if (dtype == CELLM_F32 && add_dtype == CELLM_F32) PN_RUN(float, float);
+    else if (dtype == CELLM_BF16 && add_dtype == CELLM_F32) PN_RUN(__nv_bfloat16, float);
+    else if (dtype == CELLM_BF16 && add_dtype == CELLM_BF16) PN_RUN(__nv_bfloat16, __nv_bfloat16);
+    else return CELLM_ERR_DTYPE;
+#undef PN_RUN
+#undef PN_LAUNCH
     return CELLM_OK;
 }

@@ -135,3 +135,29 @@ CELLM_API int cellm_bias_add(void* out, const float* in, const void* b, int w_dt
 #undef LAUNCH
     return CELLM_OK;
 }
+
+// The clamped gate (common.cuh: cellm_clamped_gate): h[t, j] = g' sigmoid(slope g') (u' + 1) with g' = min(gu[t, j], limit) and
+// u' = clamp(gu[t, ff + j], -limit, limit), from 32-bit gate and up.
+template <typename T>
+__global__ void __launch_bounds__(256)
+clamped_gate_kernel(T* __restrict__ h, const float* __restrict__ gu, long long ld, int ff, float limit, float slope, size_t n) {
+    pdl_trigger();
+    pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    const size_t t = i / ff;
+    const int j = (int)(i - t * ff);
+    h[i] = from_float<T>(cellm_clamped_gate(gu[t * ld + j], gu[t * ld + ff + j], limit, slope));
+}
+
+// gu [T, >= 2 ff] 32-bit at row pitch ld; h [T, ff]. limit may be infinite.
+CELLM_API int cellm_clamped_gate_act(void* h, const float* gu, long long ld, int T, int ff, float limit, float slope, int dtype, cudaStream_t stream) {
+    const size_t n = (size_t)T * ff;
+    if (n == 0) return CELLM_OK;
+    if (ld < 2LL * ff) return CELLM_ERR_SIZE;
+    const unsigned blocks = (unsigned)((n + 255) / 256);
+    if (dtype == CELLM_F32) CELLM_RUN(clamped_gate_kernel<float>, blocks, 256, 0, stream, (float*)h, gu, ld, ff, limit, slope, n);
+    else if (dtype == CELLM_BF16) CELLM_RUN(clamped_gate_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)h, gu, ld, ff, limit, slope, n);
+    else return CELLM_ERR_DTYPE;
+    return CELLM_OK;
+}

@@ -155,6 +155,15 @@ __device__ __forceinline__ float silu_mul(float g, float u) {
     return __fdividef(g, 1.0f + e) * u;
 }
 
+// How the epilogue over blocks of gate and up rows joins the two: kind 0 silu(g) * u; 1 the clamped gate (common.cuh).
+struct GateEpi {
+    int kind = 0;
+    float limit = 0.f, slope = 0.f;
+};
+__device__ __forceinline__ float gate_up(float g, float u, const GateEpi& e) {
+    return e.kind == 0 ? silu_mul(g, u) : cellm_clamped_gate_rounded(g, u, e.limit, e.slope);
+}
+
 // What the epilogue of in_proj needs for the gated short convolution of a decode step (every token of the step
 // belongs to a request of its own).
 struct ConvEpi {

@@ -10,6 +10,8 @@ CacheManager::CacheManager(int page_size, std::vector<GroupSpec> groups, int num
     if (page_size <= 0) throw CacheError("cache: page size must be positive");
     for (const auto& g : groups_) {
         if (g.window < 0 || g.keep_first < 0) throw CacheError("cache: a window and its kept first keys must not be negative");
+        if (g.chunk < 0 || (g.chunk > 0 && (g.window > 0 || g.keep_first > 0)))
+            throw CacheError("cache: a group reads chunks of positions or a window of keys, not both");
         allocs_.push_back(std::make_unique<BlockAllocator>(g.num_pages));
     }
 }
@@ -77,10 +79,10 @@ void CacheManager::commit(int64_t id, int new_total) {
                          std::to_string(rc.reserved));
     rc.tokens = new_total;
     for (size_t g = 0; g < groups_.size(); ++g) {
-        const int w = groups_[g].window;
-        if (w <= 0) continue;
-        // The next token sits at position >= tokens and reads keys >= tokens - w + 1.
-        const int first_key = rc.tokens - w + 1;
+        const int w = groups_[g].window, c = groups_[g].chunk;
+        if (w <= 0 && c <= 0) continue;
+        // The next token sits at position >= tokens and reads keys >= tokens - w + 1 (chunks: keys from its chunk's start on).
+        const int first_key = c > 0 ? rc.tokens / c * c : rc.tokens - w + 1;
         // pages that hold one of the kept first keys are never given back
         rc.first_live[g] = std::max(rc.first_live[g], std::min(blocks_for(groups_[g].keep_first), (int)rc.blocks[g].size()));
         while (rc.first_live[g] < (int)rc.blocks[g].size() &&
@@ -105,7 +107,8 @@ void CacheManager::release(int64_t id) {
 }
 
 int CacheManager::pages_for(int g, int tokens, int portion) const {
-    const int w = groups_.at((size_t)g).window;
+    // a chunk holds as many keys at its end as a window of its size
+    const int w = std::max(groups_.at((size_t)g).window, groups_.at((size_t)g).chunk);
     if (w <= 0) return blocks_for(tokens);
     // Live keys span at most window - 1 earlier keys plus one portion, and may
     // straddle page edges at both ends.

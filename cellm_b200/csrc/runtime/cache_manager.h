@@ -8,7 +8,8 @@
 // of fixed-size state. The reference's PageTable
 // (crates/cellm-cache/src/pagetable.rs:8-122) is the per-request block list of
 // one such group; it frees only on cancel (crates/cellm-sdk/src/lib.rs:401-403),
-// here pages also go back when a window has passed them.
+// here pages also go back when a window has passed them or a
+// chunk of positions has ended.
 #pragma once
 #include <cstdint>
 #include <map>
@@ -23,6 +24,7 @@ struct GroupSpec {
     int num_pages;
     int window;  // 0: every key is kept; w > 0: a token reads only the last w keys (itself included)
     int keep_first = 0;  // with a window: the sequence's first keep_first keys stay readable, so their pages are kept
+    int chunk = 0;   // c > 0 (instead of a window): a token reads the keys of its own run of c positions, counted from position 0
 };
 
 struct RequestCache {

@@ -74,6 +74,15 @@ typedef int (*GemmGroupedFn)(P c, CP a, CP w, int M, int N, int K, int groups, i
                              P err, P stream);
 typedef int (*ActivationFn)(P h, CP u, i64 ld, int T, int n, int act, int tag, P stream);
 
+typedef int (*RouteSoftmaxFn)(P idx, P wts, P gate, CP z, i64 ldz, CP bias, int b_tag, int T, int E, int top, float scale, int has_gate, P stream);
+typedef int (*ExpertsGatedRowwiseFn)(P out, P mid, P smid, CP y, i64 ldy, CP gu, CP down, CP sgu, CP sdown, CP idx, CP wts, CP gate, int T, int H,
+                                     int ff, int sff, int top, int E, int out_tag, int tag, P stream);
+typedef int (*GemmGatedFn)(P c, CP a, CP w, int M, int N, int K, i64 lda, i64 ldw, i64 ldc, int out_tag, int bn, int split_k, int gate_kind,
+                           float limit, float slope, int w_is_static, P ws, P counters, P err, P stream);
+typedef int (*GemmGroupedGatedFn)(P c, CP a, CP w, int M, int N, int K, int groups, i64 lda, i64 ldw, i64 ldc, int out_tag, CP tile_group,
+                                  int gate_kind, float limit, float slope, P err, P stream);
+typedef int (*ClampedGateFn)(P h, CP gu, i64 ld, int T, int ff, float limit, float slope, int tag, P stream);
+
 struct KernelError : std::runtime_error {
     int code;
     KernelError(const char* what, int c) : std::runtime_error(std::string(what) + ": status " + std::to_string(c)), code(c) {}
@@ -149,9 +158,11 @@ struct Run {
            "gemm_plain");
     }
 
-    // The tensor-core product with a given tile shape and split; c: [M, N] (or [M, N/2] with the SwiGLU epilogue).
+    // The tensor-core product with a given tile shape and split; c: [M, N] (or [M, N/2] with the epilogue over gate and up:
+    // `gate` names its kind where that is not SwiGLU).
+    struct Gate { int kind; float limit, slope; };
     void gemm_tc(void* c, const void* a, const ExecLinear& l, i64 M, i64 N, i64 lda, i64 out_dtype, i64 bn, i64 split_k,
-                 i64 epilogue, i64 ldc = -1) {
+                 i64 epilogue, i64 ldc = -1, const Gate* gate = nullptr) {
         if (ldc < 0) ldc = epilogue ? N / 2 : N;
         const i64 split = effective_split(l.K, split_k);
         // swapped tiles whose K split is one thread-block cluster (2..8 CTAs) sum their pieces through shared
@@ -167,6 +178,11 @@ struct Run {
         // plain tiles leave the sum of their K-split pieces to a second kernel; swapped tiles outside a cluster let
         // the last CTA of a tile sum them
         void* counters = (split > 1 && !in_cluster && bn < 0) ? s.counters : nullptr;
+        if (gate)
+            LAUNCH(fn<GemmGatedFn>(FN_GEMM_GATED)(c, a, l.w, (int)M, (int)N, (int)l.K, lda, l.ldw, ldc, (int)out_dtype, (int)bn, (int)split_k,
+                                              gate->kind, gate->limit, gate->slope, (int)p.static_flag, ws, counters, s.err, s.stream),
+               "gemm_gated_tcgen05");
+        else
         LAUNCH(fn<GemmTcFn>(FN_GEMM_TCGEN05)(c, a, l.w, (int)M, (int)N, (int)l.K, lda, l.ldw, ldc, (int)out_dtype, (int)bn,
                                          (int)split_k, (int)epilogue, (int)p.static_flag, ws, counters, s.err, s.stream),
            "gemm_tcgen05");
@@ -697,6 +713,27 @@ void Run::attention(const AttentionParams& L, const ExecItem& it, const void* x,
 
 void Run::gated_mlp(const GatedMlpParams& L, const void* x, void* out) {
     const i64 T = s.T, H = p.H;
+    const i64 out_dtype = L.out32 ? (i64)EXEC_F32 : act;
+    if (L.fused || L.act == 2) {
+        if (L.bg || L.bu || L.bd || L.extra) throw std::runtime_error("executor: biases or stacked rows beside a gate in the product's epilogue");
+        void* h = arena.take(T * L.ff * elt(act));
+        if (L.fused) {
+            if (act != EXEC_BF16 || !tc_ok(L.gate_up, H)) throw std::runtime_error("executor: activations do not fit the product with the gate in its epilogue");
+            i64 bn, split;
+            plan_tiles(T, L.gate_up.N, L.gate_up.K, p.sms, &bn, &split);
+            if (bn == 64) bn = 128;
+            else if (bn > 128 && bn < 256) bn = 256;
+            const Gate gate{L.act == 2 ? 1 : 0, (float)L.limit, (float)L.slope};
+            gemm_tc(h, x, L.gate_up, T, L.gate_up.N, H, act, bn, split, 1, -1, &gate);
+        } else {
+            void* gu = linear(x, L.gate_up, T, H, EXEC_F32);
+            LAUNCH(fn<ClampedGateFn>(FN_CLAMPED_GATE)(h, gu, L.gate_up.N, (int)T, (int)L.ff, (float)L.limit, (float)L.slope, (int)act, s.stream),
+                   "clamped_gate");
+        }
+        product(out, h, L.down, T, L.ff, out_dtype);
+        return;
+    }
+    if (L.out32 && L.bd) throw std::runtime_error("executor: a 32-bit result of a gated feed-forward with a bias");
     // gate and up stay 32-bit until act(g) * u is formed; the way back takes its bias before it is rounded
     void* gu = linear(x, L.gate_up, T, H, EXEC_F32);
     void* h = arena.take(T * L.ff * elt(act));
@@ -710,7 +747,7 @@ void Run::gated_mlp(const GatedMlpParams& L, const void* x, void* out) {
         void* sums = linear(h, L.down, T, L.ff, EXEC_F32);
         LAUNCH(fn<BiasAddFn>(FN_BIAS_ADD)(out, sums, L.bd, (int)L.b_dtype, (int)T, (int)L.down.N, (int)act, s.stream), "bias_add");
     } else {
-        product(out, h, L.down, T, L.ff, act);
+        product(out, h, L.down, T, L.ff, out_dtype);
     }
 }
 
@@ -718,11 +755,18 @@ void Run::routed_mlp(const RoutedMlpParams& L, const void* x, void* out) {
     const i64 T = s.T, H = p.H, e = elt(act);
     if (L.up.dtype != act || L.down.dtype != act || L.router.dtype != act)
         throw std::runtime_error("executor: experts whose element type differs from the activations'");
+    if (L.out32 && !L.gated && act != EXEC_F32) throw std::runtime_error("executor: a 32-bit result is built for gated experts");
     void* idx = arena.take(T * L.top * 4);
     void* wts = arena.take(T * L.top * 4);
     void* gate = L.shared_gate ? arena.take(T * 4) : nullptr;
     // the router's sums (and the shared expert's gate, one row more of the same matrix) as a product with 32-bit output
     void* z = linear(x, L.router, T, H, EXEC_F32);
+    const i64 out_dtype = L.out32 ? (i64)EXEC_F32 : act;
+    if (L.softmax)
+        LAUNCH(fn<RouteSoftmaxFn>(FN_ROUTE_SOFTMAX)(idx, wts, gate, z, L.router.N, L.correction, (int)L.c_dtype, (int)T, (int)L.experts, (int)L.top,
+                                                (float)L.scale, L.shared_gate ? 1 : 0, s.stream),
+               "route_softmax");
+    else
     LAUNCH(fn<RouteFn>(FN_ROUTE)(idx, wts, gate, z, L.router.N, L.correction, (int)L.c_dtype, (int)T, (int)L.experts, (int)L.top,
                              (int)L.n_groups, (int)L.keep, (float)L.scale, L.shared_gate ? 1 : 0, s.stream),
            "route");
@@ -731,6 +775,12 @@ void Run::routed_mlp(const RoutedMlpParams& L, const void* x, void* out) {
         // few tokens (and 32-bit): every token's chosen experts, and the shared one as one expert more, walked row by row
         void* mid = arena.take(T * L.top * L.ff * e);
         void* smid = L.shared_up.w ? arena.take(T * L.shared_ff * e) : nullptr;
+        if (L.gated)
+            LAUNCH(fn<ExpertsGatedRowwiseFn>(FN_EXPERTS_GATED_ROWWISE)(out, mid, smid, x, H, L.up.w, L.down.w, L.shared_up.w, L.shared_down.w, idx, wts,
+                                                                   gate, (int)T, (int)H, (int)L.ff, (int)L.shared_ff, (int)L.top, (int)L.experts,
+                                                                   (int)out_dtype, (int)act, s.stream),
+                   "experts_gated_rowwise");
+        else
         LAUNCH(fn<ExpertsRowwiseFn>(FN_EXPERTS_ROWWISE)(out, mid, smid, x, H, L.up.w, L.down.w, L.shared_up.w, L.shared_down.w, idx, wts, gate,
                                                     (int)T, (int)H, (int)L.ff, (int)L.shared_ff, (int)L.top, (int)L.experts, (int)L.act,
                                                     (int)act, s.stream),
@@ -742,7 +792,15 @@ void Run::routed_mlp(const RoutedMlpParams& L, const void* x, void* out) {
     void* shared = nullptr;
     if (L.shared_up.w) {
         void* h = arena.take(T * L.shared_ff * e);
-        if (tc_ok(L.shared_up, H)) {        // the activation on the 32-bit sums in the product's epilogue
+        if (L.gated) {
+            if (!tc_ok(L.shared_up, H)) throw std::runtime_error("executor: a shared expert's matrix that the tensor cores cannot read");
+            i64 bn, split;
+            plan_tiles(T, L.shared_up.N, H, p.sms, &bn, &split);
+            if (bn == 64) bn = 128;
+            else if (bn > 128 && bn < 256) bn = 256;
+            const Gate swiglu{0, 0.f, 0.f};
+            gemm_tc(h, x, L.shared_up, T, L.shared_up.N, H, act, bn, split, 1, -1, &swiglu);
+        } else if (tc_ok(L.shared_up, H)) {        // the activation on the 32-bit sums in the product's epilogue
             LAUNCH(fn<GemmGroupedFn>(FN_GEMM_GROUPED)(h, x, L.shared_up.w, (int)T, (int)L.shared_ff, (int)H, 1, H, L.shared_up.ldw, L.shared_ff,
                                                   (int)EXEC_BF16, nullptr, (int)L.act, s.err, s.stream),
                    "gemm_grouped_tcgen05");
@@ -763,6 +821,11 @@ void Run::routed_mlp(const RoutedMlpParams& L, const void* x, void* out) {
         void* xs = arena.take(rows * H * 2);
         LAUNCH(fn<MoeGatherFn>(FN_MOE_GATHER)(xs, x, H, row_slot, tile_group, (int)rows, (int)L.top, (int)H, s.stream), "moe_gather");
         void* mid = arena.take(rows * L.ff * 2);
+        if (L.gated)
+            LAUNCH(fn<GemmGroupedGatedFn>(FN_GEMM_GROUPED_GATED)(mid, xs, L.up.w, (int)rows, (int)(2 * L.ff), (int)H, (int)L.experts, H, L.up.ldw, L.ff,
+                                                             (int)EXEC_BF16, tile_group, 0, 0.f, 0.f, s.err, s.stream),
+                   "gemm_grouped_gated_tcgen05");
+        else
         LAUNCH(fn<GemmGroupedFn>(FN_GEMM_GROUPED)(mid, xs, L.up.w, (int)rows, (int)L.ff, (int)H, (int)L.experts, H, L.up.ldw, L.ff, (int)EXEC_BF16,
                                               tile_group, (int)L.act, s.err, s.stream),
                "gemm_grouped_tcgen05");
@@ -770,6 +833,9 @@ void Run::routed_mlp(const RoutedMlpParams& L, const void* x, void* out) {
         LAUNCH(fn<GemmGroupedFn>(FN_GEMM_GROUPED)(ys, mid, L.down.w, (int)rows, (int)H, (int)L.ff, (int)L.experts, L.ff, L.down.ldw, H,
                                               (int)EXEC_BF16, tile_group, -1, s.err, s.stream),
                "gemm_grouped_tcgen05");
+        if (L.out32)
+            LAUNCH(fn<MoeCombineFn>(FN_MOE_COMBINE32)(out, ys, slot_row, wts, shared, gate, (int)T, (int)H, (int)L.top, s.stream), "moe_combine32");
+        else
         LAUNCH(fn<MoeCombineFn>(FN_MOE_COMBINE)(out, ys, slot_row, wts, shared, gate, (int)T, (int)H, (int)L.top, s.stream), "moe_combine");
     }
 }

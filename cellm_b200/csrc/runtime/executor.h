@@ -118,11 +118,20 @@ struct LatentAttentionParams {
     const void* sinks;          // [heads] 32-bit: one more term exp(sink_h) in a head's denominator; null: none
 };
 // down . (act(gate . y + bg) * (up . y + bu)) + bd; act 0 silu, 1 gelu (tanh form); the biases may be null.
-struct GatedMlpParams { ExecLinear gate_up, down; const void* bg; const void* bu; const void* bd; i64 b_dtype, ff, act, extra; };
+// act 2, the clamped gate (no biases): g' sigmoid(slope g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit).
+// fused: gate_up holds blocks of 64 gate rows followed by their 64 up rows for the product's epilogue (act 0 or 2, ff a
+// multiple of 64, no biases). out32: the result is 32-bit (for a record run by itself).
+struct GatedMlpParams {
+    ExecLinear gate_up, down; const void* bg; const void* bu; const void* bd; i64 b_dtype, ff, act, extra;
+    i64 fused, out32; double limit, slope;
+};
 
 // Routed experts: out = sum over the token's `top` chosen experts of weight * down_e act(up_e y) (+ sigmoid(g . y) * shared(y)).
 // up: [experts * ff, H] and down: [experts * H, ff], the experts' matrices one below the other. router: [experts (+ 1), H], the
 // last row the shared expert's gate when it has one. The choice: see routed.cu. act: 0 gelu (erf), 1 gelu (tanh), 2 silu, 3 relu.
+// gated: the experts are down_e (silu(gate_e y) * (up_e y)); `up` (and shared_up) holds gate and up in blocks of 64 rows,
+// [experts * 2 ff, H], ff (and shared_ff) a multiple of 64; act is not read. softmax: the router chooses by the largest sums
+// (+ correction, a bias; null: none) and weighs by the softmax over the chosen. out32: as above.
 struct RoutedMlpParams {
     ExecLinear up, down, router;
     const void* correction; i64 c_dtype;
@@ -130,6 +139,7 @@ struct RoutedMlpParams {
     i64 ff, act;
     ExecLinear shared_up, shared_down;      // w null: no shared expert
     i64 shared_ff, shared_gate;
+    i64 gated, softmax, out32;
 };
 
 struct ExecOps { i64 n; const ExecOp* ops; };
@@ -152,7 +162,8 @@ enum ExecFn {
     FN_ATTENTION_DECODE, FN_ATTENTION_TC, FN_ATTENTION_FLASH, FN_GEMM_TCGEN05, FN_GEMM_CONV, FN_GEMM_ROPE,
     FN_GATED_NORM_ADD, FN_STREAM_CAST, FN_MINGRU_SCAN, FN_LATENT_PREP, FN_HEAD_PRODUCT, FN_GATED_ACT, FN_BIAS_ADD, FN_ATTENTION_LATENT, FN_HEAD_PRODUCT_MMA,
     FN_EMBED_POS, FN_ATTN_PREP, FN_ATTENTION_PLAIN_WIDE, FN_ROUTE, FN_EXPERTS_ROWWISE, FN_ACTIVATION, FN_ADD2_RMSNORM,
-    FN_MOE_SORT, FN_MOE_GATHER, FN_MOE_COMBINE, FN_GEMM_GROUPED, FN_ATTENTION_PLAIN_MASKED, FN_COUNT
+    FN_MOE_SORT, FN_MOE_GATHER, FN_MOE_COMBINE, FN_GEMM_GROUPED, FN_ATTENTION_PLAIN_MASKED,
+    FN_ROUTE_SOFTMAX, FN_EXPERTS_GATED_ROWWISE, FN_MOE_COMBINE32, FN_GEMM_GATED, FN_GEMM_GROUPED_GATED, FN_CLAMPED_GATE, FN_COUNT
 };
 
 struct ExecProgram {

@@ -68,6 +68,19 @@ _SIGNATURES = {
         "cellm_weighted_sum2": [P, P, F, P, F, L, I, P],
         "cellm_xielu": [P, P, L, I, I, P, I, P],
         "cellm_head_gate_mul": [P, P, L, I, I, I, I, P],
+        "cellm_route_softmax": [P, P, P, P, L, P, I, I, I, I, F, I, P],
+        "cellm_experts_gated_rowwise": [P, P, P, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
+        "cellm_moe_combine32": [P, P, P, P, P, P, I, I, I, P],
+        "cellm_clamped_gate_act": [P, P, L, I, I, F, F, I, P],
+        "cellm_embed_norm": [P, P, I, P, P, I, I, I, F, F, P, P],
+        "cellm_post_norm": [P, P, P, I, F, P, I, I, F, I, P],
+        "cellm_turned_attn_prep": [P, P, P, P, L, P, I, I, F, I, F, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, P],
+        "cellm_attention_plain_chunked": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P],
+        "cellm_decay_scan": [P, P, L, I, P, L, P, L, P, L, P, L, P, L, P, P, I, I, I, I, I, P, P],
+        "cellm_rotate_heads": [P, L, I, I, I, I, I, P, F, P, I, P],
+        "cellm_ssd_prep": [P, P, P, P, L, I, I, I, P, I, P, P, L, I, P, P, P, P, P, I, I, P, P],
+        "cellm_gated_group_norm": [P, P, P, L, P, P, L, P, I, I, I, I, F, I, P],
+        "cellm_head_norm_silu": [P, P, P, L, I, I, I, F, I, P],
     },
     "gemm_plain": {
         "cellm_gemm_plain": [P, P, P, I, I, I, L, L, L, I, I, P],
@@ -78,12 +91,14 @@ _SIGNATURES = {
     "attention_tc": {
         "cellm_attention_tc": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, P],
         "cellm_attention_tc_supports": [I, I, I, I],
+        "cellm_attention_tc_chunked": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, P],
         "cellm_attention_tc_gated": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, P, L, P, P],
     },
     "attention_flash": {
         "cellm_attention_flash": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, I, P, P],
         "cellm_attention_flash_supports": [I],
         "cellm_attention_flash_sink": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, I, P, P, I, P, P, P],
+        "cellm_attention_flash_chunked": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, I, P, P],
         "cellm_attention_flash_masked": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, I, I, P, P, L, P, P],
     },
     "attention_latent": {
@@ -94,6 +109,8 @@ _SIGNATURES = {
     "gemm_tcgen05": {
         "cellm_gemm_tcgen05": [P, P, P, I, I, I, L, L, L, I, I, I, I, I, P, P, P, P],
         "cellm_gemm_grouped_tcgen05": [P, P, P, I, I, I, I, L, L, L, I, P, I, P, P],
+        "cellm_gemm_gated_tcgen05": [P, P, P, I, I, I, L, L, L, I, I, I, I, F, F, I, P, P, P, P],
+        "cellm_gemm_grouped_gated_tcgen05": [P, P, P, I, I, I, I, L, L, L, I, P, I, F, F, P, P],
         "cellm_gemm_xielu_tcgen05": [P, P, P, I, I, I, L, L, L, I, P, P, P],
         "cellm_gemm_conv_tcgen05": [P, P, P, I, I, I, L, L, I, I, I, P, P, I, P, L, P, I, I, P, P],
         "cellm_gemm_rope_tcgen05": [P, P, P, I, I, L, L, I, I, P, P, F, P, P, I, P, P, I, I, I, I, P, I, P, P],

@@ -27,6 +27,18 @@ def embed(table: torch.Tensor, ids: torch.Tensor, err: torch.Tensor, scale: floa
     return out
 
 
+def embed_norm(table: torch.Tensor, ids: torch.Tensor, w: torch.Tensor, eps: float, err: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
+    """Rows of `table` [V, H] for int32 ids [T], times `scale`, RMS-normed with the float32 weight w [H], as float32 [T, H]."""
+    require_cuda(table, ids, w, err)
+    T, (V, H) = ids.numel(), table.shape
+    if w.dtype != torch.float32 or w.numel() != H:
+        raise ValueError("embed_norm: a float32 weight of the rows' width")
+    out = torch.empty((T, H), dtype=torch.float32, device=table.device)
+    check(fn(_LIB, "cellm_embed_norm")(ptr(out), ptr(table), tag(table), ptr(ids), ptr(w), T, H, V, float(scale), float(eps), ptr(err),
+                                       stream_of(table)), "embed_norm")
+    return out
+
+
 def add_rmsnorm(x: torch.Tensor, delta: Optional[torch.Tensor], w: torch.Tensor, eps: float,
                 act_dtype: torch.dtype, rows: Optional[torch.Tensor] = None, groups: int = 1) -> torch.Tensor:
     """x [*, H] float32 (+= delta in place when rows is None); returns the normed

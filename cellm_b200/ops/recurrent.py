@@ -7,7 +7,7 @@ from typing import Optional
 
 import torch
 
-from ._lib import check, fn, ptr, require_cuda, stream_of, tag
+from ._lib import check, count_launch, fn, ptr, require_cuda, stream_of, tag
 
 _LIB = "kernels_common"
 
@@ -287,3 +287,137 @@ def activation(u: torch.Tensor, act: str, act_dtype: torch.dtype) -> torch.Tenso
     check(fn(_LIB, "cellm_activation")(ptr(h), ptr(u), u.stride(0), T, n, {"gelu": 0, "gelu_tanh": 1, "silu": 2, "relu": 3, "relu2": 4, "tanh": 5}[act],
                                        tag(act_dtype), stream_of(u)), "activation")
     return h
+
+
+def turned_attn_prep(proj: torch.Tensor, freq, rot: int, interleaved: bool, amp: float, norm_eps: Optional[float], ctx, cache, nh: int, nkv: int,
+                     hd: int, vd: int, width: int, act_dtype: torch.dtype) -> torch.Tensor:
+    """Queries and keys turned (cos and sin times `amp`), then divided by each head's root mean square (norm_eps None: not);
+    k and v go to the token's page. proj [T, ld] float32 holds q | k | v (nkv = 0: q alone, nothing is written). Returns
+    q [T, nh * width] in `act_dtype`, zeros behind a head's own entries; rows of the pools are as wide as the cache's."""
+    _f32(proj, freq)
+    T = ctx.T
+    q = torch.empty((T, nh * width), dtype=act_dtype, device=proj.device)
+    k, v, bt = (cache.k, cache.v, cache.block_table) if nkv else (None, None, None)
+    if nkv and (k.dtype != act_dtype or v.dtype != act_dtype or k.shape[1:] != (nkv, cache.page_size, width) or v.shape[1:3] != k.shape[1:3]):
+        raise ValueError("turned_attn_prep: pools [pages, kv heads, page size, width] of the activations' element type")
+    check(fn(_LIB, "cellm_turned_attn_prep")(
+        ptr(q), ptr(k), ptr(v), ptr(proj), proj.stride(0), ptr(freq), int(rot), int(interleaved), float(amp), int(norm_eps is not None),
+        float(norm_eps or 0.0), ptr(ctx.positions), ptr(ctx.seq_of_token), ptr(bt), bt.stride(0) if nkv else 0, k.shape[0] if nkv else 0,
+        cache.page_size if nkv else 0, T, nh, nkv, hd, vd, width, v.shape[3] if nkv else 0, tag(act_dtype), ptr(ctx.err), stream_of(proj)),
+        "turned_attn_prep")
+    return q
+
+
+def attention_plain_chunked(q: torch.Tensor, cache, ctx, nh: int, nkv: int, hd: int, vd: int, scale: float, chunk: int) -> torch.Tensor:
+    """The plain attention in chunks: position i reads the keys j <= i with floor(j / chunk) = floor(i / chunk) (chunk 0: every
+    earlier key). q [T, nh * hd]; returns [T, nh * vd]."""
+    k, v, bt = cache.k, cache.v, cache.block_table
+    out = torch.empty((q.shape[0], nh * vd), dtype=q.dtype, device=q.device)
+    check(fn(_LIB, "cellm_attention_plain_chunked")(ptr(out), ptr(q), ptr(k), ptr(v), ptr(ctx.positions), ptr(ctx.seq_of_token), ptr(bt),
+                                                    bt.stride(0), k.shape[0], cache.page_size, q.shape[0], nh, nkv, hd, vd, float(scale), int(chunk),
+                                                    tag(q), ptr(ctx.err), stream_of(q)), "attention_plain_chunked")
+    return out
+
+
+FLASH_CHUNKED_WIDTHS = (32, 64, 96, 128)
+
+
+def attention_flash_chunked(q: torch.Tensor, cache, ctx, nh: int, nkv: int, hd: int, scale: float, chunk: int) -> torch.Tensor:
+    """The same on the tensor cores (bfloat16; keys and values of one width hd of 32, 64, 96 or 128)."""
+    k, v, bt = cache.k, cache.v, cache.block_table
+    if q.dtype != torch.bfloat16 or k.dtype != torch.bfloat16 or v.shape != k.shape or hd not in FLASH_CHUNKED_WIDTHS:
+        raise ValueError("attention_flash_chunked: bfloat16 and keys and values of one width of 32, 64, 96 or 128")
+    T, G = q.shape[0], nh // nkv
+    wide = ctx.max_q_len * G > 16
+    rows = 64 if wide else 16
+    n_tiles = sum(-(-n * G // rows) for n in ctx.q_lens)
+    longest = ctx.max_total_len
+    span = min(longest, chunk + ctx.max_q_len) if chunk > 0 else longest
+    nsplit = max(1, min(-(-span // 128), 296 // max(1, n_tiles * nkv), 32))
+    out = torch.empty((T, nh * hd), dtype=q.dtype, device=q.device)
+    part_o = part_ml = None
+    if nsplit > 1:
+        part_o = torch.empty((nsplit, T * nh, hd), dtype=torch.float32, device=q.device)
+        part_ml = torch.empty((nsplit, T * nh, 2), dtype=torch.float32, device=q.device)
+        count_launch()
+    check(fn("attention_flash", "cellm_attention_flash_chunked")(
+        ptr(out), ptr(part_o), ptr(part_ml), ptr(q), ptr(k), ptr(v), ptr(ctx.cu_seqlens), ptr(ctx.ctx_lens), ptr(bt), bt.stride(0),
+        ctx.B, T, n_tiles, k.shape[0], cache.page_size, nh, nkv, hd, float(scale), int(chunk), int(wide), nsplit, ptr(ctx.err),
+        stream_of(q)), "attention_flash_chunked")
+    return out
+
+
+def attention_tc_chunked(q: torch.Tensor, cache, ctx, nh: int, nkv: int, scale: float, chunk: int) -> torch.Tensor:
+    """The same for prompt portions on the tcgen05 tensor cores (heads of 64; attention_tc_supports says which sizes)."""
+    from .attention import attention_tc_supports
+    k, v, bt = cache.k, cache.v, cache.block_table
+    pages, _, page_size, hd = k.shape
+    if q.dtype != torch.bfloat16 or v.shape != k.shape or not attention_tc_supports(hd, nh, nkv, page_size) or scale <= 0:
+        raise ValueError("attention_tc_chunked: bfloat16, heads of 64, a group size dividing 128, pages of 8..128 tokens")
+    tok_per_cta = 256 // (nh // nkv)
+    n_tiles = sum((n + tok_per_cta - 1) // tok_per_cta for n in ctx.q_lens)
+    out = torch.empty_like(q)
+    check(fn("attention_tc", "cellm_attention_tc_chunked")(
+        ptr(out), ptr(q), ptr(k), ptr(v), ptr(ctx.cu_seqlens), ptr(ctx.ctx_lens), ptr(bt), bt.stride(0), ctx.B, q.shape[0], n_tiles, pages,
+        page_size, nh, nkv, hd, float(scale), int(chunk), ptr(ctx.err), stream_of(q)), "attention_tc_chunked")
+    return out
+
+
+def rotate_heads(x: torch.Tensor, col0: int, n_heads: int, hd: int, freq: torch.Tensor, rot: int, interleaved: bool, amp: float, positions) -> None:
+    """The first `rot` entries of n_heads heads of hd, side by side from column col0 of x [T, ld] float32 on, turn by the
+    token's position in place (cos and sin times `amp`)."""
+    _f32(x, freq)
+    check(fn(_LIB, "cellm_rotate_heads")(ptr(x), x.stride(0), int(col0), int(n_heads), int(hd), int(rot), int(interleaved), ptr(freq), float(amp),
+                                         ptr(positions), x.shape[0], stream_of(x)), "rotate_heads")
+
+
+def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, write: Optional[torch.Tensor], state: torch.Tensor, ctx,
+               heads: int, groups: int, dim: int, vd: int) -> torch.Tensor:
+    """S <- decay S + write k v^T, o = S^T q over every request's tokens of the step, one decay and one writing factor per
+    head; state [slots, heads, dim, vd] float32 is moved on. q, k [T, groups * dim] (head h reads group h / (heads / groups))
+    and v [T, heads * vd] float32, rows may be strided; decay and write [T, heads], or [heads] where they are constants
+    (write None: 1). Returns float32 [T, heads * vd]."""
+    _f32(q, k, v, decay, write, state)
+    pitch = lambda t: 0 if t is None or t.dim() == 1 else t.stride(0)
+    o = torch.empty((ctx.T, heads * vd), dtype=torch.float32, device=q.device)
+    check(fn(_LIB, "cellm_decay_scan")(ptr(o), ptr(state), state.stride(0), state.shape[0], ptr(q), q.stride(0), ptr(k), k.stride(0), ptr(v),
+                                       v.stride(0), ptr(decay), pitch(decay), ptr(write), pitch(write), ptr(ctx.cu_seqlens), ptr(ctx.slot_ids),
+                                       ctx.B, heads, groups, dim, vd, ptr(ctx.err), stream_of(q)), "decay_scan")
+    return o
+
+
+def ssd_prep(proj: torch.Tensor, col0: int, C: int, col_dt: int, taps: torch.Tensor, conv_bias: torch.Tensor, conv_state, dt_bias: torch.Tensor,
+             A_log: torch.Tensor, ctx, heads: int):
+    """Mamba-2's inputs: (silu(conv(columns col0 .. col0 + C of proj) + conv_bias) [T, C], step sizes softplus(proj + dt_bias)
+    [T, heads], decays exp(-exp(A_log) step) [T, heads]), all float32. taps [C, n]; conv_state [slots, n - 1, C] or None."""
+    _f32(proj, taps, conv_bias, conv_state, dt_bias, A_log)
+    T, dev = ctx.T, proj.device
+    xbc = torch.empty((T, C), dtype=torch.float32, device=dev)
+    step = torch.empty((T, heads), dtype=torch.float32, device=dev)
+    decay = torch.empty((T, heads), dtype=torch.float32, device=dev)
+    check(fn(_LIB, "cellm_ssd_prep")(ptr(xbc), ptr(step), ptr(decay), ptr(proj), proj.stride(0), int(col0), int(C), int(col_dt), ptr(taps),
+                                     taps.shape[1], ptr(conv_bias), ptr(conv_state), conv_state.stride(0) if conv_state is not None else 0,
+                                     conv_state.shape[0] if conv_state is not None else 1 << 30, ptr(dt_bias), ptr(A_log), ptr(ctx.seq_of_token),
+                                     ptr(ctx.cu_seqlens), ptr(ctx.slot_ids), T, heads, ptr(ctx.err), stream_of(proj)), "ssd_prep")
+    return xbc, step, decay
+
+
+def gated_group_norm(o: torch.Tensor, x: Optional[torch.Tensor], D: Optional[torch.Tensor], z: torch.Tensor, w: torch.Tensor, vd: int, groups: int,
+                     eps: float, act_dtype: torch.dtype) -> torch.Tensor:
+    """(o + D_h x) * silu(z), then each of `groups` equal parts of a row divided by its own root mean square, times w [inner].
+    o [T, inner] float32, heads of vd; x and z float32 with rows that may be strided (D None: no term in x)."""
+    _f32(o, x, D, z, w)
+    T, inner = o.shape
+    out = torch.empty((T, inner), dtype=act_dtype, device=o.device)
+    check(fn(_LIB, "cellm_gated_group_norm")(ptr(out), ptr(o), ptr(x), x.stride(0) if x is not None else 0, ptr(D), ptr(z), z.stride(0), ptr(w), T,
+                                             inner, vd, int(groups), float(eps), tag(act_dtype), stream_of(o)), "gated_group_norm")
+    return out
+
+
+def head_norm_silu(o: torch.Tensor, gate: torch.Tensor, heads: int, vd: int, eps: float, act_dtype: torch.dtype) -> torch.Tensor:
+    """o [T, heads * vd] float32 -> o / rms over each head * silu(gate [T, heads * vd] float32, rows may be strided)."""
+    _f32(o, gate)
+    out = torch.empty(o.shape, dtype=act_dtype, device=o.device)
+    check(fn(_LIB, "cellm_head_norm_silu")(ptr(out), ptr(o), ptr(gate), gate.stride(0), o.shape[0], heads, vd, float(eps), tag(act_dtype),
+                                           stream_of(o)), "head_norm_silu")
+    return out

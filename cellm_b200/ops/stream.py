@@ -1,6 +1,7 @@
 """Python entry points of the kernels around the 32-bit residual stream of layers that run their sublayers one after
 the other and add each result times a constant (norms with a mean and a bias, the start of another pass over the same
-layers, a token's own row gated by the stream), and of the activation with learned numbers."""
+layers, a token's own row gated by the stream) or norm the stream behind each sum, and of the activation with learned
+numbers."""
 from __future__ import annotations
 
 from typing import Optional
@@ -99,3 +100,17 @@ def head_gate_mul(o: torch.Tensor, gate: torch.Tensor, heads: int) -> torch.Tens
     T = o.shape[0]
     check(fn(_LIB, "cellm_head_gate_mul")(ptr(o), ptr(gate), gate.stride(0), T, heads, o.shape[1] // heads, tag(o), stream_of(o)), "head_gate_mul")
     return o
+
+
+def post_norm(x: torch.Tensor, a: torch.Tensor, alpha: float, w: torch.Tensor, eps: float, act_dtype: torch.dtype) -> torch.Tensor:
+    """x [T, H] float32 becomes r / sqrt(mean(r^2) + eps) * w with r = alpha * x + a, in place; returns the new stream in
+    `act_dtype` (x itself for float32). a [T, H] float32 or `act_dtype`, w [H] float32."""
+    require_cuda(x, a, w)
+    _f32(x, w)
+    T, H = x.shape
+    if a.shape != x.shape or w.numel() != H:
+        raise ValueError("post_norm: a result of the stream's shape and a weight of its width")
+    y = torch.empty((T, H), dtype=act_dtype, device=x.device) if act_dtype != torch.float32 else None
+    check(fn(_LIB, "cellm_post_norm")(ptr(y), ptr(x), ptr(a), tag(a), float(alpha), ptr(w), T, H, float(eps), tag(act_dtype), stream_of(x)),
+          "post_norm")
+    return y if y is not None else x

@@ -273,3 +273,47 @@ class ScaledPreNormBlock(Block):
 
 
 register_block("pre_norm_scaled", ScaledPreNormBlock)
+
+
+class PostNormBlock(Block):
+    """A layer whose sublayers read the residual stream itself and whose norms sit behind the sums, so that the stream is
+    normed after each of them:
+
+        x <- norm1(alpha x + mixer(x));    x <- norm2(alpha x + feed_forward(x))      (the layer may have no feed-forward)
+
+    Sum and norm are one kernel, which also leaves the stream in the activations' type for what reads it next: the
+    feed-forward, or the mixer of the next item of the run order. The norms must be RMS norms without groups; the stream,
+    the sums and the norms are 32-bit.
+
+    params: alpha (default 1)."""
+    graph_safe = True
+
+    def __init__(self, mixer_norm, mixer, feed_forward_norm, feed_forward, params=None, weights=None, dtype=None):
+        import torch
+        from ..config.errors import ConfigError
+        self.mixer, self.feed_forward, self.dtype = mixer, feed_forward, dtype
+        self.mixer_norm, self.feed_forward_norm = mixer_norm, feed_forward_norm
+        self.alpha = float((params or {}).get("alpha", 1.0))
+        if (feed_forward is None) != (feed_forward_norm is None):
+            raise ConfigError("post_norm: a feed-forward and its norm come together")
+        for n in (mixer_norm, feed_forward_norm):
+            if n is not None and (not all(hasattr(n, a) for a in ("weight", "eps", "groups")) or n.groups != 1):
+                raise ConfigError("post_norm: the norms must be RMS norms without groups")
+        self.w1 = mixer_norm.weight.to(torch.float32).contiguous()
+        self.w2 = feed_forward_norm.weight.to(torch.float32).contiguous() if feed_forward_norm is not None else None
+
+    def forward(self, residual: Residual, ctx: StepContext, cache: CacheBinding) -> None:
+        from .. import ops
+        x = residual.flush()
+        item = ctx.extras.get("order_item", 0)
+        # the block of the item before this one left the stream in the activations' type
+        before, h = ctx.extras.pop("stream_after_item", (None, None))
+        if before is None or before != item - 1:
+            h = ops.stream_cast(x, self.dtype)
+        h = ops.post_norm(x, self.mixer.forward(h, ctx, cache), self.alpha, self.w1, self.mixer_norm.eps, self.dtype)
+        if self.feed_forward is not None:
+            h = ops.post_norm(x, self.feed_forward.forward(h, ctx), self.alpha, self.w2, self.feed_forward_norm.eps, self.dtype)
+        ctx.extras["stream_after_item"] = (item, h)
+
+
+register_block("post_norm", PostNormBlock)

@@ -7,6 +7,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
+from ..config.errors import ConfigError
 from .base import Embedding, Head, TensorSpec
 from .linear import Linear
 from .registry import register_embedding, register_head
@@ -16,13 +17,16 @@ class TokenEmbedding(Embedding):
     graph_safe = True
 
     """params: vocab_size, dim, scale (default 1: the row as it is), max_positions (default 0: none; else a table of
-    learned position vectors is added, unscaled). weights: weight [vocab, dim], positions [max_positions, dim]."""
+    learned position vectors is added, unscaled), norm_eps (None; else the row is RMS-normed with a weight, in the look-up's
+    kernel). weights: weight [vocab, dim], positions [max_positions, dim], norm [dim]."""
 
     @classmethod
     def weight_specs(cls, params):
         specs = {"weight": TensorSpec((params["vocab_size"], params["dim"]), "embedding")}
         if params.get("max_positions"):
             specs["positions"] = TensorSpec((params["max_positions"], params["dim"]), "embedding")
+        if params.get("norm_eps") is not None:
+            specs["norm"] = TensorSpec((params["dim"],), "norm")
         return specs
 
     def __init__(self, params: dict, weights: dict, dtype: torch.dtype):
@@ -31,14 +35,23 @@ class TokenEmbedding(Embedding):
         self.positions = None
         if params.get("max_positions"):
             self.positions = weights["positions"].to(self.weight.dtype).contiguous()
+        self.norm_eps, self.norm_w = params.get("norm_eps"), None
+        if self.norm_eps is not None:
+            if self.positions is not None:
+                raise ConfigError("lookup: a norm over the row beside position vectors is not built")
+            self.norm_w = weights["norm"].to(torch.float32).contiguous()
 
     def emit(self, emitter) -> None:
+        if self.norm_w is not None:
+            return super().emit(emitter)
         from ..ops._lib import tag
         from ..runtime import records as R
         n = 0 if self.positions is None else self.positions.shape[0]
         emitter.native(R.EMBED, R.EmbedParams(self.weight.data_ptr(), tag(self.weight), self.scale, R.ptr(self.positions), n), part=self)
 
     def forward(self, token_ids: torch.Tensor, ctx) -> torch.Tensor:
+        if self.norm_w is not None:
+            return ops.embed_norm(self.weight, token_ids, self.norm_w, float(self.norm_eps), ctx.err, self.scale)
         return ops.embed(self.weight, token_ids, ctx.err, self.scale, self.positions, ctx.positions if self.positions is not None else None)
 
 

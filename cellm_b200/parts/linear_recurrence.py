@@ -24,12 +24,25 @@
     S <- diag(d) S - (a * u)(u^T S) + k v^T (the old S on the right);   o = S^T r
     out = W_o (rms_norm(o per head) * w * sigmoid(W_g h))    (w: a row for every head)
 
+`retention`: linear attention with one constant decay per head.
+
+    q, k, v = W h;   the first `rotary_dim` entries of every q and k head turn by the token's position
+    S <- d_h S + dim^(-1/2) k v^T        o = S^T q
+    out = W_o (rms_norm(o per head, no weight) * silu(W_g h))
+
+`mamba2`: Mamba-2's state-space duality, one decay per head and token.
+
+    z | x | B | C | dt = W_in h;   x, B, C = silu(conv(x | B | C) + bias)   (a short causal convolution over time per channel)
+    dt = softplus(dt + dt_bias);   S <- exp(-exp(A_log_h) dt) S + dt B x^T;   y = S^T C + D_h x    (head h reads the B and C of
+    group floor(h / (heads / groups)))
+    out = W_o (rms_norm(y * silu(z), each of `norm_groups` equal parts by itself) * w)
+
 `weighted_pair`: two mixers side by side over the same input, out = a * first(h) + b * second(h) with constants a, b.
 
 Everything that enters a recurrence is 32-bit (the projections keep their 32-bit sums; gates, decays, unit vectors and
 the state are computed in 32-bit), and a request's tokens are walked in order from the state the step before left, so
-the state after a token does not depend on how the sequence was cut. The delta rule also keeps the convolution's last
-taps - 1 projected rows in the slot."""
+the state after a token does not depend on how the sequence was cut. The gated delta rule and Mamba-2 also keep the
+convolution's last taps - 1 projected rows in the slot."""
 from __future__ import annotations
 
 import torch
@@ -37,7 +50,7 @@ import torch
 from ..config.errors import ConfigError
 from .base import CacheBinding, FixedState, Mixer, StepContext, TensorSpec
 from .linear import Linear, stack_rows
-from .registry import register_mixer
+from .registry import part_class, register_mixer
 from .sink_attention import bindings_of
 
 
@@ -208,6 +221,119 @@ class GeneralDeltaMixer(Mixer):
 
 
 register_mixer("general_delta", GeneralDeltaMixer)
+
+
+class RetentionMixer(Mixer):
+    graph_safe = True
+
+    """params: hidden_size, heads, dim, value_dim, decay (a list of one number per head), eps, position (PartSpec of a rotation,
+    or None), out_dtype32 (default False).
+    weights: q, k [heads*dim, H]; v, g [heads*vd, H]; o [H, heads*vd]."""
+
+    @classmethod
+    def weight_specs(cls, params):
+        H, h, d, vd = (int(params[k]) for k in ("hidden_size", "heads", "dim", "value_dim"))
+        return {"q": TensorSpec((h * d, H), "linear"), "k": TensorSpec((h * d, H), "linear"), "v": TensorSpec((h * vd, H), "linear"),
+                "g": TensorSpec((h * vd, H), "linear"), "o": TensorSpec((H, h * vd), "linear")}
+
+    @classmethod
+    def cache_need(cls, params):
+        return FixedState((int(params["heads"]), int(params["dim"]), int(params["value_dim"])), torch.float32)
+
+    def __init__(self, params: dict, weights: dict, dtype: torch.dtype):
+        self.H, self.heads, self.dim, self.vd = (int(params[k]) for k in ("hidden_size", "heads", "dim", "value_dim"))
+        self.eps, self.dtype = float(params["eps"]), dtype
+        decay = [float(x) for x in params["decay"]]
+        if len(decay) != self.heads:
+            raise ConfigError(f"retention: {len(decay)} decays for {self.heads} heads")
+        dev = weights["q"].device
+        self.in_proj = Linear(stack_rows(weights["q"], weights["k"], weights["v"], weights["g"]), dtype)
+        self.out_proj = Linear(weights["o"], dtype)
+        self.out32 = bool(params.get("out_dtype32", False))
+        self.decay = torch.tensor(decay, dtype=torch.float32, device=dev)
+        # k's factor dim^(-1/2), as the factor with which a head writes
+        self.write = torch.full((self.heads,), self.dim ** -0.5, dtype=torch.float32, device=dev)
+        pos = params.get("position")
+        self.position = part_class("position", pos.kind)(pos.params, dev) if pos is not None else None
+        self.rot, self.interleaved, self.freq, self.amp = 0, False, None, 1.0
+        if self.position is not None:
+            r = self.position.rotation(amplitude=True)
+            if r is None:
+                raise ConfigError("retention: the position encoding must be a rotation")
+            self.rot, self.interleaved, self.freq, self.amp = int(r[0]), bool(r[1]), r[2], float(self.position.amplitude)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheBinding) -> torch.Tensor:
+        from .. import ops
+        state = bindings_of(cache, 1)[0].state
+        hd, hv = self.heads * self.dim, self.heads * self.vd
+        proj = self.in_proj(x, out_dtype=torch.float32)
+        if self.rot:
+            ops.rotate_heads(proj, 0, 2 * self.heads, self.dim, self.freq, self.rot, self.interleaved, self.amp, ctx.positions)
+        o = ops.decay_scan(proj, proj[:, hd:], proj[:, 2 * hd:], self.decay, self.write, state, ctx, self.heads, self.heads, self.dim, self.vd)
+        y = ops.head_norm_silu(o, proj[:, 2 * hd + hv:], self.heads, self.vd, self.eps, self.dtype)
+        return self.out_proj(y, out_dtype=torch.float32 if self.out32 else None)
+
+
+register_mixer("retention", RetentionMixer)
+
+
+class Mamba2Mixer(Mixer):
+    graph_safe = True
+
+    """params: hidden_size, heads, value_dim, state (rows of a head's state), groups (default 1), norm_groups (default 1),
+    conv_taps, eps, out_dtype32 (default False).
+    weights: in [2 * heads*vd + 2 * groups*state + heads, H]; conv [heads*vd + 2 * groups*state, taps], conv_bias; dt_bias,
+    A_log, D [heads]; norm [heads*vd]; o [H, heads*vd]."""
+
+    @classmethod
+    def _sizes(cls, params):
+        h, vd, n, g = (int(params[k]) for k in ("heads", "value_dim", "state", "groups"))
+        return h, vd, n, g, h * vd, h * vd + 2 * g * n
+
+    @classmethod
+    def weight_specs(cls, params):
+        H, taps = int(params["hidden_size"]), int(params["conv_taps"])
+        h, vd, n, g, inner, C = cls._sizes(params)
+        return {"in": TensorSpec((inner + C + h, H), "linear"), "conv": TensorSpec((C, taps), "conv_tap_wide"), "conv_bias": TensorSpec((C,), "bias"),
+                "dt_bias": TensorSpec((h,), "bias"), "A_log": TensorSpec((h,), "log_rate"), "D": TensorSpec((h,), "norm"),
+                "norm": TensorSpec((inner,), "norm"), "o": TensorSpec((H, inner), "linear")}
+
+    @classmethod
+    def cache_need(cls, params):
+        h, vd, n, g, inner, C = cls._sizes(params)
+        state, taps = FixedState((h, n, vd), torch.float32), int(params["conv_taps"])
+        return (FixedState((taps - 1, C), torch.float32), state) if taps > 1 else state
+
+    def __init__(self, params: dict, weights: dict, dtype: torch.dtype):
+        self.heads, self.vd, self.n, self.groups, self.inner, self.C = self._sizes(params)
+        self.norm_groups, self.taps = int(params.get("norm_groups", 1)), int(params["conv_taps"])
+        if self.heads % self.groups:
+            raise ConfigError(f"mamba2: {self.heads} heads are not a multiple of {self.groups} groups")
+        if self.norm_groups < 1 or self.inner % self.norm_groups:
+            raise ConfigError(f"mamba2: {self.inner} values do not form {self.norm_groups} equal parts")
+        self.eps, self.dtype = float(params["eps"]), dtype
+        self.in_proj, self.out_proj = Linear(weights["in"], dtype), Linear(weights["o"], dtype)
+        self.out32 = bool(params.get("out_dtype32", False))
+        self.conv_w = weights["conv"].to(torch.float32).contiguous()
+        self.conv_b, self.dt_bias, self.A_log, self.D, self.norm_w = (_f32(weights, k) for k in ("conv_bias", "dt_bias", "A_log", "D", "norm"))
+        self.n_needs = 2 if self.taps > 1 else 1
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheBinding) -> torch.Tensor:
+        from .. import ops
+        b = bindings_of(cache, self.n_needs)
+        conv_state, state = (b[0].state if self.taps > 1 else None), b[-1].state
+        inner, gn = self.inner, self.groups * self.n
+        proj = self.in_proj(x, out_dtype=torch.float32)
+        xbc, step, decay = ops.ssd_prep(proj, inner, self.C, inner + self.C, self.conv_w, self.conv_b, conv_state, self.dt_bias, self.A_log, ctx,
+                                        self.heads)
+        if conv_state is not None:
+            ops.conv_state_update(conv_state, proj, inner, None, self.taps, ctx)
+        o = ops.decay_scan(xbc[:, inner + gn:], xbc[:, inner:], xbc, decay, step, state, ctx, self.heads, self.groups, self.n, self.vd)
+        y = ops.gated_group_norm(o, xbc, self.D, proj, self.norm_w, self.vd, self.norm_groups, self.eps, self.dtype)
+        return self.out_proj(y, out_dtype=torch.float32 if self.out32 else None)
+
+
+register_mixer("mamba2", Mamba2Mixer)
 
 
 class SideBySideMixer(Mixer):

@@ -7,14 +7,19 @@ that every token runs.
     the `top` experts with the largest c are chosen; weight_k = s_k / (sum of the chosen s + 1e-20) * route_scale
     out = sum_k weight_k * D_k act(U_k h)  +  sigmoid(g . h) * D_s act(U_s h)
 
-The experts' matrices are kept one below the other, so that a kernel reaches expert e by an offset. The router's
-rows and the shared expert's gate row form one matrix."""
+Two choices are parameters. `scores` "softmax": the `top` experts with the largest z + bias are chosen and weighed by the
+softmax over the chosen sums (no sigmoid, no groups). `gated`: an expert (the shared one too) is D (silu(G h) * (U h)).
+
+The experts' matrices are kept one below the other, so that a kernel reaches expert e by an offset; gate and up rows of
+gated experts lie in blocks of 64, so that the grouped product's epilogue joins the two (widths are padded to multiples of
+64 with zeros). The router's rows and the shared expert's gate row form one matrix."""
 from __future__ import annotations
 
 import torch
 
 from ..config.errors import ConfigError
 from .base import FeedForward, StepContext, TensorSpec
+from .gated_mlp import blocked_gate_up, widened_columns
 from .linear import stack_rows
 from .registry import register_feed_forward
 
@@ -26,8 +31,10 @@ class RoutedExperts(FeedForward):
 
     """params: hidden_size, experts, top, ff_dim, activation ("gelu": the exact form), route_scale, groups (default 1),
     keep_groups (default groups), correction (default True), shared_ff (default 0: no shared expert), shared_gate
-    (default True). weights: router [experts, H], correction [experts], up_<e> [ff, H] and down_<e> [H, ff] for every
-    expert e, shared_up [shared_ff, H], shared_down [H, shared_ff], shared_gate [1, H]."""
+    (default True), scores ("sigmoid", the default, or "softmax"), gated (default False), out_dtype32 (default False; gated
+    experts only). weights: router [experts, H], correction [experts] (the router's bias under "softmax"), up_<e> [ff, H] and
+    down_<e> [H, ff] for every expert e, shared_up [shared_ff, H], shared_down [H, shared_ff], shared_gate [1, H]; and, if
+    gated, gate_<e> [ff, H], shared_gate_proj [shared_ff, H]."""
 
     @classmethod
     def weight_specs(cls, params):
@@ -36,10 +43,14 @@ class RoutedExperts(FeedForward):
         if params.get("correction", True):
             specs["correction"] = TensorSpec((E,), "bias")
         for e in range(E):
+            if params.get("gated"):
+                specs[f"gate_{e}"] = TensorSpec((ff, H), "linear")
             specs[f"up_{e}"] = TensorSpec((ff, H), "linear")
             specs[f"down_{e}"] = TensorSpec((H, ff), "linear")
         sff = params.get("shared_ff", 0)
         if sff:
+            if params.get("gated"):
+                specs["shared_gate_proj"] = TensorSpec((sff, H), "linear")
             specs["shared_up"] = TensorSpec((sff, H), "linear")
             specs["shared_down"] = TensorSpec((H, sff), "linear")
             if params.get("shared_gate", True):
@@ -61,16 +72,35 @@ class RoutedExperts(FeedForward):
             raise ConfigError(f"routed_experts: {self.E} experts in {self.groups} groups of which {self.keep} are kept")
         if self.keep * (self.E // self.groups) < self.top:
             raise ConfigError(f"routed_experts: {self.keep} groups of {self.E // self.groups} experts cannot give {self.top} choices")
-        self.up = stack_rows(*[weights[f"up_{e}"] for e in range(self.E)])
-        self.down = stack_rows(*[weights[f"down_{e}"] for e in range(self.E)])
+        self.gated, self.out32 = bool(params.get("gated")), bool(params.get("out_dtype32", False))
+        scores = params.get("scores", "sigmoid")
+        if scores not in ("sigmoid", "softmax"):
+            raise ConfigError(f"routed_experts: scores {scores!r}; known: 'sigmoid', 'softmax'")
+        self.softmax = scores == "softmax"
+        if self.softmax and self.groups != 1:
+            raise ConfigError("routed_experts: groups of experts under softmax scores are not built")
+        if self.out32 and not self.gated:
+            raise ConfigError("routed_experts: a 32-bit result is built for gated experts")
+        if self.gated:
+            self.up = stack_rows(*[blocked_gate_up(weights[f"gate_{e}"], weights[f"up_{e}"]) for e in range(self.E)])
+            self.down = stack_rows(*[widened_columns(weights[f"down_{e}"]) for e in range(self.E)])
+            self.ff = int(self.down.shape[1])
+        else:
+            self.up = stack_rows(*[weights[f"up_{e}"] for e in range(self.E)])
+            self.down = stack_rows(*[weights[f"down_{e}"] for e in range(self.E)])
         dev = self.up.device
         self.shared_ff = int(params.get("shared_ff", 0))
         self.has_gate = bool(self.shared_ff and params.get("shared_gate", True))
         self.router = stack_rows(weights["router"], weights["shared_gate"]) if self.has_gate else weights["router"].contiguous()
         self.correction = (weights["correction"].contiguous() if params.get("correction", True)
                            else torch.zeros(self.E, dtype=torch.float32, device=dev))
-        self.shared_up = weights["shared_up"].contiguous() if self.shared_ff else None
-        self.shared_down = weights["shared_down"].contiguous() if self.shared_ff else None
+        if self.gated and self.shared_ff:
+            self.shared_up = blocked_gate_up(weights["shared_gate_proj"], weights["shared_up"])
+            self.shared_down = widened_columns(weights["shared_down"])
+            self.shared_ff = int(self.shared_down.shape[1])
+        else:
+            self.shared_up = weights["shared_up"].contiguous() if self.shared_ff else None
+            self.shared_down = weights["shared_down"].contiguous() if self.shared_ff else None
         self._record = None
 
     def record(self):
@@ -86,6 +116,7 @@ class RoutedExperts(FeedForward):
             if self.shared_ff:
                 p.shared_up, p.shared_down = R.linear(self.shared_up), R.linear(self.shared_down)
             p.shared_ff, p.shared_gate = self.shared_ff, int(self.has_gate)
+            p.gated, p.softmax, p.out32 = int(self.gated), int(self.softmax), int(self.out32)
             self._record = R.Record(R.ROUTED_MLP, p, part=self)
         return self._record
 
@@ -93,6 +124,8 @@ class RoutedExperts(FeedForward):
         rec = self.record()
         if rec is None:
             raise ConfigError("routed_experts: matrices kept in another element type than the activations")
+        if self.out32:                      # the executor's registers hold results in the activations' type
+            return super().emit(emitter)
         emitter.records.append(rec)
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
@@ -100,7 +133,8 @@ class RoutedExperts(FeedForward):
         rec = self.record()
         if rec is None:
             raise ConfigError("routed_experts: matrices kept in another element type than the activations")
-        return part_program(self.dtype, x.device, self.H).run_part(rec, x, ctx)
+        out = torch.empty((x.shape[0], self.H), dtype=torch.float32, device=x.device) if self.out32 else None
+        return part_program(self.dtype, x.device, self.H).run_part(rec, x, ctx, out=out)
 
 
 register_feed_forward("routed_experts", RoutedExperts)

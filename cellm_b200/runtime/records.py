@@ -88,13 +88,14 @@ class LatentAttentionParams(Structure):
 
 class GatedMlpParams(Structure):
     _fields_ = [("gate_up", ExecLinear), ("down", ExecLinear), ("bg", PTR), ("bu", PTR), ("bd", PTR), ("b_dtype", I64),
-                ("ff", I64), ("act", I64), ("extra", I64)]
+                ("ff", I64), ("act", I64), ("extra", I64), ("fused", I64), ("out32", I64), ("limit", F64), ("slope", F64)]
 
 
 class RoutedMlpParams(Structure):
     _fields_ = [("up", ExecLinear), ("down", ExecLinear), ("router", ExecLinear), ("correction", PTR), ("c_dtype", I64),
                 ("experts", I64), ("top", I64), ("n_groups", I64), ("keep", I64), ("scale", F64), ("ff", I64), ("act", I64),
-                ("shared_up", ExecLinear), ("shared_down", ExecLinear), ("shared_ff", I64), ("shared_gate", I64)]
+                ("shared_up", ExecLinear), ("shared_down", ExecLinear), ("shared_ff", I64), ("shared_gate", I64),
+                ("gated", I64), ("softmax", I64), ("out32", I64)]
 
 
 class ExecOps(Structure):
@@ -123,7 +124,10 @@ ENTRY_POINTS = [("kernels_common", "cellm_embed"), ("kernels_common", "cellm_add
                 ("kernels_common", "cellm_experts_rowwise"), ("kernels_common", "cellm_activation"),
                 ("kernels_common", "cellm_add2_rmsnorm"), ("kernels_common", "cellm_moe_sort"), ("kernels_common", "cellm_moe_gather"),
                 ("kernels_common", "cellm_moe_combine"), ("gemm_tcgen05", "cellm_gemm_grouped_tcgen05"),
-                ("kernels_common", "cellm_attention_plain_masked")]
+                ("kernels_common", "cellm_attention_plain_masked"), ("kernels_common", "cellm_route_softmax"),
+                ("kernels_common", "cellm_experts_gated_rowwise"), ("kernels_common", "cellm_moe_combine32"),
+                ("gemm_tcgen05", "cellm_gemm_gated_tcgen05"), ("gemm_tcgen05", "cellm_gemm_grouped_gated_tcgen05"),
+                ("kernels_common", "cellm_clamped_gate_act")]
 # libraries a model whose activations are 32-bit never calls into (they need not be compiled for it)
 BF16_ONLY_LIBRARIES = ("attention_decode", "attention_tc", "attention_flash", "gemm_tcgen05", "attention_latent")
 # libraries that only records of these kinds reach (a program without such a record need not have them compiled)
