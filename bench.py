@@ -275,7 +275,7 @@ def step_matrices(model, tokens: int):
 def design_shapes(design: str) -> dict:
     from cellm_b200.config import presets
     return {"vezalorn": presets.VEZALORN_SHAPES, "tufadra": presets.TUFADRA_SHAPES, "padadra": presets.PADADRA_SHAPES,
-            "bozovik": presets.BOZOVIK_SHAPES}[design]
+            "bozovik": presets.BOZOVIK_SHAPES, "tikizen": presets.TIKIZEN_SHAPES}[design]
 
 
 def compare_designs(args, rng) -> int:
@@ -292,8 +292,9 @@ def compare_designs(args, rng) -> int:
     for size in [s for s in args.sizes.split(",") if s]:
         shape, like = design_shapes(args.design)[size]
         row = {}
-        beside = (like, LFM2_SHAPES[like]) if isinstance(like, str) else like
-        for name, config in ((args.design, shape), beside):
+        beside = [(like, LFM2_SHAPES[like])] if isinstance(like, str) else (like if isinstance(like, list) else [like])
+        names = [b[0] for b in beside]
+        for name, config in [(args.design, shape)] + beside[:args.beside]:
             with tempfile.TemporaryDirectory(prefix="cellm_bench_") as d:
                 write_random_model(d, config, seed=0, dtype="bfloat16", init=InitSpec(norm_jitter=0.0))
                 loaded = load_model(d, "bfloat16", "cuda:0")
@@ -318,7 +319,7 @@ def compare_designs(args, rng) -> int:
             del loaded
             torch.cuda.empty_cache()
         out[size] = row
-    print(json.dumps({"metric": "prefill and decode of %s beside %s at equal sizes" % (args.design, "LFM2" if isinstance(like, str) else like[0]), "dtype": "bf16",
+    print(json.dumps({"metric": "prefill and decode of %s beside %s at equal sizes" % (args.design, "LFM2" if isinstance(like, str) else " and ".join(names[:args.beside])), "dtype": "bf16",
                       "data": "synthetic: random token ids, random-init weights", "peaks": pk_src, "steps": args.steps,
                       "warmup": args.warmup, "prompt_len": PROMPT_LEN, "sizes": out}))
     return 0
@@ -332,10 +333,11 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--no-points", action="store_true", help="skip the batch-1 and batch-64 runs")
-    ap.add_argument("--design", default=None, choices=["vezalorn", "tufadra", "padadra", "bozovik"],
+    ap.add_argument("--design", default=None, choices=["vezalorn", "tufadra", "padadra", "bozovik", "tikizen"],
                     help="instead of the default workload: prefill and decode throughput of this design at a few sizes, "
                          "beside LFM2 at equal width, depth and feed-forward (random weights); prints one JSON line")
     ap.add_argument("--sizes", default="700m,1.2b", help="with --design: which of the shapes to run")
+    ap.add_argument("--beside", type=int, default=8, help="with --design: how many of the models beside it to run (0: the design alone)")
     ap.add_argument("--profile-region", choices=["decode", "prefill"], default=None,
                     help="for a profiler started with --profile-from-start off: run the set-up, then one eager "
                          "decode step (or one prefill) between cudaProfilerStart/Stop, print no bench line")

@@ -130,3 +130,38 @@ BOZOVIK_SHAPES = {
     "1.2b": (_bozovik(2048, 16, [2, 5, 8, 10, 12, 14], [0, 7, 15], 32, 8, 32, 16, 8192), ("padadra", PADADRA_SHAPES["1.2b"][0])),
     "700m": (_bozovik(1536, 16, [2, 5, 8, 10, 12, 14], [0, 7, 15], 24, 8, 24, 12, 6912), ("padadra", PADADRA_SHAPES["700m"][0])),
 }
+
+
+# ---- Tikizen shapes beside Padadra's and Tufadra's -----------------------------------------------------------------
+def _tikizen(width: int, layers: int, attention_at, retention_at, moe_at, heads: int, kv_heads: int, ret_heads: int, ssd_heads: int, ff: int,
+             expert_ff: int, shared_ff: int, vocab: int = 65536) -> dict:
+    """Layers of a width and count that a Padadra shape has: attention inside chunks of 1,024 positions (heads of 64) where
+    Padadra has its two mixers side by side, every second of these reading the keys of the one before; retention (heads of
+    128 x 128) at a few places and Mamba-2 (states of 128 x 64 a head, one group of B and C, inner width twice the model's)
+    at the others. Feed-forwards of Padadra's width, and at a few places Tufadra's mixture (64 experts of which 6 are
+    chosen, a shared one), gated."""
+    rot = {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 64, "scale": 0.125, "mask": {"size": 1024}, "rot": rot}
+    ret = {"heads": ret_heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5.0 - 3.0 * h / max(ret_heads - 1, 1)) for h in range(ret_heads)],
+           "rot": {"base": 10000.0, "dims": 128}}
+    ssd = {"heads": ssd_heads, "vdim": 64, "state": 128, "groups": 1, "norm_groups": 1, "conv": 4}
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": 64, "top": 6}, "shared": {"ff": shared_ff}}
+
+    def layer(i):
+        mlp = dict(moe) if i in moe_at else dict(dense)
+        if i in attention_at:
+            n = attention_at.index(i)
+            return {"type": "attention", "mixer": dict(att, **({"kv_from": attention_at[n - 1]} if n % 2 else {})), "mlp": mlp}
+        return {"type": "retention", "mixer": dict(ret), "mlp": mlp} if i in retention_at else {"type": "mamba2", "mixer": dict(ssd), "mlp": mlp}
+    return {"architecture": "Tikizen", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "postln_alpha": 2.0,
+            "layers": [layer(i) for i in range(layers)]}
+
+
+# name -> (Tikizen shape, [(a close design's name, its shape of equal width and depth), ...])
+TIKIZEN_SHAPES = {
+    "1.2b": (_tikizen(2048, 16, [2, 5, 8, 10, 12, 14], [3, 7, 11, 15], [1, 5, 9, 13], 32, 8, 16, 64, 8192, 1024, 2048),
+             [("padadra", PADADRA_SHAPES["1.2b"][0]), ("tufadra", TUFADRA_SHAPES["1.2b"][0])]),
+    "700m": (_tikizen(1536, 16, [2, 5, 8, 10, 12, 14], [3, 7, 11, 15], [1, 5, 9, 13], 24, 8, 12, 48, 6912, 896, 1536),
+             [("padadra", PADADRA_SHAPES["700m"][0]), ("tufadra", TUFADRA_SHAPES["700m"][0])]),
+}

@@ -71,6 +71,7 @@ struct WalkVectors {
     const float* num[2];
     long long num_ld[2];
     int vec16;          // every start is a multiple of 16 bytes: copies of four values
+    int max_len = 1 << 30;      // longer portions are left alone (another kernel takes them)
 };
 
 // MODE 0: HGRN2; 1: the gated delta rule; 2: the generalized delta rule (five vectors a token: chunks of four tokens for
@@ -95,7 +96,7 @@ state_walk_kernel(float* __restrict__ o_out, float* __restrict__ state, long lon
     const int slot = slot_ids[b];
     if (slot < 0 || slot >= n_slots) { if (tid == 0) atomicOr(err, CELLM_DEV_BAD_SLOT); return; }
     const int start = cu_seqlens[b], end = cu_seqlens[b + 1];
-    if (end <= start) return;
+    if (end <= start || end - start > vec.max_len) return;
     float* st = state + (size_t)slot * slot_stride + (size_t)h * dim * vd;
     const bool live = j < vd;
     if (dim < DIM) {            // the rows beyond the head's own stay zero in every stage
@@ -717,6 +718,7 @@ decay_scan_kernel(float* __restrict__ o_out, float* __restrict__ state, long lon
     const int slot = slot_ids[b];
     if (slot < 0 || slot >= n_slots) { if (lane == 0) atomicOr(err, CELLM_DEV_BAD_SLOT); return; }
     const int start = cu_seqlens[b], end = cu_seqlens[b + 1];
+    if (end - start > vec.max_len) return;
     float* st = state + (size_t)slot * slot_stride + (size_t)h * dim * vd;
     const bool live = j < vd;
     for (int i = 0; i < dim; ++i) S(i) = live ? st[(size_t)i * vd + j] : 0.f;
@@ -742,11 +744,12 @@ decay_scan_kernel(float* __restrict__ o_out, float* __restrict__ state, long lon
 
 // q, k: rows of `dim` values per head group, [T, ld_q] and [T, ld_k] 32-bit; head h reads group h / (heads / groups).
 // v [T, ld_v]: heads x vd. decay [T (or one row), heads] at pitch ld_d (0: one row of constants), write likewise (null:
-// 1). state [slots][heads][dim][vd] is moved on; o_out [T, heads * vd] gets S^T q.
+// 1). state [slots][heads][dim][vd] is moved on; o_out [T, heads * vd] gets S^T q. Portions of more than max_len tokens (0: no
+// such limit) are left alone.
 CELLM_API int cellm_decay_scan(float* o_out, float* state, long long slot_stride, int n_slots, const float* q, long long ld_q,
                                const float* k, long long ld_k, const float* v, long long ld_v, const float* decay, long long ld_d,
                                const float* write, long long ld_w, const int* cu_seqlens, const int* slot_ids, int B, int heads,
-                               int groups, int dim, int vd, int* err, cudaStream_t stream) {
+                               int groups, int dim, int vd, int max_len, int* err, cudaStream_t stream) {
     if (B <= 0) return CELLM_OK;
     if (heads <= 0 || groups <= 0 || heads % groups || dim <= 0 || vd <= 0 || dim > RECURRENT_MAX_DIM) return CELLM_ERR_SIZE;
     if (!decay) return CELLM_ERR_ARG;
@@ -755,6 +758,7 @@ CELLM_API int cellm_decay_scan(float* o_out, float* state, long long slot_stride
     vec.p[0] = q, vec.p[1] = k, vec.ld[0] = ld_q, vec.ld[1] = ld_k;
     vec.num[0] = decay, vec.num[1] = write, vec.num_ld[0] = ld_d, vec.num_ld[1] = ld_w;
     vec.vec16 = dim % 4 == 0 && ld_q % 4 == 0 && ld_k % 4 == 0 && aligned16(q) && aligned16(k);
+    if (max_len > 0) vec.max_len = max_len;
 #define DECAY_WALK(D, R)                                                                                           \
     CELLM_RUN((state_walk_kernel<D, R, 3>), dim3(B, heads, (vd + WalkShape<D, R>::CPB - 1) / WalkShape<D, R>::CPB), WALK_THREADS, 0, stream, \
               o_out, state, slot_stride, n_slots, vec, v, ld_v, (const float*)nullptr, cu_seqlens, slot_ids, heads, dim, vd, err)
@@ -816,12 +820,12 @@ CELLM_API int cellm_rotate_heads(float* x, long long ld, int col0, int n_heads, 
 
 // Mamba-2's inputs. Channels col0 .. col0 + C of proj (x | B | C side by side) pass a causal convolution over time with a
 // bias and silu into xbc [T, C]; the step sizes dt = softplus(proj[col_dt + h] + dt_bias_h) go to step [T, heads] and the
-// decays exp(-exp(A_log_h) dt) to decay [T, heads]. A thread a channel walks `run` tokens with the taps' inputs in
+// logarithms of the decays, -exp(A_log_h) dt, to logd and the decays to decay [T, heads]. A thread a channel walks `run` tokens with the taps' inputs in
 // registers (TAPS > 0), or reads them anew for every token (TAPS 0: any number of taps). The last row of blocks forms the
 // step sizes.
 template <int TAPS>
 __global__ void __launch_bounds__(256)
-ssd_prep_kernel(float* __restrict__ xbc, float* __restrict__ step, float* __restrict__ decay, ConvTaps cv, const float* __restrict__ conv_bias,
+ssd_prep_kernel(float* __restrict__ xbc, float* __restrict__ step, float* __restrict__ logd, float* __restrict__ decay, ConvTaps cv, const float* __restrict__ conv_bias,
                 const float* __restrict__ state_base, long long slot_stride, int n_slots, int col_dt, const float* __restrict__ dt_bias,
                 const float* __restrict__ A_log, const int* __restrict__ seq_of_token, const int* __restrict__ cu_seqlens,
                 const int* __restrict__ slot_ids, int T, int heads, int run, int* __restrict__ err) {
@@ -833,7 +837,9 @@ ssd_prep_kernel(float* __restrict__ xbc, float* __restrict__ step, float* __rest
             const int t = t0 + i / heads, h = i % heads;
             const float dt = cellm_softplus(cv.proj[(size_t)t * cv.ld + col_dt + h] + dt_bias[h]);
             step[(size_t)t * heads + h] = dt;
-            decay[(size_t)t * heads + h] = expf(-expf(A_log[h]) * dt);
+            const float l = fmaxf(-expf(A_log[h]) * dt, -1e4f);        // a decay of zero stays one, and sums of logarithms finite
+            logd[(size_t)t * heads + h] = l;
+            decay[(size_t)t * heads + h] = expf(l);
         }
         return;
     }
@@ -881,7 +887,7 @@ ssd_prep_kernel(float* __restrict__ xbc, float* __restrict__ step, float* __rest
     }
 }
 
-CELLM_API int cellm_ssd_prep(float* xbc, float* step, float* decay, const float* proj, long long ld, int col0, int C, int col_dt,
+CELLM_API int cellm_ssd_prep(float* xbc, float* step, float* logd, float* decay, const float* proj, long long ld, int col0, int C, int col_dt,
                              const float* taps, int n_taps, const float* conv_bias, const float* state, long long slot_stride,
                              int n_slots, const float* dt_bias, const float* A_log, const int* seq_of_token, const int* cu_seqlens,
                              const int* slot_ids, int T, int heads, int* err, cudaStream_t stream) {
@@ -892,7 +898,7 @@ CELLM_API int cellm_ssd_prep(float* xbc, float* step, float* decay, const float*
     cv.proj = proj; cv.ld = ld; cv.col0 = col0; cv.bias = nullptr; cv.taps = taps; cv.state = nullptr; cv.n_taps = n_taps; cv.C = C;
     const int run = T >= 512 ? 8 : 1;
     const dim3 grid((unsigned)((T + run - 1) / run), (unsigned)((C + 255) / 256 + 1));
-#define SSD_PREP(N) CELLM_RUN(ssd_prep_kernel<N>, grid, 256, 0, stream, xbc, step, decay, cv, conv_bias, state, slot_stride, n_slots, col_dt, \
+#define SSD_PREP(N) CELLM_RUN(ssd_prep_kernel<N>, grid, 256, 0, stream, xbc, step, logd, decay, cv, conv_bias, state, slot_stride, n_slots, col_dt, \
                               dt_bias, A_log, seq_of_token, cu_seqlens, slot_ids, T, heads, run, err)
     if (n_taps == 4) SSD_PREP(4);
     else if (n_taps == 3) SSD_PREP(3);

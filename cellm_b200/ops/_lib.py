@@ -76,9 +76,9 @@ _SIGNATURES = {
         "cellm_post_norm": [P, P, P, I, F, P, I, I, F, I, P],
         "cellm_turned_attn_prep": [P, P, P, P, L, P, I, I, F, I, F, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, P],
         "cellm_attention_plain_chunked": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P],
-        "cellm_decay_scan": [P, P, L, I, P, L, P, L, P, L, P, L, P, L, P, P, I, I, I, I, I, P, P],
+        "cellm_decay_scan": [P, P, L, I, P, L, P, L, P, L, P, L, P, L, P, P, I, I, I, I, I, I, P, P],
         "cellm_rotate_heads": [P, L, I, I, I, I, I, P, F, P, I, P],
-        "cellm_ssd_prep": [P, P, P, P, L, I, I, I, P, I, P, P, L, I, P, P, P, P, P, I, I, P, P],
+        "cellm_ssd_prep": [P, P, P, P, P, L, I, I, I, P, I, P, P, L, I, P, P, P, P, P, I, I, P, P],
         "cellm_gated_group_norm": [P, P, P, L, P, P, L, P, I, I, I, I, F, I, P],
         "cellm_head_norm_silu": [P, P, P, L, I, I, I, F, I, P],
     },
@@ -100,6 +100,10 @@ _SIGNATURES = {
         "cellm_attention_flash_sink": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, I, P, P, I, P, P, P],
         "cellm_attention_flash_chunked": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, I, P, P],
         "cellm_attention_flash_masked": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, I, I, P, P, L, P, P],
+    },
+    "decay_chunks": {
+        "cellm_decay_chunks": [P, P, L, I, P, L, P, L, P, L, P, L, P, L, P, P, I, I, I, I, I, I, I, P, P, P, P],
+        "cellm_decay_chunks_supports": [I, I],
     },
     "attention_latent": {
         "cellm_attention_latent": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P, P, P],

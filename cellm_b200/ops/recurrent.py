@@ -371,35 +371,54 @@ def rotate_heads(x: torch.Tensor, col0: int, n_heads: int, hd: int, freq: torch.
                                          ptr(positions), x.shape[0], stream_of(x)), "rotate_heads")
 
 
+# Portions of this many tokens and more run the scalar-decay recurrence in chunks (measured; see decay_scan).
+CHUNKED_FROM = 64
+
+
 def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, write: Optional[torch.Tensor], state: torch.Tensor, ctx,
-               heads: int, groups: int, dim: int, vd: int) -> torch.Tensor:
+               heads: int, groups: int, dim: int, vd: int, logd: Optional[torch.Tensor] = None) -> torch.Tensor:
     """S <- decay S + write k v^T, o = S^T q over every request's tokens of the step, one decay and one writing factor per
     head; state [slots, heads, dim, vd] float32 is moved on. q, k [T, groups * dim] (head h reads group h / (heads / groups))
     and v [T, heads * vd] float32, rows may be strided; decay and write [T, heads], or [heads] where they are constants
-    (write None: 1). Returns float32 [T, heads * vd]."""
-    _f32(q, k, v, decay, write, state)
+    (write None: 1). Returns float32 [T, heads * vd]. `logd` (the decays' logarithms, of decay's shape): portions of
+    CHUNKED_FROM tokens and more run in chunks on the tensor cores where the sizes allow, the others token by token; without
+    it all run token by token, and a state is then bit-identical however the sequence was cut."""
+    _f32(q, k, v, decay, write, state, logd)
     pitch = lambda t: 0 if t is None or t.dim() == 1 else t.stride(0)
     o = torch.empty((ctx.T, heads * vd), dtype=torch.float32, device=q.device)
+    long = [n for n in ctx.q_lens if n >= CHUNKED_FROM] if logd is not None and ctx.max_q_len >= CHUNKED_FROM and max(dim, vd) <= 128 else []
+    if long:
+        n_chunks = sum(-(-n // 64) for n in long)
+        ws = torch.empty((n_chunks * heads * (dim * vd + 1),), dtype=torch.float32, device=q.device)
+        tot = ws[n_chunks * heads * dim * vd:]
+        check(fn("decay_chunks", "cellm_decay_chunks")(ptr(o), ptr(state), state.stride(0), state.shape[0], ptr(q), q.stride(0), ptr(k), k.stride(0), ptr(v),
+                                                       v.stride(0), ptr(logd), pitch(logd), ptr(write), pitch(write), ptr(ctx.cu_seqlens),
+                                                       ptr(ctx.slot_ids), ctx.B, n_chunks, CHUNKED_FROM, heads, groups, dim, vd, ptr(ws), ptr(tot),
+                                                       ptr(ctx.err), stream_of(q)), "decay_chunks")
+        count_launch(2)
+        if len(long) == ctx.B:
+            return o
     check(fn(_LIB, "cellm_decay_scan")(ptr(o), ptr(state), state.stride(0), state.shape[0], ptr(q), q.stride(0), ptr(k), k.stride(0), ptr(v),
                                        v.stride(0), ptr(decay), pitch(decay), ptr(write), pitch(write), ptr(ctx.cu_seqlens), ptr(ctx.slot_ids),
-                                       ctx.B, heads, groups, dim, vd, ptr(ctx.err), stream_of(q)), "decay_scan")
+                                       ctx.B, heads, groups, dim, vd, CHUNKED_FROM - 1 if long else 0, ptr(ctx.err), stream_of(q)), "decay_scan")
     return o
 
 
 def ssd_prep(proj: torch.Tensor, col0: int, C: int, col_dt: int, taps: torch.Tensor, conv_bias: torch.Tensor, conv_state, dt_bias: torch.Tensor,
              A_log: torch.Tensor, ctx, heads: int):
     """Mamba-2's inputs: (silu(conv(columns col0 .. col0 + C of proj) + conv_bias) [T, C], step sizes softplus(proj + dt_bias)
-    [T, heads], decays exp(-exp(A_log) step) [T, heads]), all float32. taps [C, n]; conv_state [slots, n - 1, C] or None."""
+    [T, heads], the decays' logarithms -exp(A_log) step and the decays [T, heads]), all float32. taps [C, n]; conv_state [slots, n - 1, C] or None."""
     _f32(proj, taps, conv_bias, conv_state, dt_bias, A_log)
     T, dev = ctx.T, proj.device
     xbc = torch.empty((T, C), dtype=torch.float32, device=dev)
     step = torch.empty((T, heads), dtype=torch.float32, device=dev)
+    logd = torch.empty((T, heads), dtype=torch.float32, device=dev)
     decay = torch.empty((T, heads), dtype=torch.float32, device=dev)
-    check(fn(_LIB, "cellm_ssd_prep")(ptr(xbc), ptr(step), ptr(decay), ptr(proj), proj.stride(0), int(col0), int(C), int(col_dt), ptr(taps),
+    check(fn(_LIB, "cellm_ssd_prep")(ptr(xbc), ptr(step), ptr(logd), ptr(decay), ptr(proj), proj.stride(0), int(col0), int(C), int(col_dt), ptr(taps),
                                      taps.shape[1], ptr(conv_bias), ptr(conv_state), conv_state.stride(0) if conv_state is not None else 0,
                                      conv_state.shape[0] if conv_state is not None else 1 << 30, ptr(dt_bias), ptr(A_log), ptr(ctx.seq_of_token),
                                      ptr(ctx.cu_seqlens), ptr(ctx.slot_ids), T, heads, ptr(ctx.err), stream_of(proj)), "ssd_prep")
-    return xbc, step, decay
+    return xbc, step, logd, decay
 
 
 def gated_group_norm(o: torch.Tensor, x: Optional[torch.Tensor], D: Optional[torch.Tensor], z: torch.Tensor, w: torch.Tensor, vd: int, groups: int,

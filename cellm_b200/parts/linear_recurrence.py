@@ -41,7 +41,9 @@
 
 Everything that enters a recurrence is 32-bit (the projections keep their 32-bit sums; gates, decays, unit vectors and
 the state are computed in 32-bit), and a request's tokens are walked in order from the state the step before left, so
-the state after a token does not depend on how the sequence was cut. The gated delta rule and Mamba-2 also keep the
+the state after a token does not depend on how the sequence was cut. Under bfloat16 the two recurrences with one decay a
+head run long portions of a prompt in chunks of 64 tokens on the tensor cores (decay_chunks.cu; the state stays 32-bit,
+operands enter as two bfloat16 numbers each), which differs from the walk in rounding only. The gated delta rule and Mamba-2 also keep the
 convolution's last taps - 1 projected rows in the slot."""
 from __future__ import annotations
 
@@ -251,6 +253,9 @@ class RetentionMixer(Mixer):
         self.out_proj = Linear(weights["o"], dtype)
         self.out32 = bool(params.get("out_dtype32", False))
         self.decay = torch.tensor(decay, dtype=torch.float32, device=dev)
+        if any(x < 0 for x in decay):
+            raise ConfigError("retention: a negative decay")
+        self.logd = torch.log(torch.tensor(decay, dtype=torch.float64).clamp_min(1e-300)).to(torch.float32).to(dev) if dtype == torch.bfloat16 else None
         # k's factor dim^(-1/2), as the factor with which a head writes
         self.write = torch.full((self.heads,), self.dim ** -0.5, dtype=torch.float32, device=dev)
         pos = params.get("position")
@@ -269,7 +274,8 @@ class RetentionMixer(Mixer):
         proj = self.in_proj(x, out_dtype=torch.float32)
         if self.rot:
             ops.rotate_heads(proj, 0, 2 * self.heads, self.dim, self.freq, self.rot, self.interleaved, self.amp, ctx.positions)
-        o = ops.decay_scan(proj, proj[:, hd:], proj[:, 2 * hd:], self.decay, self.write, state, ctx, self.heads, self.heads, self.dim, self.vd)
+        o = ops.decay_scan(proj, proj[:, hd:], proj[:, 2 * hd:], self.decay, self.write, state, ctx, self.heads, self.heads, self.dim, self.vd,
+                           self.logd)
         y = ops.head_norm_silu(o, proj[:, 2 * hd + hv:], self.heads, self.vd, self.eps, self.dtype)
         return self.out_proj(y, out_dtype=torch.float32 if self.out32 else None)
 
@@ -324,11 +330,12 @@ class Mamba2Mixer(Mixer):
         conv_state, state = (b[0].state if self.taps > 1 else None), b[-1].state
         inner, gn = self.inner, self.groups * self.n
         proj = self.in_proj(x, out_dtype=torch.float32)
-        xbc, step, decay = ops.ssd_prep(proj, inner, self.C, inner + self.C, self.conv_w, self.conv_b, conv_state, self.dt_bias, self.A_log, ctx,
+        xbc, step, logd, decay = ops.ssd_prep(proj, inner, self.C, inner + self.C, self.conv_w, self.conv_b, conv_state, self.dt_bias, self.A_log, ctx,
                                         self.heads)
         if conv_state is not None:
             ops.conv_state_update(conv_state, proj, inner, None, self.taps, ctx)
-        o = ops.decay_scan(xbc[:, inner + gn:], xbc[:, inner:], xbc, decay, step, state, ctx, self.heads, self.groups, self.n, self.vd)
+        o = ops.decay_scan(xbc[:, inner + gn:], xbc[:, inner:], xbc, decay, step, state, ctx, self.heads, self.groups, self.n, self.vd,
+                           logd if self.dtype == torch.bfloat16 else None)
         y = ops.gated_group_norm(o, xbc, self.D, proj, self.norm_w, self.vd, self.norm_groups, self.eps, self.dtype)
         return self.out_proj(y, out_dtype=torch.float32 if self.out32 else None)
 

@@ -471,7 +471,7 @@ def test_decay_walk_alone(heads, groups, dim, vd, constants):
     still weigh at the end, another's so small that only the last token does."""
     from cellm_b200 import ops
     g = torch.Generator().manual_seed(heads * 100 + dim + constants)
-    lens, slots, n = [141, 19], [3, 1], groups * dim
+    lens, slots, n = [201, 19], [3, 1], groups * dim
     ld = 2 * n + heads * vd + 4                                            # q | k | v and something behind them
     proj = [torch.randn(L, ld, generator=g) for L in lens]
     if constants:
@@ -504,6 +504,20 @@ def test_decay_walk_alone(heads, groups, dim, vd, constants):
             torch.testing.assert_close(outs[name][b].double(), want[b], rtol=3e-5, atol=3e-5 * float(want[b].abs().max()))
     for b in range(len(lens)):
         assert torch.equal(outs["whole"][b], outs["portions"][b]) and torch.equal(outs["whole"][b], outs["single"][b])
+    # long portions in chunks on the tensor cores, the others token by token, and both kinds side by side
+    log = lambda d: torch.log(d.clamp_min(1e-30))
+    for sizes in ((512,), (64, 65, 12), (70, 1), (63, 100)):
+        state = torch.full((4, heads, dim, vd), 7.0, device=DEV)
+        state[slots] = 0
+
+        def run_chunks(rows, ctx):
+            p = rows(proj)
+            d, wr = (d0.to(DEV), w0.to(DEV)) if constants else (rows(decay), rows(write))
+            return ops.decay_scan(p, p[:, n:], p[:, 2 * n:], d, wr, state, ctx, heads, groups, dim, vd, log(d).contiguous())
+        got = walk_in_cuts(lens, slots, sizes, run_chunks)
+        assert float(state[0].min()) == 7.0 and float(state[2].max()) == 7.0
+        for b in range(len(lens)):
+            torch.testing.assert_close(got[b].double(), want[b], rtol=1e-4, atol=1e-4 * float(want[b].abs().max()))
     # no writing factor: one
     state = torch.zeros((1, heads, dim, vd), device=DEV)
     p = proj[1].to(DEV)
