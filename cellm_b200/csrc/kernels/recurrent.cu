@@ -823,6 +823,7 @@ CELLM_API int cellm_rotate_heads(float* x, long long ld, int col0, int n_heads, 
 // logarithms of the decays, -exp(A_log_h) dt, to logd and the decays to decay [T, heads]. A thread a channel walks `run` tokens with the taps' inputs in
 // registers (TAPS > 0), or reads them anew for every token (TAPS 0: any number of taps). The last row of blocks forms the
 // step sizes.
+#define SSD_RUN 8
 template <int TAPS>
 __global__ void __launch_bounds__(256)
 ssd_prep_kernel(float* __restrict__ xbc, float* __restrict__ step, float* __restrict__ logd, float* __restrict__ decay, ConvTaps cv, const float* __restrict__ conv_bias,
@@ -853,6 +854,26 @@ ssd_prep_kernel(float* __restrict__ xbc, float* __restrict__ step, float* __rest
     }
     pdl_wait();
     int end = -1, start = 0;
+    if constexpr (TAPS > 0) {
+        if (t1 - t0 == SSD_RUN) {
+            const int b = seq_of_token[t0];
+            start = cu_seqlens[b];
+            if (t0 - (TAPS - 1) >= start && t1 <= cu_seqlens[b + 1]) {      // the run and its past lie in one portion: all loads at once
+                float x[SSD_RUN + TAPS - 1];
+#pragma unroll
+                for (int j = 0; j < SSD_RUN + TAPS - 1; ++j) x[j] = cv.proj[(size_t)(t0 - (TAPS - 1) + j) * cv.ld + cv.col0 + c];
+#pragma unroll
+                for (int r = 0; r < SSD_RUN; ++r) {
+                    float y = 0.f;
+#pragma unroll
+                    for (int j = 0; j < TAPS; ++j) y = fmaf(w[j], x[r + j], y);
+                    y += bias;
+                    xbc[(size_t)(t0 + r) * cv.C + c] = y * sigmoidf_(y);
+                }
+                return;
+            }
+        }
+    }
     for (int t = t0; t < t1; ++t) {
         bool fresh = t == t0;
         if (t >= end) {         // another request's portion begins
@@ -896,7 +917,7 @@ CELLM_API int cellm_ssd_prep(float* xbc, float* step, float* logd, float* decay,
     if (n_taps > 1 && !state) return CELLM_ERR_ARG;
     ConvTaps cv;
     cv.proj = proj; cv.ld = ld; cv.col0 = col0; cv.bias = nullptr; cv.taps = taps; cv.state = nullptr; cv.n_taps = n_taps; cv.C = C;
-    const int run = T >= 512 ? 8 : 1;
+    const int run = T >= 512 ? SSD_RUN : 1;
     const dim3 grid((unsigned)((T + run - 1) / run), (unsigned)((C + 255) / 256 + 1));
 #define SSD_PREP(N) CELLM_RUN(ssd_prep_kernel<N>, grid, 256, 0, stream, xbc, step, logd, decay, cv, conv_bias, state, slot_stride, n_slots, col_dt, \
                               dt_bias, A_log, seq_of_token, cu_seqlens, slot_ids, T, heads, run, err)
@@ -936,6 +957,52 @@ gated_group_norm_kernel(TA* __restrict__ out, const float* __restrict__ o, const
     for (int i = threadIdx.x; i < Hg; i += blockDim.x) out[t * inner + lo + i] = from_float<TA>(vals[i] * inv * w[lo + i]);
 }
 
+// The same where a part is a multiple of four values and at most 4 * PER * 1024: a thread holds PER pieces of four in registers.
+template <typename TA, int PER>
+__global__ void __launch_bounds__(1024)
+gated_group_norm_vec4_kernel(TA* __restrict__ out, const float* __restrict__ o, const float* __restrict__ x, long long ld_x,
+                             const float* __restrict__ D, const float* __restrict__ z, long long ld_z, const float* __restrict__ w, int inner,
+                             int vd, int Hg, float eps) {
+    __shared__ float scratch[32];
+    pdl_trigger();
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    const int lo = blockIdx.y * Hg;
+    float4 v[PER];
+    float ss = 0.f;
+#pragma unroll
+    for (int p = 0; p < PER; ++p) {
+        const int i = (threadIdx.x + p * blockDim.x) * 4, c = lo + i;
+        v[p] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < Hg) {
+            const float4 g = *reinterpret_cast<const float4*>(z + t * ld_z + c);
+            float4 a = *reinterpret_cast<const float4*>(o + t * inner + c);
+            if (D) {                // four neighbours lie in one head
+                const float4 u = *reinterpret_cast<const float4*>(x + t * ld_x + c);
+                const float d = D[c / vd];
+                a.x = fmaf(d, u.x, a.x), a.y = fmaf(d, u.y, a.y), a.z = fmaf(d, u.z, a.z), a.w = fmaf(d, u.w, a.w);
+            }
+            v[p] = make_float4(a.x * (g.x * sigmoidf_(g.x)), a.y * (g.y * sigmoidf_(g.y)), a.z * (g.z * sigmoidf_(g.z)), a.w * (g.w * sigmoidf_(g.w)));
+        }
+        ss = fmaf(v[p].x, v[p].x, ss), ss = fmaf(v[p].y, v[p].y, ss), ss = fmaf(v[p].z, v[p].z, ss), ss = fmaf(v[p].w, v[p].w, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.f / sqrtf(ss / (float)Hg + eps);
+#pragma unroll
+    for (int p = 0; p < PER; ++p) {
+        const int i = (threadIdx.x + p * blockDim.x) * 4, c = lo + i;
+        if (i < Hg) {
+            const float4 g = *reinterpret_cast<const float4*>(w + c);
+            const float4 y = make_float4(v[p].x * inv * g.x, v[p].y * inv * g.y, v[p].z * inv * g.z, v[p].w * inv * g.w);
+            if constexpr (sizeof(TA) == 4) *reinterpret_cast<float4*>(out + t * inner + c) = y;
+            else {
+                const __nv_bfloat162 a = __floats2bfloat162_rn(y.x, y.y), b = __floats2bfloat162_rn(y.z, y.w);
+                *reinterpret_cast<uint2*>(out + t * inner + c) = make_uint2(*reinterpret_cast<const unsigned*>(&a), *reinterpret_cast<const unsigned*>(&b));
+            }
+        }
+    }
+}
+
 // o [T, inner] 32-bit (heads of vd side by side), x at pitch ld_x and z at pitch ld_z likewise; D [heads] (null: no term in
 // x); w [inner].
 CELLM_API int cellm_gated_group_norm(void* out, const float* o, const float* x, long long ld_x, const float* D, const float* z, long long ld_z,
@@ -946,6 +1013,17 @@ CELLM_API int cellm_gated_group_norm(void* out, const float* o, const float* x, 
     const int Hg = inner / groups;
     const size_t smem = (size_t)Hg * sizeof(float);
     if (smem > 200 * 1024) return CELLM_ERR_SIZE;
+    if (Hg % 4 == 0 && vd % 4 == 0 && inner % 4 == 0 && ld_z % 4 == 0 && (!D || ld_x % 4 == 0) && Hg <= 8192 && aligned16(out) && aligned16(o) &&
+        aligned16(z) && aligned16(w) && (!D || aligned16(x))) {
+        const int pieces = Hg / 4, threads = pieces <= 1024 ? (pieces + 31) / 32 * 32 : 1024;
+        const dim3 grid((unsigned)T, (unsigned)groups);
+#define GGN_VEC(TA, PER) CELLM_RUN((gated_group_norm_vec4_kernel<TA, PER>), grid, threads, 0, stream, (TA*)out, o, x, ld_x, D, z, ld_z, w, inner, vd, Hg, eps)
+        if (dtype == CELLM_F32) { if (pieces <= 1024) GGN_VEC(float, 1); else GGN_VEC(float, 2); }
+        else if (dtype == CELLM_BF16) { if (pieces <= 1024) GGN_VEC(__nv_bfloat16, 1); else GGN_VEC(__nv_bfloat16, 2); }
+        else return CELLM_ERR_DTYPE;
+#undef GGN_VEC
+        return CELLM_OK;
+    }
     const int threads = Hg >= 256 ? 256 : Hg >= 128 ? 128 : 64;
 #define GGN_RUN(TA)                                                                                                          \
     do {                                                                                                                      \

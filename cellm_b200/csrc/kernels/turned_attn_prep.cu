@@ -10,8 +10,9 @@
 // arithmetic is 32-bit; angles are pos * (hi + lo) in split arithmetic from tables made in 64-bit.
 #include "common.cuh"
 
-template <typename TA>
-__global__ void __launch_bounds__(256)
+// M > 0: a lane holds its entries of a head (lane + 32 m, m < M) in registers between the norm's sum and the store.
+template <typename TA, int M>
+__global__ void __launch_bounds__(1024)
 turned_attn_prep_kernel(TA* __restrict__ q_out, TA* __restrict__ k_pool, TA* __restrict__ v_pool, const float* __restrict__ proj, long long ld,
                         const float* __restrict__ freq, int rot, int interleaved, float amp, int norm, float eps,
                         const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
@@ -58,17 +59,34 @@ turned_attn_prep_kernel(TA* __restrict__ q_out, TA* __restrict__ k_pool, TA* __r
             else { first = i < half; p = first ? i : i - half; other = first ? i + half : i - half; }
             return first ? x[i] * cs[p] - x[other] * sn[p] : x[i] * cs[p] + x[other] * sn[p];
         };
-        float inv = 1.f;
-        if (norm) {
-            float ss = 0.f;
-            for (int i = lane; i < hd; i += 32) { const float v = turned(i); ss = fmaf(v, v, ss); }
-            inv = 1.f / sqrtf(warp_sum(ss) / (float)hd + eps);
-        }
-        TA* dst;
+        TA* dst = nullptr;
         if (hh < nh) dst = q_out + ((size_t)t * nh + hh) * width_k;
         else if (page >= 0) dst = k_pool + (((size_t)page * nkv + (hh - nh)) * page_size + in_page) * width_k;
-        else continue;
-        for (int i = lane; i < width_k; i += 32) dst[i] = from_float<TA>(i < hd ? turned(i) * inv : 0.f);
+        if constexpr (M > 0) {
+            float v[M], ss = 0.f;
+#pragma unroll
+            for (int m = 0; m < M; ++m) {
+                const int i = lane + 32 * m;
+                v[m] = i < hd ? turned(i) : 0.f;
+                ss = fmaf(v[m], v[m], ss);
+            }
+            const float inv = norm ? 1.f / sqrtf(warp_sum(ss) / (float)hd + eps) : 1.f;
+            if (!dst) continue;
+#pragma unroll
+            for (int m = 0; m < M; ++m) {
+                const int i = lane + 32 * m;
+                if (i < width_k) dst[i] = from_float<TA>(v[m] * inv);
+            }
+        } else {
+            float inv = 1.f;
+            if (norm) {
+                float ss = 0.f;
+                for (int i = lane; i < hd; i += 32) { const float v = turned(i); ss = fmaf(v, v, ss); }
+                inv = 1.f / sqrtf(warp_sum(ss) / (float)hd + eps);
+            }
+            if (!dst) continue;
+            for (int i = lane; i < width_k; i += 32) dst[i] = from_float<TA>(i < hd ? turned(i) * inv : 0.f);
+        }
     }
 }
 
@@ -83,15 +101,20 @@ CELLM_API int cellm_turned_attn_prep(void* q_out, void* k_pool, void* v_pool, co
     if (nkv > 0 && (nh % nkv || vd <= 0 || width_v < vd || page_size <= 0)) return CELLM_ERR_SIZE;
     if ((rot > 0 && !freq) || (nkv > 0 && (!k_pool || !v_pool || !block_table))) return CELLM_ERR_ARG;
     const size_t smem = (size_t)rot * sizeof(float);
-    const int threads = nh + 2 * nkv >= 8 ? 256 : 128;
-    if (dtype == CELLM_F32)
-        CELLM_RUN(turned_attn_prep_kernel<float>, T, threads, smem, stream, (float*)q_out, (float*)k_pool, (float*)v_pool, proj, ld, freq, rot,
-                  interleaved, amp, norm, eps, positions, seq_of_token, block_table, bt_stride, num_pages, page_size, nh, nkv, hd, vd, width_k,
-                  width_v, err);
-    else if (dtype == CELLM_BF16)
-        CELLM_RUN(turned_attn_prep_kernel<__nv_bfloat16>, T, threads, smem, stream, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_pool,
-                  (__nv_bfloat16*)v_pool, proj, ld, freq, rot, interleaved, amp, norm, eps, positions, seq_of_token, block_table, bt_stride,
-                  num_pages, page_size, nh, nkv, hd, vd, width_k, width_v, err);
-    else return CELLM_ERR_DTYPE;
+    // a warp a head: few tokens take a warp for (nearly) every head, many share a block's warps among the heads
+    const int heads = nh + 2 * nkv, threads = T >= 296 ? (heads >= 8 ? 256 : 128) : heads >= 32 ? 1024 : heads * 32;
+#define TAP_RUN(TA, M)                                                                                                                        \
+    CELLM_RUN((turned_attn_prep_kernel<TA, M>), T, threads, smem, stream, (TA*)q_out, (TA*)k_pool, (TA*)v_pool, proj, ld, freq, rot, interleaved, amp, \
+              norm, eps, positions, seq_of_token, block_table, bt_stride, num_pages, page_size, nh, nkv, hd, vd, width_k, width_v, err)
+    if (dtype == CELLM_F32) {
+        if (width_k <= 64) TAP_RUN(float, 2);
+        else if (width_k <= 128) TAP_RUN(float, 4);
+        else TAP_RUN(float, 0);
+    } else if (dtype == CELLM_BF16) {
+        if (width_k <= 64) TAP_RUN(__nv_bfloat16, 2);
+        else if (width_k <= 128) TAP_RUN(__nv_bfloat16, 4);
+        else TAP_RUN(__nv_bfloat16, 0);
+    } else return CELLM_ERR_DTYPE;
+#undef TAP_RUN
     return CELLM_OK;
 }
