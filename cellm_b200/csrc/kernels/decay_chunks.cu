@@ -34,7 +34,9 @@ struct ChunkArgs {
     const int* cu_seqlens;
     const int* slot_ids;
     int B, min_len, heads, groups, dim, vd, hpc;      // hpc: heads a CTA (of one group)
-    float* ws;              // [chunk][head][dim][vd]: a chunk's own contribution, then the state before it
+    int pitch;              // vd rounded up to a multiple of 8: a row's width in ws
+    float* ws;              // [chunk][head][dim][pitch]: a chunk's own contribution; then, in the same bytes, the state before it
+                            // in packs of eight values, [8 hi | 8 lo] bfloat16
     float* tot;             // [chunk][head]: c_last
 };
 
@@ -50,38 +52,51 @@ __device__ __forceinline__ int find_chunk(const ChunkArgs& a, int chunk, int& t0
     return 0;
 }
 
+// Eight values of a 32-bit row of `width` values from column c0 on (zeros behind the width).
+__device__ __forceinline__ void load8(float (&x)[8], const float* row, int c0, int width, bool ok, bool vec) {
+    if (ok && vec && c0 < width) {
+        const float4 a = *reinterpret_cast<const float4*>(row + c0), b = *reinterpret_cast<const float4*>(row + c0 + 4);
+        x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+    } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = (ok && c0 + e < width) ? row[c0 + e] : 0.f;
+    }
+}
+__device__ __forceinline__ bool rows_of_packs(const float* src, long long ld, int width) {
+    return (width & 7) == 0 && (ld & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0;
+}
+// The two bfloat16 numbers of eight values.
+__device__ __forceinline__ void split8(const float (&x)[8], uint4& hi, uint4& lo) {
+    uint32_t h[4], l[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const __nv_bfloat162 p = __floats2bfloat162_rn(x[2 * e], x[2 * e + 1]);
+        h[e] = *reinterpret_cast<const uint32_t*>(&p);
+        const float2 back = __bfloat1622float2(p);
+        l[e] = pack_bf16(x[2 * e] - back.x, x[2 * e + 1] - back.y);
+    }
+    hi = make_uint4(h[0], h[1], h[2], h[3]);
+    lo = make_uint4(l[0], l[1], l[2], l[3]);
+}
+
 // Rows of a tile [CL][W] (W bfloat16 wide, permuted as mma_tiles.cuh says) from 32-bit rows of `width` values at pitch ld,
 // times scale[row], as hi and lo; zeros behind the width and behind `len` rows.
 template <int W>
-__device__ __forceinline__ void split_rows(uint8_t* hi, uint8_t* lo, const float* src, long long ld, int width, int rows, int len, const float* scale) {
+__device__ __forceinline__ void split_rows(uint8_t* hi, uint8_t* lo, const float* src, long long ld, int width, int len, const float* scale) {
     constexpr int CH = W / 8;
-    const bool vec = (width & 7) == 0 && (ld & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0;
-    for (int i = threadIdx.x; i < rows * CH; i += THREADS) {
-        const int row = i / CH, chunk = i % CH, c0 = chunk * 8;
+    const bool vec = rows_of_packs(src, ld, width);
+#pragma unroll 2
+    for (int i = threadIdx.x; i < CL * CH; i += THREADS) {
+        const int row = i / CH, chunk = i % CH;
         float x[8];
-        if (row < len && vec && c0 < width) {
-            const float4 a = *reinterpret_cast<const float4*>(src + (size_t)row * ld + c0), b = *reinterpret_cast<const float4*>(src + (size_t)row * ld + c0 + 4);
-            x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
-        } else {
-#pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] = (row < len && c0 + e < width) ? src[(size_t)row * ld + c0 + e] : 0.f;
-        }
+        load8(x, src + (size_t)row * ld, chunk * 8, width, row < len, vec);
         if (scale) {
             const float f = scale[row];
 #pragma unroll
             for (int e = 0; e < 8; ++e) x[e] *= f;
         }
-        uint32_t h[4], l[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const __nv_bfloat162 p = __floats2bfloat162_rn(x[2 * e], x[2 * e + 1]);
-            h[e] = *reinterpret_cast<const uint32_t*>(&p);
-            const float2 back = __bfloat1622float2(p);
-            l[e] = pack_bf16(x[2 * e] - back.x, x[2 * e + 1] - back.y);
-        }
         const int off = tile_offset<W>(row, chunk);
-        *reinterpret_cast<uint4*>(hi + off) = make_uint4(h[0], h[1], h[2], h[3]);
-        *reinterpret_cast<uint4*>(lo + off) = make_uint4(l[0], l[1], l[2], l[3]);
+        split8(x, *reinterpret_cast<uint4*>(hi + off), *reinterpret_cast<uint4*>(lo + off));
     }
 }
 
@@ -126,40 +141,44 @@ decay_chunk_states_kernel(const ChunkArgs a) {
     const int len = find_chunk(a, blockIdx.x, t0);
     if (len == 0) return;
     const int h0 = blockIdx.y * a.hpc, g = h0 / (a.heads / a.groups);
-    split_rows<NP>(k_h, k_l, a.k + (size_t)t0 * a.ld_k + (size_t)g * a.dim, a.ld_k, a.dim, CL, len, nullptr);
+    split_rows<NP>(k_h, k_l, a.k + (size_t)t0 * a.ld_k + (size_t)g * a.dim, a.ld_k, a.dim, len, nullptr);
     constexpr int MT = NP / 16, SHARES = 8 / MT;           // warps of a row tile share its column pairs
     const int mt = warp % MT, share = warp / MT;
+    __syncthreads();
+    uint32_t ah[CL / 16][4], al[CL / 16][4];               // the keys serve every head of the CTA
+#pragma unroll
+    for (int kk = 0; kk < CL / 16; ++kk) {
+        const int ar = kk * 16 + (lane & 7) + ((lane >> 4) << 3), ac = mt * 2 + ((lane >> 3) & 1);        // k's rows are the product's columns
+        ldmatrix_x4_trans(ah[kk], k_h + tile_offset<NP>(ar, ac));
+        ldmatrix_x4_trans(al[kk], k_l + tile_offset<NP>(ar, ac));
+    }
     for (int h = h0; h < h0 + a.hpc; ++h) {
         chunk_sums(a, t0, len, h, cum, wr);
         __syncthreads();
         if (threadIdx.x < CL) fac[threadIdx.x] = wr[threadIdx.x] * expf(cum[CL - 1] - cum[threadIdx.x]);
         if (threadIdx.x == 0) a.tot[(size_t)blockIdx.x * a.heads + h] = cum[CL - 1];
         __syncthreads();
-        split_rows<VP>(v_h, v_l, a.v + (size_t)t0 * a.ld_v + (size_t)h * a.vd, a.ld_v, a.vd, CL, len, fac);
+        split_rows<VP>(v_h, v_l, a.v + (size_t)t0 * a.ld_v + (size_t)h * a.vd, a.ld_v, a.vd, len, fac);
         __syncthreads();
-        float* dst = a.ws + ((size_t)blockIdx.x * a.heads + h) * a.dim * a.vd;
+        float* dst = a.ws + ((size_t)blockIdx.x * a.heads + h) * a.dim * a.pitch;
         for (int n2 = share; n2 < VP / 16; n2 += SHARES) {
             float c[2][4] = {};
 #pragma unroll
             for (int kk = 0; kk < CL / 16; ++kk) {
-                uint32_t ah[4], al[4], bh[4], bl[4];
-                const int ar = kk * 16 + (lane & 7) + ((lane >> 4) << 3), ac = mt * 2 + ((lane >> 3) & 1);        // k's rows are the product's columns
-                ldmatrix_x4_trans(ah, k_h + tile_offset<NP>(ar, ac));
-                ldmatrix_x4_trans(al, k_l + tile_offset<NP>(ar, ac));
+                uint32_t bh[4], bl[4];
                 const int br = kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), bc = n2 * 2 + (lane >> 4);
                 ldmatrix_x4_trans(bh, v_h + tile_offset<VP>(br, bc));
                 ldmatrix_x4_trans(bl, v_l + tile_offset<VP>(br, bc));
-                mma3(c[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
-                mma3(c[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+                mma3(c[0], ah[kk], al[kk], bh[0], bh[1], bl[0], bl[1]);
+                mma3(c[1], ah[kk], al[kk], bh[2], bh[3], bl[2], bl[3]);
             }
             const int row = mt * 16 + (lane >> 2);
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
                 const int col = n2 * 16 + n * 8 + (lane & 3) * 2;
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int r = row + (e >> 1) * 8, j = col + (e & 1);
-                    if (r < a.dim && j < a.vd) dst[(size_t)r * a.vd + j] = c[n][e];
+                if (col < a.pitch) {        // an even pitch: both or none (columns behind vd hold zeros)
+                    if (row < a.dim) *reinterpret_cast<float2*>(dst + (size_t)row * a.pitch + col) = make_float2(c[n][0], c[n][1]);
+                    if (row + 8 < a.dim) *reinterpret_cast<float2*>(dst + (size_t)(row + 8) * a.pitch + col) = make_float2(c[n][2], c[n][3]);
                 }
             }
         }
@@ -167,62 +186,83 @@ decay_chunk_states_kernel(const ChunkArgs a) {
     }
 }
 
-// The states before every chunk, in place of the chunks' contributions; the state behind the last one into the slot.
-template <int V>        // values a thread: 4 where a head's state is a multiple of four values, else 1
+// The states before every chunk, in place of the chunks' contributions and already split into two bfloat16 numbers each; the
+// state behind the last one into the slot. A thread a pack of eight columns of one row.
 __global__ void __launch_bounds__(256)
-decay_chunk_pass_kernel(const ChunkArgs a, float* __restrict__ state, long long slot_stride, int n_slots, int* __restrict__ err) {
+decay_chunk_pass_kernel(const ChunkArgs a, float* __restrict__ state, long long slot_stride, int n_slots, int vec, int* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     const int b = blockIdx.x, h = blockIdx.y;
-    const int n_el = a.dim * a.vd, i = (blockIdx.z * 256 + threadIdx.x) * V;
+    const int packs = a.pitch / 8, i = blockIdx.z * 256 + threadIdx.x, row = i / packs, c0 = (i % packs) * 8;
     int first = 0, n = 0;
     for (int bb = 0; bb <= b; ++bb) {
         const int len = a.cu_seqlens[bb + 1] - a.cu_seqlens[bb];
         first += n;
         n = len < a.min_len ? 0 : (len + CL - 1) / CL;
     }
-    if (n == 0 || i >= n_el) return;
+    if (n == 0 || row >= a.dim) return;
     const int slot = a.slot_ids[b];
     if (slot < 0 || slot >= n_slots) { if (threadIdx.x == 0) atomicOr(err, CELLM_DEV_BAD_SLOT); return; }
-    float* st = state + (size_t)slot * slot_stride + (size_t)h * n_el + i;
-    float* w = a.ws + ((size_t)first * a.heads + h) * n_el + i;
-    const size_t pitch = (size_t)a.heads * n_el;
+    float* st = state + (size_t)slot * slot_stride + ((size_t)h * a.dim + row) * a.vd;
+    float* w = a.ws + (((size_t)first * a.heads + h) * a.dim + row) * a.pitch + c0;
+    const size_t step = (size_t)a.heads * a.dim * a.pitch;
     const float* tot = a.tot + (size_t)first * a.heads + h;
-    float s[V];
-#pragma unroll
-    for (int e = 0; e < V; ++e) s[e] = st[e];
-    constexpr int AHEAD = 8;
-    for (int c0 = 0; c0 < n; c0 += AHEAD) {
-        float d[AHEAD][V], f[AHEAD];
+    float s[8];
+    load8(s, st, c0, a.vd, true, vec != 0);
+    constexpr int AHEAD = 4;
+    for (int k0 = 0; k0 < n; k0 += AHEAD) {
+        float d[AHEAD][8], f[AHEAD];
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u) {
-            if (c0 + u < n) {
-                if constexpr (V == 4) {
-                    const float4 x = *reinterpret_cast<const float4*>(w + (size_t)(c0 + u) * pitch);
-                    d[u][0] = x.x; d[u][1] = x.y; d[u][2] = x.z; d[u][3] = x.w;
-                } else {
-                    d[u][0] = w[(size_t)(c0 + u) * pitch];
-                }
-                f[u] = expf(tot[(size_t)(c0 + u) * a.heads]);
+            if (k0 + u < n) {
+                load8(d[u], w + (size_t)(k0 + u) * step, 0, 8, true, true);
+                f[u] = expf(tot[(size_t)(k0 + u) * a.heads]);
             }
         }
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u) {
-            if (c0 + u < n) {
-                if constexpr (V == 4) *reinterpret_cast<float4*>(w + (size_t)(c0 + u) * pitch) = make_float4(s[0], s[1], s[2], s[3]);
-                else w[(size_t)(c0 + u) * pitch] = s[0];
+            if (k0 + u < n) {
+                uint4* dst = reinterpret_cast<uint4*>(w + (size_t)(k0 + u) * step);
+                uint4 hi, lo;
+                split8(s, hi, lo);
+                dst[0] = hi;
+                dst[1] = lo;
 #pragma unroll
-                for (int e = 0; e < V; ++e) s[e] = fmaf(f[u], s[e], d[u][e]);
+                for (int e = 0; e < 8; ++e) s[e] = fmaf(f[u], s[e], d[u][e]);
             }
         }
     }
+    if (vec) {
+        *reinterpret_cast<float4*>(st + c0) = make_float4(s[0], s[1], s[2], s[3]);
+        *reinterpret_cast<float4*>(st + c0 + 4) = make_float4(s[4], s[5], s[6], s[7]);
+    } else {
 #pragma unroll
-    for (int e = 0; e < V; ++e) st[e] = s[e];
+        for (int e = 0; e < 8; ++e)
+            if (c0 + e < a.vd) st[c0 + e] = s[e];
+    }
 }
 
-// Eight warps: four row tiles of 16 tokens, and two halves of the value's columns.
+// The packs of a head's state before the chunk into a tile [NP][VP] (zeros behind its rows and columns), by asynchronous copies.
 template <int NP, int VP>
-__global__ void __launch_bounds__(THREADS)
+__device__ __forceinline__ void copy_state(const ChunkArgs& a, uint8_t* hi, uint8_t* lo, int chunk, int h) {
+    constexpr int CH = VP / 8;
+    const float* src = a.ws + ((size_t)chunk * a.heads + h) * a.dim * a.pitch;
+#pragma unroll 2
+    for (int i = threadIdx.x; i < NP * CH; i += THREADS) {
+        const int row = i / CH, c = i % CH;
+        const bool ok = row < a.dim && c * 8 < a.pitch;
+        const float* p = ok ? src + (size_t)row * a.pitch + c * 8 : src;
+        const int off = tile_offset<VP>(row, c);
+        cp_async16(hi + off, p, ok ? 16 : 0);
+        cp_async16(lo + off, p + 4, ok ? 16 : 0);
+    }
+}
+
+// Eight warps: four row tiles of 16 tokens, and two halves of the value's columns. A head's state arrives by asynchronous
+// copies while the head before is at work, in the keys' place and its own by turns (where the keys' tile is large enough);
+// its values are fetched into registers under the products with the state.
+template <int NP, int VP>
+__global__ void __launch_bounds__(THREADS, VP == 128 ? 1 : 2)
 decay_chunk_outputs_kernel(const ChunkArgs a, float* __restrict__ o_out) {
     extern __shared__ __align__(128) uint8_t dc_smem[];
     uint8_t* q_h = dc_smem;
@@ -232,7 +272,9 @@ decay_chunk_outputs_kernel(const ChunkArgs a, float* __restrict__ o_out) {
     uint8_t* v_h = k_l + CL * NP * 2;
     uint8_t* v_l = v_h + CL * VP * 2;
     uint8_t* s_h = v_l + CL * VP * 2;
-    uint8_t* s_l = s_h + NP * VP * 2;
+    constexpr bool TURNS = VP <= CL;
+    constexpr int STATE = NP * VP * 2;
+    auto state_tile = [&](int n) { return TURNS && (n & 1) ? k_h : s_h; };
     __shared__ float cum[CL], wr[CL];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int rt = warp & 3, half = warp >> 2;
@@ -242,8 +284,10 @@ decay_chunk_outputs_kernel(const ChunkArgs a, float* __restrict__ o_out) {
     const int len = find_chunk(a, blockIdx.x, t0);
     if (len == 0) return;
     const int h0 = blockIdx.y * a.hpc, grp = h0 / (a.heads / a.groups);
-    split_rows<NP>(q_h, q_l, a.q + (size_t)t0 * a.ld_q + (size_t)grp * a.dim, a.ld_q, a.dim, CL, len, nullptr);
-    split_rows<NP>(k_h, k_l, a.k + (size_t)t0 * a.ld_k + (size_t)grp * a.dim, a.ld_k, a.dim, CL, len, nullptr);
+    copy_state<NP, VP>(a, s_h, s_h + STATE, blockIdx.x, h0);
+    cp_async_commit();
+    split_rows<NP>(q_h, q_l, a.q + (size_t)t0 * a.ld_q + (size_t)grp * a.dim, a.ld_q, a.dim, len, nullptr);
+    split_rows<NP>(k_h, k_l, a.k + (size_t)t0 * a.ld_k + (size_t)grp * a.dim, a.ld_k, a.dim, len, nullptr);
     __syncthreads();
     // q_t . k_s for the warp's 16 tokens and the keys up to them
     float qk[CL / 8][4];
@@ -268,11 +312,32 @@ decay_chunk_outputs_kernel(const ChunkArgs a, float* __restrict__ o_out) {
         }
     }
     const int row_a = rt * 16 + (lane >> 2), row_b = row_a + 8;
-    for (int h = h0; h < h0 + a.hpc; ++h) {
+    constexpr int VCH = VP / 8, VIT = CL * VCH / THREADS;          // packs of the values a thread fetches
+    const bool v_vec = rows_of_packs(a.v + (size_t)t0 * a.ld_v, a.ld_v, a.vd);
+    for (int n = 0; n < a.hpc; ++n) {
+        const int h = h0 + n;
+        __syncthreads();            // the keys, and the head before's tiles and sums, are used up
         chunk_sums(a, t0, len, h, cum, wr);
-        split_rows<VP>(v_h, v_l, a.v + (size_t)t0 * a.ld_v + (size_t)h * a.vd, a.ld_v, a.vd, CL, len, nullptr);
-        split_rows<VP>(s_h, s_l, a.ws + ((size_t)blockIdx.x * a.heads + h) * a.dim * a.vd, a.vd, a.vd, NP, a.dim, nullptr);
+        float vx[VIT][8];
+#pragma unroll
+        for (int it = 0; it < VIT; ++it) {
+            const int i = threadIdx.x + it * THREADS, row = i / VCH;
+            load8(vx[it], a.v + (size_t)(t0 + (row < len ? row : 0)) * a.ld_v + (size_t)h * a.vd, (i % VCH) * 8, a.vd, row < len, v_vec);
+        }
+        if (TURNS) {
+            if (n + 1 < a.hpc) {
+                uint8_t* next = state_tile(n + 1);
+                copy_state<NP, VP>(a, next, next + STATE, blockIdx.x, h + 1);
+            }
+            cp_async_commit();
+            cp_async_wait<1>();
+        } else {
+            if (n > 0) { copy_state<NP, VP>(a, s_h, s_h + STATE, blockIdx.x, h); cp_async_commit(); }
+            cp_async_wait<0>();
+        }
         __syncthreads();
+        const uint8_t* st_h = state_tile(n);
+        const uint8_t* st_l = st_h + STATE;
         float acc[VP / 16][4];
 #pragma unroll
         for (int n = 0; n < VP / 16; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
@@ -287,12 +352,18 @@ decay_chunk_outputs_kernel(const ChunkArgs a, float* __restrict__ o_out) {
             for (int n2 = 0; n2 < VP / 32; ++n2) {
                 uint32_t bh[4], bl[4];
                 const int bc = half * (VP / 16) + n2 * 2 + (lane >> 4);
-                ldmatrix_x4_trans(bh, s_h + tile_offset<VP>(br, bc));
-                ldmatrix_x4_trans(bl, s_l + tile_offset<VP>(br, bc));
+                ldmatrix_x4_trans(bh, st_h + tile_offset<VP>(br, bc));
+                ldmatrix_x4_trans(bl, st_l + tile_offset<VP>(br, bc));
                 mma3(acc[2 * n2], ah, al, bh[0], bh[1], bl[0], bl[1]);
                 mma3(acc[2 * n2 + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
             }
         }
+#pragma unroll
+        for (int it = 0; it < VIT; ++it) {
+            const int i = threadIdx.x + it * THREADS, off = tile_offset<VP>(i / VCH, i % VCH);
+            split8(vx[it], *reinterpret_cast<uint4*>(v_h + off), *reinterpret_cast<uint4*>(v_l + off));
+        }
+        __syncthreads();
         const float ca = cum[row_a], cb = cum[row_b], ea = expf(ca), eb = expf(cb);
 #pragma unroll
         for (int n = 0; n < VP / 16; ++n) { acc[n][0] *= ea; acc[n][1] *= ea; acc[n][2] *= eb; acc[n][3] *= eb; }
@@ -343,7 +414,6 @@ decay_chunk_outputs_kernel(const ChunkArgs a, float* __restrict__ o_out) {
                 }
             }
         }
-        __syncthreads();
     }
 }
 
@@ -359,10 +429,8 @@ int launch_chunks(const ChunkArgs& a, float* o_out, float* state, long long slot
     }
     const dim3 grid((unsigned)n_chunks, (unsigned)(a.heads / a.hpc));
     CELLM_RUN((decay_chunk_states_kernel<NP, VP>), grid, THREADS, smem_s, stream, a);
-    const int n_el = a.dim * a.vd;
-    const bool vec = n_el % 4 == 0 && slot_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(state) & 15) == 0 && (reinterpret_cast<uintptr_t>(a.ws) & 15) == 0;
-    if (vec) CELLM_RUN(decay_chunk_pass_kernel<4>, dim3(a.B, a.heads, (n_el / 4 + 255) / 256), 256, 0, stream, a, state, slot_stride, n_slots, err);
-    else CELLM_RUN(decay_chunk_pass_kernel<1>, dim3(a.B, a.heads, (n_el + 255) / 256), 256, 0, stream, a, state, slot_stride, n_slots, err);
+    const int vec = a.vd % 8 == 0 && slot_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(state) & 15) == 0;
+    CELLM_RUN(decay_chunk_pass_kernel, dim3(a.B, a.heads, (a.dim * (a.pitch / 8) + 255) / 256), 256, 0, stream, a, state, slot_stride, n_slots, vec, err);
     CELLM_RUN((decay_chunk_outputs_kernel<NP, VP>), grid, THREADS, smem_o, stream, a, o_out);
     return CELLM_OK;
 }
@@ -373,8 +441,8 @@ int launch_chunks(const ChunkArgs& a, float* o_out, float* state, long long slot
 CELLM_API int cellm_decay_chunks_supports(int dim, int vd) { return dim >= 1 && dim <= 128 && vd >= 1 && vd <= 128; }
 
 // Arguments as cellm_decay_scan's, with the logarithms of the decays (logd, pitch 0: one row of constants). n_chunks: the
-// sum over the portions of at least min_len tokens of ceil(length / 64). ws: [n_chunks, heads, dim, vd] and tot: [n_chunks,
-// heads] 32-bit scratch. Portions shorter than min_len (at least 1) are not touched.
+// sum over the portions of at least min_len tokens of ceil(length / 64). ws: [n_chunks, heads, dim, vd rounded up to a multiple
+// of 8] (16-byte aligned) and tot: [n_chunks, heads] 32-bit scratch. Portions shorter than min_len (at least 1) are not touched.
 CELLM_API int cellm_decay_chunks(float* o_out, float* state, long long slot_stride, int n_slots, const float* q, long long ld_q, const float* k,
                                  long long ld_k, const float* v, long long ld_v, const float* logd, long long ld_d, const float* write,
                                  long long ld_w, const int* cu_seqlens, const int* slot_ids, int B, int n_chunks, int min_len, int heads,
@@ -382,11 +450,12 @@ CELLM_API int cellm_decay_chunks(float* o_out, float* state, long long slot_stri
     if (B <= 0 || n_chunks <= 0) return CELLM_OK;
     if (heads <= 0 || groups <= 0 || heads % groups || min_len < 1 || !cellm_decay_chunks_supports(dim, vd)) return CELLM_ERR_SIZE;
     if (!logd || !ws || !tot) return CELLM_ERR_ARG;
+    if (reinterpret_cast<uintptr_t>(ws) & 15) return CELLM_ERR_ALIGN;
     ChunkArgs a;
     a.q = q, a.k = k, a.v = v, a.logd = logd, a.write = write;
     a.ld_q = ld_q, a.ld_k = ld_k, a.ld_v = ld_v, a.ld_d = ld_d, a.ld_w = ld_w;
     a.cu_seqlens = cu_seqlens, a.slot_ids = slot_ids, a.B = B, a.min_len = min_len;
-    a.heads = heads, a.groups = groups, a.dim = dim, a.vd = vd, a.ws = ws, a.tot = tot;
+    a.heads = heads, a.groups = groups, a.dim = dim, a.vd = vd, a.pitch = (vd + 7) / 8 * 8, a.ws = ws, a.tot = tot;
     // heads of a group taken by one CTA: as many (a power of two that divides the group) as leave some three CTAs an SM
     a.hpc = 1;
     while ((heads / groups) % (a.hpc * 2) == 0 && (long long)n_chunks * (heads / (a.hpc * 2)) >= 444) a.hpc *= 2;

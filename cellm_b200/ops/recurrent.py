@@ -389,8 +389,9 @@ def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.T
     long = [n for n in ctx.q_lens if n >= CHUNKED_FROM] if logd is not None and ctx.max_q_len >= CHUNKED_FROM and max(dim, vd) <= 128 else []
     if long:
         n_chunks = sum(-(-n // 64) for n in long)
-        ws = torch.empty((n_chunks * heads * (dim * vd + 1),), dtype=torch.float32, device=q.device)
-        tot = ws[n_chunks * heads * dim * vd:]
+        n_ws = n_chunks * heads * dim * (-(-vd // 8) * 8)
+        ws = torch.empty((n_ws + n_chunks * heads,), dtype=torch.float32, device=q.device)
+        tot = ws[n_ws:]
         check(fn("decay_chunks", "cellm_decay_chunks")(ptr(o), ptr(state), state.stride(0), state.shape[0], ptr(q), q.stride(0), ptr(k), k.stride(0), ptr(v),
                                                        v.stride(0), ptr(logd), pitch(logd), ptr(write), pitch(write), ptr(ctx.cu_seqlens),
                                                        ptr(ctx.slot_ids), ctx.B, n_chunks, CHUNKED_FROM, heads, groups, dim, vd, ptr(ws), ptr(tot),
