@@ -165,3 +165,29 @@ TIKIZEN_SHAPES = {
     "700m": (_tikizen(1536, 16, [2, 5, 8, 10, 12, 14], [3, 7, 11, 15], [1, 5, 9, 13], 24, 8, 12, 48, 6912, 896, 1536),
              [("padadra", PADADRA_SHAPES["700m"][0]), ("tufadra", TUFADRA_SHAPES["700m"][0])]),
 }
+
+
+# ---- Gonozen shapes beside Tufadra's and Bozovik's -----------------------------------------------------------------
+def _gonozen(width: int, layers: int, full_at, heads: int, q_rank: int, experts: int, top: int, ff: int, shared_ff: int, vocab: int = 65536) -> dict:
+    """Layers of a width and count that a Tufadra and a Bozovik shape have: latent attention as Bozovik's (heads of 128 + 64
+    rotated values, a latent of 512) over every earlier row at a few places, its form without rotation and with a window of
+    1,024 (queries through a latent) elsewhere, and behind every layer Tufadra's mixture (64 experts of which 6 are chosen,
+    in 8 groups of which 4 are kept, a shared one), here gated."""
+    rot = {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}
+    full = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "rot": rot}
+    windowed = {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": 512, "q_rank": q_rank, "scale": 128 ** -0.5, "mask": {"size": 1024}}
+    mlp = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "shared": {"ff": shared_ff, "limit": 7.0},
+           "router": {"experts": experts, "top": top, "groups": {"count": 8, "keep": 4}}}
+    return {"architecture": "Gonozen", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "layers": [{"type": "latent_attention", "mixer": dict(full), "mlp": dict(mlp)} if i in full_at else
+                       {"type": "latent_attention_2", "mixer": dict(windowed), "mlp": dict(mlp)} for i in range(layers)]}
+
+
+# name -> (Gonozen shape, [(a close design's name, its shape of equal width and depth), ...]): Tufadra has the mixture behind every
+# layer, Bozovik seven layers of windowed latent attention
+GONOZEN_SHAPES = {
+    "1.2b": (_gonozen(2048, 16, [2, 5, 8, 11, 14], 16, 1024, 64, 6, 1024, 2048),
+             [("tufadra", TUFADRA_SHAPES["1.2b"][0]), ("bozovik", BOZOVIK_SHAPES["1.2b"][0])]),
+    "700m": (_gonozen(1536, 16, [2, 5, 8, 11, 14], 12, 768, 64, 6, 896, 1536),
+             [("tufadra", TUFADRA_SHAPES["700m"][0]), ("bozovik", BOZOVIK_SHAPES["700m"][0])]),
+}

@@ -25,7 +25,7 @@ latent_flash_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
                     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ pool,
                     const int* __restrict__ cu_seqlens, const int* __restrict__ ctx_lens, const int* __restrict__ block_table,
                     int bt_stride, int B, int T, int num_pages, int page_size, int nh, int kw, int dv, float scale_log2e,
-                    int nsplit, int window, const float* __restrict__ sinks, int* __restrict__ err) {
+                    int nsplit, int window, const float* __restrict__ sinks, const float* __restrict__ gate, int* __restrict__ err) {
     constexpr int NT = DVW / 8;
     extern __shared__ __align__(128) uint8_t smem_raw[];
     const int stride = kw + 8;                                   // elements per row in shared memory (16 bytes of padding)
@@ -198,7 +198,11 @@ latent_flash_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
             if (row_a < rows) l_a += exp2f(sinks[row_a % nh] * 1.4426950408889634f - (m_a == -INFINITY ? 0.f : m_a));
             if (row_b < rows) l_b += exp2f(sinks[row_b % nh] * 1.4426950408889634f - (m_b == -INFINITY ? 0.f : m_b));
         }
-        const float inv_a = l_a > 0.f ? 1.0f / l_a : 0.f, inv_b = l_b > 0.f ? 1.0f / l_b : 0.f;
+        float inv_a = l_a > 0.f ? 1.0f / l_a : 0.f, inv_b = l_b > 0.f ? 1.0f / l_b : 0.f;
+        if (gate) {         // an output gate: the head's sum times the sigmoid of one number per (token, head) row
+            if (row_a < rows) inv_a *= 1.0f / (1.0f + __expf(-gate[base_row + row_a]));
+            if (row_b < rows) inv_b *= 1.0f / (1.0f + __expf(-gate[base_row + row_b]));
+        }
         if (row_a < rows) {
             __nv_bfloat16* dst = out + (base_row + row_a) * dv + col;
 #pragma unroll
@@ -231,7 +235,7 @@ latent_flash_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
 // The pieces of a row merged in their order: out = sum_s 2^(m_s - M) o_s / sum_s 2^(m_s - M) l_s.
 __global__ void latent_merge_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ part_o,
                                     const float* __restrict__ part_ml, size_t n_rows, int dv, int nsplit,
-                                    const float* __restrict__ sinks, int nh) {
+                                    const float* __restrict__ sinks, const float* __restrict__ gate, int nh) {
     extern __shared__ float ml[];        // [nsplit][2]: maximum and sum of each piece, then its weight in [s][0]
     pdl_trigger();
     pdl_wait();
@@ -247,7 +251,7 @@ __global__ void latent_merge_kernel(__nv_bfloat16* __restrict__ out, const float
     float L = 0.f;
     for (int s = 0; s < nsplit; ++s) L += ml[2 * s] == -INFINITY ? 0.f : fast_exp2(ml[2 * s] - M) * ml[2 * s + 1];   // in the pieces' order
     if (sinks) L += exp2f(sinks[r % nh] * 1.4426950408889634f - (M == -INFINITY ? 0.f : M));          // the sink counts once
-    const float inv = L > 0.f ? 1.0f / L : 0.f;
+    const float inv = (L > 0.f ? 1.0f / L : 0.f) * (gate ? 1.0f / (1.0f + __expf(-gate[r])) : 1.0f);
     for (int d = threadIdx.x; d < dv; d += blockDim.x) {
         float acc = 0.f;
 #pragma unroll 8
@@ -346,11 +350,12 @@ CELLM_API int cellm_attention_latent_supports(int kw, int dv) {
 // q: [T, nh, kw] (a head's query against the cached rows); out: [T, nh, dv]; pool: one layer's rows. part_o
 // [nsplit, T * nh, dv] and part_ml [nsplit, T * nh, 2] floats are needed when nsplit > 1. n_tiles: the sum over the
 // requests of ceil(tokens * nh / 64). window: 0, or how many of its last rows a token reads (itself included). sinks [nh]
-// 32-bit: one more term exp(sink_h) in a head's denominator (null: none).
+// 32-bit: one more term exp(sink_h) in a head's denominator (null: none). gate [T, nh] 32-bit: a head's output is multiplied
+// by the sigmoid of its number (null: none).
 CELLM_API int cellm_attention_latent(void* out, float* part_o, float* part_ml, const void* q, const void* pool,
                                      const int* cu_seqlens, const int* ctx_lens, const int* block_table, int bt_stride, int B,
                                      int T, int n_tiles, int num_pages, int page_size, int nh, int kw, int dv, float scale,
-                                     int nsplit, int window, const float* sinks, int* err, cudaStream_t stream) {
+                                     int nsplit, int window, const float* sinks, const float* gate, int* err, cudaStream_t stream) {
     if (T <= 0 || B <= 0 || n_tiles <= 0) return CELLM_OK;
     if (!cellm_attention_latent_supports(kw, dv) || nh <= 0 || page_size <= 0 || nsplit < 1 || !(scale > 0.f) || window < 0) return CELLM_ERR_SIZE;
     if (((uintptr_t)q & 15) || ((uintptr_t)pool & 15) || ((uintptr_t)out & 3)) return CELLM_ERR_ALIGN;
@@ -366,7 +371,7 @@ CELLM_API int cellm_attention_latent(void* out, float* part_o, float* part_ml, c
             cudaFuncSetAttribute(latent_flash_kernel<DVW, BN, SUB, MAXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         CELLM_RUN((latent_flash_kernel<DVW, BN, SUB, MAXT>), grid, threads, smem, stream, (__nv_bfloat16*)out, part_o, part_ml,  \
                   (const __nv_bfloat16*)q, (const __nv_bfloat16*)pool, cu_seqlens, ctx_lens, block_table, bt_stride, B, T,  \
-                  num_pages, page_size, nh, kw, dv, scale_log2e, nsplit, window, sinks, err);                               \
+                  num_pages, page_size, nh, kw, dv, scale_log2e, nsplit, window, sinks, gate, err);                               \
     } while (0)
     if (dvw == 256 && bn == 64) LAUNCH(256, 64, 32, 256);
     else if (dvw == 256) LAUNCH(256, 32, 32, 256);
@@ -377,7 +382,7 @@ CELLM_API int cellm_attention_latent(void* out, float* part_o, float* part_ml, c
 #undef LAUNCH
     if (nsplit > 1)
         CELLM_RUN(latent_merge_kernel, (unsigned)((size_t)T * nh), dv >= 256 ? 256 : (dv >= 128 ? 128 : 64), (size_t)nsplit * 2 * sizeof(float), stream, (__nv_bfloat16*)out, part_o,
-                  part_ml, (size_t)T * nh, dv, nsplit, sinks, nh);
+                  part_ml, (size_t)T * nh, dv, nsplit, sinks, gate, nh);
     return CELLM_OK;
 }
 

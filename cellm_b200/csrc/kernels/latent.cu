@@ -8,8 +8,11 @@
 // part] (kv_rank + rot_dim values), every head reads the same rows, the weighted sum of the rows' first kv_rank
 // values is formed, and V_h turns that sum into the head's output.
 //
-//   latent_prep     norm of c, rotation of the shared key part, cache write; the queries' unrotated parts gathered
-//                   head by head, their rotated parts turned and put behind the place of K_h^T q_h
+// Queries may come through a latent of their own (c_q, RMS-normed with a weight, times a matrix), and a head's output may
+// be multiplied by the sigmoid of one number a token (its pre-activation is a column of the first product).
+//
+//   latent_prep     norm of c, rotation of the shared key part, cache write; norm of c_q; the queries' unrotated parts
+//                   gathered head by head, their rotated parts turned and put behind the place of K_h^T q_h
 //   head_product    out[t, h, :] = W[h] in[t, h, :] for per-head matrices W[h] [N, K] (K_h^T and V_h above)
 //
 // Norm, angles and rotation are 32-bit. Cache layout of one layer: [page][slot in page][kv_rank + rot_dim].
@@ -28,13 +31,18 @@ __device__ __forceinline__ void split_angle(int pos, float hi, float lo, float* 
     *s_out = s * ce + c * se;
 }
 
+// What a launch of the preparation does; a block's role follows from blockIdx.y (in this order, the roles asked for).
+enum { LP_LATENT = 1, LP_QUERY_NORM = 2, LP_QUERIES = 4 };
+
 template <typename TP, typename TA, typename TW>
 __global__ void __launch_bounds__(128)
-latent_prep_kernel(TA* __restrict__ q_plain, TA* __restrict__ q_full, const TP* __restrict__ proj, long long ld,
+latent_prep_kernel(TA* __restrict__ q_plain, TA* __restrict__ q_full, const TP* __restrict__ q_rows, long long q_ld,
+                   TA* __restrict__ cq, const TP* __restrict__ cq_rows, int q_rank, const TW* __restrict__ cq_norm_w,
+                   float* __restrict__ gate_out, const TP* __restrict__ gate_rows, const TP* __restrict__ down_rows, long long ld,
                    const TW* __restrict__ c_norm_w, float eps, const int* __restrict__ positions,
                    const int* __restrict__ seq_of_token, const int* __restrict__ block_table, int bt_stride,
                    TA* __restrict__ pool, int num_pages, int page_size, int heads, int dim, int rot_dim, int rank,
-                   int rot, int interleaved, const float* __restrict__ inv_freq, int* __restrict__ err) {
+                   int rot, int interleaved, const float* __restrict__ inv_freq, float amplitude, int roles, int* __restrict__ err) {
     extern __shared__ float smem[];
     float* cs = smem;                // [rot/2]
     float* sn = smem + rot / 2;      // [rot/2]
@@ -42,95 +50,135 @@ latent_prep_kernel(TA* __restrict__ q_plain, TA* __restrict__ q_full, const TP* 
     pdl_trigger();
     const int t = blockIdx.x;
     const int pos = positions[t];
-    for (int p = threadIdx.x; p < rot / 2; p += blockDim.x) split_angle(pos, inv_freq[2 * p], inv_freq[2 * p + 1], &cs[p], &sn[p]);
-    TA* cache_row = nullptr;
-    if (pool) {
-        const int b = seq_of_token[t];
-        const int page = block_table[(size_t)b * bt_stride + pos / page_size];
-        if (page < 0 || page >= num_pages) {
-            if (threadIdx.x == 0) atomicOr(err, CELLM_DEV_BAD_PAGE);
-        } else {
-            cache_row = pool + ((size_t)page * page_size + pos % page_size) * (rank + rot_dim);
-        }
+    for (int p = threadIdx.x; p < rot / 2; p += blockDim.x) {
+        float c, s;
+        split_angle(pos, inv_freq[2 * p], inv_freq[2 * p + 1], &c, &s);
+        cs[p] = c * amplitude;
+        sn[p] = s * amplitude;
     }
-    __syncthreads();
-    pdl_wait();
-    const TP* row = proj + (size_t)t * ld;
     const int qw = dim + rot_dim, kw = rank + rot_dim;
-    // blockIdx.y = 0: the latent and the shared key part; 1..: a run of query heads each, so that a token's work is
-    // spread over several blocks when the tokens are few
-    if (blockIdx.y > 0) {
-    const int per = (heads + gridDim.y - 2) / (gridDim.y - 1);
-    const int h_lo = min(heads, ((int)blockIdx.y - 1) * per), h_hi = min(heads, h_lo + per);
-    // queries: the unrotated part head by head; the rotated part turned, behind the kv_rank places of its head
-    for (int i = h_lo * dim + threadIdx.x; i < h_hi * dim; i += blockDim.x) {
-        const int h = i / dim, d = i - h * dim;
-        q_plain[(size_t)t * heads * dim + i] = from_float<TA>(to_float(row[h * qw + d]));
-    }
-    for (int i = h_lo * rot_dim + threadIdx.x; i < h_hi * rot_dim; i += blockDim.x) {
-        const int h = i / rot_dim, d = i - h * rot_dim;
-        const TP* src = row + h * qw + dim;
+    // a value of a turned run of rot_dim values: pairs (2p, 2p + 1) when interleaved, (p, p + rot/2) otherwise; the
+    // pair's first entry is u cos - v sin
+    auto turned = [&](const TP* src, int d) {
         float v = to_float(src[d]);
         if (d < rot) {
-            // pairs (2p, 2p + 1) when interleaved, (p, p + rot/2) otherwise; the pair's first entry is u cos - v sin
             const int half = rot >> 1;
             const int p = interleaved ? d >> 1 : (d < half ? d : d - half);
             const bool second = interleaved ? (d & 1) : d >= half;
             const float other = to_float(src[interleaved ? d ^ 1 : (second ? d - half : d + half)]);
             v = second ? v * cs[p] + other * sn[p] : v * cs[p] - other * sn[p];
         }
-        q_full[((size_t)t * heads + h) * kw + rank + d] = from_float<TA>(v);
-    }
-    return;
-    }
-    // the latent: divided by its root mean square, times its weight; the shared key part turned; both to the cache
-    const TP* down = row + (size_t)heads * qw;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < rank; i += blockDim.x) {
-        const float v = to_float(down[i]);
-        ss += v * v;
-    }
-    ss = block_sum(ss, scratch);
-    const float inv = 1.0f / sqrtf(ss / (float)rank + eps);
-    if (cache_row) {
-        for (int i = threadIdx.x; i < rank; i += blockDim.x)
-            cache_row[i] = from_float<TA>(to_float(down[i]) * inv * to_float(c_norm_w[i]));
-        for (int d = threadIdx.x; d < rot_dim; d += blockDim.x) {
-            float v = to_float(down[rank + d]);
-            if (d < rot) {
-                const int half = rot >> 1;
-                const int p = interleaved ? d >> 1 : (d < half ? d : d - half);
-                const bool second = interleaved ? (d & 1) : d >= half;
-                const float other = to_float(down[rank + (interleaved ? d ^ 1 : (second ? d - half : d + half))]);
-                v = second ? v * cs[p] + other * sn[p] : v * cs[p] - other * sn[p];
+        return v;
+    };
+    int role = blockIdx.y;
+    if (roles & LP_LATENT) {
+        if (role == 0) {
+            // the latent: divided by its root mean square, times its weight; the shared key part turned; both to the cache
+            TA* cache_row = nullptr;
+            if (pool) {
+                const int b = seq_of_token[t];
+                const int page = block_table[(size_t)b * bt_stride + pos / page_size];
+                if (page < 0 || page >= num_pages) {
+                    if (threadIdx.x == 0) atomicOr(err, CELLM_DEV_BAD_PAGE);
+                } else {
+                    cache_row = pool + ((size_t)page * page_size + pos % page_size) * kw;
+                }
             }
-            cache_row[rank + d] = from_float<TA>(v);
+            __syncthreads();
+            pdl_wait();
+            const TP* down = down_rows + (size_t)t * ld;
+            float ss = 0.f;
+            for (int i = threadIdx.x; i < rank; i += blockDim.x) {
+                const float v = to_float(down[i]);
+                ss += v * v;
+            }
+            ss = block_sum(ss, scratch);
+            const float inv = 1.0f / sqrtf(ss / (float)rank + eps);
+            if (cache_row) {
+                for (int i = threadIdx.x; i < rank; i += blockDim.x)
+                    cache_row[i] = from_float<TA>(to_float(down[i]) * inv * to_float(c_norm_w[i]));
+                for (int d = threadIdx.x; d < rot_dim; d += blockDim.x) cache_row[rank + d] = from_float<TA>(turned(down + rank, d));
+            }
+            return;
         }
+        --role;
     }
+    if (roles & LP_QUERY_NORM) {
+        if (role == 0) {
+            // the queries' latent: divided by its root mean square, times its weight; the heads' gates as 32-bit numbers
+            pdl_wait();
+            const TP* row = cq_rows + (size_t)t * ld;
+            float ss = 0.f;
+            for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
+                const float v = to_float(row[i]);
+                ss += v * v;
+            }
+            ss = block_sum(ss, scratch);
+            const float inv = 1.0f / sqrtf(ss / (float)q_rank + eps);
+            for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
+                cq[(size_t)t * q_rank + i] = from_float<TA>(to_float(row[i]) * inv * to_float(cq_norm_w[i]));
+            if (gate_out)
+                for (int h = threadIdx.x; h < heads; h += blockDim.x) gate_out[(size_t)t * heads + h] = to_float(gate_rows[(size_t)t * ld + h]);
+            return;
+        }
+        --role;
+    }
+    // the queries, a run of heads a block (so that a token's work is spread over several blocks when the tokens are few):
+    // the unrotated part head by head where a gathered copy is wanted; the rotated part turned, behind the kv_rank places
+    // of its head; the heads' gates
+    __syncthreads();
+    pdl_wait();
+    const TP* row = q_rows + (size_t)t * q_ld;
+    const int runs = (int)gridDim.y - ((roles & LP_LATENT) ? 1 : 0) - ((roles & LP_QUERY_NORM) ? 1 : 0);
+    const int per = (heads + runs - 1) / runs;
+    const int h_lo = min(heads, role * per), h_hi = min(heads, h_lo + per);
+    if (q_plain)
+        for (int i = h_lo * dim + threadIdx.x; i < h_hi * dim; i += blockDim.x) {
+            const int h = i / dim, d = i - h * dim;
+            q_plain[(size_t)t * heads * dim + i] = from_float<TA>(to_float(row[h * qw + d]));
+        }
+    for (int i = h_lo * rot_dim + threadIdx.x; i < h_hi * rot_dim; i += blockDim.x) {
+        const int h = i / rot_dim, d = i - h * rot_dim;
+        q_full[((size_t)t * heads + h) * kw + rank + d] = from_float<TA>(turned(row + h * qw + dim, d));
+    }
+    if (gate_out && !(roles & LP_QUERY_NORM))
+        for (int h = h_lo + threadIdx.x; h < h_hi; h += blockDim.x) gate_out[(size_t)t * heads + h] = to_float(gate_rows[(size_t)t * ld + h]);
 }
 
-// proj: [T, ld] = [heads * (dim + rot_dim) queries | kv_rank latent | rot_dim shared key part] (32-bit, or the
-// activations' type); q_plain: [T, heads * dim]; q_full: [T, heads, kv_rank + rot_dim] (only the last rot_dim of each
-// head are written); pool: one layer's rows or null (the item reads another's cache). rot: how many of the rot_dim
-// values turn (even), in pairs (2p, 2p + 1) if `interleaved`, else (p, p + rot / 2); inv_freq: [rot / 2] pairs of floats
-// (frequency, remainder).
-CELLM_API int cellm_latent_prep(void* q_plain, void* q_full, const void* proj, long long ld, int proj_dtype, const void* c_norm_w,
-                                int w_dtype, float eps, const int* positions, const int* seq_of_token, const int* block_table,
-                                int bt_stride, void* pool, int num_pages, int page_size, int T, int heads, int dim, int rot_dim,
-                                int rank, int rot, int interleaved, const float* inv_freq, int act_dtype, int* err, cudaStream_t stream) {
+// proj: [T, ld], a product's columns (32-bit, or the activations' type): the queries [heads * (dim + rot_dim)], or with
+// q_rank > 0 the queries' latent [q_rank]; behind them, from column down_col, the latent [rank] and the shared key part
+// [rot_dim]; from column gate_col (< 0: none) one number a head. Three things, by `roles`:
+//   1  the latent normed and the key part turned into the cache (pool: one layer's rows; null: another's cache is read)
+//   2  the queries' latent normed into cq [T, q_rank] (with q_rank)
+//   4  of queries q_rows [T, q_ld] (heads of dim + rot_dim): the unrotated parts gathered into q_plain [T, heads * dim]
+//      (null: not wanted), the rotated parts turned into the last rot_dim values of each head of q_full [T, heads, rank + rot_dim]
+// and the gates as 32-bit numbers into gate_out [T, heads] (by 2 where it is asked for, else by 4). rot: how many of the
+// rot_dim values turn (even), in pairs (2p, 2p + 1) if `interleaved`, else (p, p + rot / 2); inv_freq: [rot / 2] pairs of
+// floats (frequency, remainder); cos and sin are multiplied by `amplitude`.
+CELLM_API int cellm_latent_prep(void* q_plain, void* q_full, void* cq, float* gate_out, const void* proj, long long ld, int proj_dtype,
+                                const void* q_rows, long long q_ld, int q_rank, const void* cq_norm_w, int down_col, int gate_col,
+                                const void* c_norm_w, int w_dtype, float eps, const int* positions, const int* seq_of_token,
+                                const int* block_table, int bt_stride, void* pool, int num_pages, int page_size, int T, int heads, int dim,
+                                int rot_dim, int rank, int rot, int interleaved, const float* inv_freq, float amplitude, int roles,
+                                int act_dtype, int* err, cudaStream_t stream) {
     if (T <= 0) return CELLM_OK;
-    if (heads <= 0 || dim < 0 || rot_dim < 0 || rank <= 0 || rot < 0 || rot > rot_dim || (rot & 1)) return CELLM_ERR_SIZE;
-    if (ld < (long long)heads * (dim + rot_dim) + rank + rot_dim) return CELLM_ERR_SIZE;
+    if (heads <= 0 || dim < 0 || rot_dim < 0 || rank <= 0 || rot < 0 || rot > rot_dim || (rot & 1) || q_rank < 0) return CELLM_ERR_SIZE;
+    if (!(roles & 7) || (roles & ~7)) return CELLM_ERR_ARG;
+    if ((roles & LP_LATENT) && (down_col < 0 || ld < (long long)down_col + rank + rot_dim || !c_norm_w)) return CELLM_ERR_SIZE;
+    if ((roles & LP_QUERY_NORM) && (q_rank < 1 || ld < q_rank || !cq || !cq_norm_w)) return CELLM_ERR_SIZE;
+    if ((roles & LP_QUERIES) && (!q_rows || q_ld < (long long)heads * (dim + rot_dim))) return CELLM_ERR_SIZE;
+    if (gate_out && (gate_col < 0 || ld < (long long)gate_col + heads)) return CELLM_ERR_SIZE;
     if (rot > 0 && !inv_freq) return CELLM_ERR_ARG;
     if (pool && (!block_table || page_size <= 0)) return CELLM_ERR_ARG;
     const size_t smem = (size_t)(rot > 0 ? rot : 2) * sizeof(float);
     // few tokens: a token's query heads in up to 8 blocks beside the block of its latent
-    const int qblocks = T >= 256 ? 1 : (heads < 8 ? heads : 8);
-    const dim3 grid((unsigned)T, (unsigned)(1 + qblocks));
+    const int qblocks = !(roles & LP_QUERIES) ? 0 : (T >= 256 ? 1 : (heads < 8 ? heads : 8));
+    const dim3 grid((unsigned)T, (unsigned)(qblocks + ((roles & LP_LATENT) ? 1 : 0) + ((roles & LP_QUERY_NORM) ? 1 : 0)));
 #define LAUNCH(TP, TA, TW)                                                                                              \
-    CELLM_RUN((latent_prep_kernel<TP, TA, TW>), grid, 128, smem, stream, (TA*)q_plain, (TA*)q_full, (const TP*)proj, ld,    \
-              (const TW*)c_norm_w, eps, positions, seq_of_token, block_table, bt_stride, (TA*)pool, num_pages, page_size, \
-              heads, dim, rot_dim, rank, rot, interleaved, inv_freq, err)
+    CELLM_RUN((latent_prep_kernel<TP, TA, TW>), grid, 128, smem, stream, (TA*)q_plain, (TA*)q_full, (const TP*)q_rows, q_ld, (TA*)cq,  \
+              (const TP*)proj, q_rank, (const TW*)cq_norm_w, gate_out, gate_col >= 0 ? (const TP*)proj + gate_col : nullptr,          \
+              (const TP*)proj + down_col, ld, (const TW*)c_norm_w, eps, positions, seq_of_token, block_table, bt_stride, (TA*)pool,   \
+              num_pages, page_size, heads, dim, rot_dim, rank, rot, interleaved, inv_freq, amplitude, roles, err)
     if (act_dtype == CELLM_F32 && proj_dtype == CELLM_F32 && w_dtype == CELLM_F32) LAUNCH(float, float, float);
     else if (act_dtype == CELLM_F32 && proj_dtype == CELLM_F32 && w_dtype == CELLM_BF16) LAUNCH(float, float, __nv_bfloat16);
     else if (act_dtype == CELLM_BF16 && proj_dtype == CELLM_F32 && w_dtype == CELLM_BF16) LAUNCH(float, __nv_bfloat16, __nv_bfloat16);

@@ -9,9 +9,11 @@
 //   the `top` experts with the largest c are chosen; their weights are s / (sum of the chosen s + 1e-20) * scale
 //   out = sum_k weight_k * D_k act(U_k h)  [+ sigmoid(g . h) * shared(h)]
 //
-// Two other forms share the parts around them: a router whose `top` experts are those with the largest z + bias and whose
-// weights are the softmax over the chosen of these sums (route_kernel<., 1>), and gated experts, D_k (silu(G_k h) * (U_k h)),
-// whose gate and up rows lie in blocks of 64 (expert_gate_up_kernel).
+// Other forms share the parts around them: a router whose `top` experts are those with the largest z + bias and whose
+// weights are the softmax over the chosen of these sums (route_kernel<., 1>); one whose scores are the softmax over all
+// experts, whose runs score by their largest, and whose weights are the chosen scores over their sum (route_kernel<., 2>);
+// and gated experts, D_k (silu(G_k h) * (U_k h)) or D_k of the clamped gate, whose gate and up rows lie in blocks of 64
+// (expert_gate_up_kernel).
 //
 // Ties go to the lower index. The chosen experts are listed by descending c, and every sum runs in an order
 // that depends on the sizes alone, so a token's result does not depend on what else is in the batch.
@@ -117,7 +119,9 @@ __device__ __forceinline__ float lane_dot_experts(const TW* const (&w)[4], const
 // warp a token, its scores in shared memory.
 #define ROUTE_THREADS 128
 
-// MODE 0: sigmoid scores, a correction for the choice; MODE 1: the softmax over the chosen z + bias (`correction` the bias).
+// MODE 0: sigmoid scores, a correction for the choice; MODE 1: the softmax over the chosen z + bias (`correction` the bias);
+// MODE 2: the softmax over all experts, a run of neighbours scored by its largest (the choice compares the sums themselves,
+// which the softmax keeps in order).
 template <typename TC, int MODE>
 __global__ void __launch_bounds__(ROUTE_THREADS)
 route_kernel(int* __restrict__ idx, float* __restrict__ wts, float* __restrict__ gate_out, const float* __restrict__ z_all, long long ldz,
@@ -137,7 +141,7 @@ route_kernel(int* __restrict__ idx, float* __restrict__ wts, float* __restrict__
     const float* zr = z_all + (size_t)t * ldz;
     const int gsz = E / n_groups;
     for (int e = lane; e < E; e += 32) {
-        if constexpr (MODE == 1) {
+        if constexpr (MODE >= 1) {
             z[e] = c[e] = zr[e] + (correction ? to_float(correction[e]) : 0.f);
         } else {
             const float s = 1.f / (1.f + expf(-zr[e]));
@@ -147,6 +151,16 @@ route_kernel(int* __restrict__ idx, float* __restrict__ wts, float* __restrict__
     }
     if (has_gate && lane == 0) gate_out[t] = 1.f / (1.f + expf(-zr[E]));
     __syncwarp();
+    if constexpr (MODE == 2) {      // z becomes the scores (the sum over the lanes' shares, lane by lane in one order)
+        float m = -INFINITY;
+        for (int e = lane; e < E; e += 32) m = fmaxf(m, c[e]);
+        m = warp_max(m);
+        float total = 0.f;
+        for (int e = lane; e < E; e += 32) total += expf(c[e] - m);
+        total = warp_sum(total);
+        for (int e = lane; e < E; e += 32) z[e] = expf(c[e] - m) / total;
+        __syncwarp();
+    }
     if (n_groups > 1) {
         for (int gi = lane; gi < n_groups; gi += 32) {
             float m1 = -INFINITY, m2 = -INFINITY;
@@ -155,7 +169,7 @@ route_kernel(int* __restrict__ idx, float* __restrict__ wts, float* __restrict__
                 if (v > m1) { m2 = m1; m1 = v; }
                 else if (v > m2) m2 = v;
             }
-            g[gi] = gsz >= 2 ? m1 + m2 : m1;
+            g[gi] = MODE == 0 && gsz >= 2 ? m1 + m2 : m1;
         }
         __syncwarp();
         for (int gi = lane; gi < n_groups; gi += 32) {
@@ -230,6 +244,26 @@ CELLM_API int cellm_route_softmax(int* idx, float* wts, float* gate_out, const f
     return CELLM_OK;
 }
 
+// The same with scores that are the softmax over all E experts (z + bias, bias null: none), chosen within the `keep` of
+// `n_groups` runs of neighbours whose largest scores are largest; weights: the chosen scores / (their sum + 1e-20) * scale.
+CELLM_API int cellm_route_softmax_all(int* idx, float* wts, float* gate_out, const float* z, long long ldz, const void* bias, int b_dtype, int T,
+                                      int E, int top, int n_groups, int keep, float scale, int has_gate, cudaStream_t stream) {
+    if (T <= 0) return CELLM_OK;
+    if (E < 1 || top < 1 || top > E || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups || keep * (E / n_groups) < top) return CELLM_ERR_SIZE;
+    if (has_gate && !gate_out) return CELLM_ERR_ARG;
+    const size_t smem = (size_t)(ROUTE_THREADS / 32) * (2 * E + 2 * n_groups + top) * sizeof(float);
+    if (smem > 48 * 1024) return CELLM_ERR_SIZE;
+    const unsigned blocks = (unsigned)((T + ROUTE_THREADS / 32 - 1) / (ROUTE_THREADS / 32));
+    if (b_dtype == CELLM_F32)
+        CELLM_RUN((route_kernel<float, 2>), blocks, ROUTE_THREADS, smem, stream, idx, wts, gate_out, z, ldz, (const float*)bias, T, E, top, n_groups,
+                  keep, scale, has_gate);
+    else if (b_dtype == CELLM_BF16)
+        CELLM_RUN((route_kernel<__nv_bfloat16, 2>), blocks, ROUTE_THREADS, smem, stream, idx, wts, gate_out, z, ldz, (const __nv_bfloat16*)bias, T, E,
+                  top, n_groups, keep, scale, has_gate);
+    else return CELLM_ERR_DTYPE;
+    return CELLM_OK;
+}
+
 // ---- the experts, row by row ----------------------------------------------------------------------------------------
 #define EXPERT_THREADS 128
 #define EXPERT_WARPS 4           // a warp forms `rpw` (1, 2 or 4) output rows at once; a block of the first kernel 4 * rpw
@@ -281,11 +315,21 @@ expert_up_kernel(TA* __restrict__ mid, TA* __restrict__ smid, const TA* __restri
 
 // Gated experts: mid[t * top + k, j] = silu(G_e y[t])[j] * (U_e y[t])[j]. gu: [E * 2 ff, H] in blocks of 64 gate rows followed by
 // their 64 up rows (ff a multiple of 64); the shared expert's sgu [2 sff, H] likewise. A warp forms `rpw` (1 or 2)
-// neighbouring outputs, their gate and up rows in flight together.
+// neighbouring outputs, their gate and up rows in flight together. gate.kind 1: the clamped gate instead, with a limit for
+// the experts and one for the shared expert.
+struct ExpertGate { int kind; float limit, shared_limit, slope; };
+
+template <typename TA> __device__ __forceinline__ float expert_gate(float g, float u, const ExpertGate& k, bool is_shared) {
+    if (k.kind == 0) return g / (1.f + expf(-g)) * u;
+    const float limit = is_shared ? k.shared_limit : k.limit;
+    return sizeof(TA) == 4 ? cellm_clamped_gate(g, u, limit, k.slope) : cellm_clamped_gate_rounded(g, u, limit, k.slope);
+}
+
 template <typename TA>
 __global__ void __launch_bounds__(EXPERT_THREADS)
 expert_gate_up_kernel(TA* __restrict__ mid, TA* __restrict__ smid, const TA* __restrict__ y, long long ldy, const TA* __restrict__ gu,
-                      const TA* __restrict__ sgu, const int* __restrict__ idx, int T, int H, int ff, int sff, int top, int E, int rpw) {
+                      const TA* __restrict__ sgu, const int* __restrict__ idx, int T, int H, int ff, int sff, int top, int E, int rpw,
+                      ExpertGate kind) {
     extern __shared__ __align__(16) float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bool is_shared = (int)blockIdx.x >= T * top;
@@ -326,7 +370,7 @@ expert_gate_up_kernel(TA* __restrict__ mid, TA* __restrict__ smid, const TA* __r
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
         const float g = warp_sum(p[2 * j]), u = warp_sum(p[2 * j + 1]);
-        if (lane == 0 && j < nr) (is_shared ? smid : mid)[(size_t)slot * rows + r0 + j] = from_float<TA>(g / (1.f + expf(-g)) * u);
+        if (lane == 0 && j < nr) (is_shared ? smid : mid)[(size_t)slot * rows + r0 + j] = from_float<TA>(expert_gate<TA>(g, u, kind, is_shared));
     }
 }
 
@@ -423,7 +467,8 @@ static int expert_rows_a_warp(long long rows_in_all, int warps, int most, long l
 // Both forms of the experts, row by row; `gated`: up and sup hold gate and up in blocks of 64.
 static int experts_rowwise_impl(void* out, void* mid, void* smid, const void* y, long long ldy, const void* up, const void* down,
                                 const void* sup, const void* sdown, const int* idx, const float* wts, const float* gate, int T, int H,
-                                int ff, int sff, int top, int E, int act, bool gated, int out_dtype, int dtype, cudaStream_t stream) {
+                                int ff, int sff, int top, int E, int act, bool gated, int out_dtype, int dtype, cudaStream_t stream,
+                                ExpertGate kind = ExpertGate{0, 0.f, 0.f, 0.f}) {
     if (T <= 0) return CELLM_OK;
     if (H < 1 || ff < 1 || top < 1 || E < 1 || sff < 0) return CELLM_ERR_SIZE;
     if ((sup == nullptr) != (sdown == nullptr) || (sup && (sff < 1 || !smid))) return CELLM_ERR_ARG;
@@ -450,7 +495,7 @@ static int experts_rowwise_impl(void* out, void* mid, void* smid, const void* y,
         }                                                                                                                         \
         if (gated)                                                                                                                \
             CELLM_RUN(expert_gate_up_kernel<TA>, grid_up, EXPERT_THREADS, smem_up, stream, (TA*)mid, (TA*)smid, (const TA*)y, ldy, \
-                      (const TA*)up, (const TA*)sup, idx, T, H, ff, sff, top, E, rpw_up);                                         \
+                      (const TA*)up, (const TA*)sup, idx, T, H, ff, sff, top, E, rpw_up, kind);                                   \
         else                                                                                                                      \
             CELLM_RUN(expert_up_kernel<TA>, grid_up, EXPERT_THREADS, smem_up, stream, (TA*)mid, (TA*)smid, (const TA*)y, ldy, (const TA*)up,  \
                       (const TA*)sup, idx, T, H, ff, sff, top, E, act, rpw_up);                                                   \
@@ -474,11 +519,15 @@ CELLM_API int cellm_experts_rowwise(void* out, void* mid, void* smid, const void
 }
 
 // Gated experts (see expert_gate_up_kernel): gu [E * 2 ff, H], down [E * H, ff], sgu [2 sff, H], sdown [H, sff]; ff and sff
-// multiples of 64. out of element type out_dtype (the activations' or 32-bit).
+// multiples of 64. out of element type out_dtype (the activations' or 32-bit). gate_kind 0: silu(g) * u; 1: the clamped gate
+// with `slope`, `limit` for the experts and `shared_limit` for the shared expert.
 CELLM_API int cellm_experts_gated_rowwise(void* out, void* mid, void* smid, const void* y, long long ldy, const void* gu, const void* down,
                                           const void* sgu, const void* sdown, const int* idx, const float* wts, const float* gate, int T, int H,
-                                          int ff, int sff, int top, int E, int out_dtype, int dtype, cudaStream_t stream) {
-    return experts_rowwise_impl(out, mid, smid, y, ldy, gu, down, sgu, sdown, idx, wts, gate, T, H, ff, sff, top, E, 0, true, out_dtype, dtype, stream);
+                                          int ff, int sff, int top, int E, int gate_kind, float limit, float shared_limit, float slope, int out_dtype,
+                                           int dtype, cudaStream_t stream) {
+    if (gate_kind < 0 || gate_kind > 1) return CELLM_ERR_ARG;
+    return experts_rowwise_impl(out, mid, smid, y, ldy, gu, down, sgu, sdown, idx, wts, gate, T, H, ff, sff, top, E, 0, true, out_dtype, dtype, stream,
+                                ExpertGate{gate_kind, limit, shared_limit, slope});
 }
 
 // ---- a plain activation: h = act(u) for 32-bit sums u [T, n] (row pitch ld) ----------------------------------------------

@@ -311,6 +311,7 @@ API long long cellm_exec_sizeof(int which) {
         case 18: return sizeof(cellm::LatentAttentionParams);
         case 19: return sizeof(cellm::GatedMlpParams);
         case 20: return sizeof(cellm::RoutedMlpParams);
+        case 21: return sizeof(cellm::ResultNormParams);
         default: return -1;
     }
 }

@@ -45,9 +45,10 @@ typedef int (*GatedNormAddFn)(P x, CP m, CP m_bias, CP gate, i64 gate_ld, int ga
 typedef int (*StreamCastFn)(P y, CP x, i64 n, int act_tag, P stream);
 typedef int (*MinGruScanFn)(P out, CP proj, i64 ld, int proj_tag, CP bz, CP bx, int w_tag, P state, i64 slot_stride, CP slot_ids, CP cu,
                             int T, int B, int W, int n_slots, int max_q_len, int act_tag, P err, P stream);
-typedef int (*LatentPrepFn)(P q_plain, P q_full, CP proj, i64 ld, int proj_tag, CP c_norm_w, int w_tag, float eps, CP positions, CP seq,
+typedef int (*LatentPrepFn)(P q_plain, P q_full, P cq, P gate_out, CP proj, i64 ld, int proj_tag, CP q_rows, i64 q_ld, int q_rank, CP cq_norm_w,
+                            int down_col, int gate_col, CP c_norm_w, int w_tag, float eps, CP positions, CP seq,
                             CP bt, int bt_stride, P pool, int pages, int page_size, int T, int heads, int dim, int rot_dim, int rank,
-                            int rot, int interleaved, CP inv_freq, int act_tag, P err, P stream);
+                            int rot, int interleaved, CP inv_freq, float amplitude, int roles, int act_tag, P err, P stream);
 typedef int (*AttentionPlainMaskedFn)(P out, CP q, CP kp, CP vp, CP positions, CP seq, CP bt, int bt_stride, int pages, int page_size,
                                       int T, int nh, int nkv, int hd, int hdv, int v_row, float scale, int window, int keep_first,
                                       CP sinks, float fixed_sink, int has_fixed_sink, CP gate, i64 gate_ld, int tag, P err, P stream);
@@ -56,8 +57,8 @@ typedef int (*GatedActFn)(P h, CP gu, i64 ld, CP bg, CP bu, int w_tag, int T, in
 typedef int (*BiasAddFn)(P out, CP in, CP b, int w_tag, int T, int N, int tag, P stream);
 typedef int (*HeadProductMmaFn)(P out, i64 ldo, i64 out_hs, CP in, i64 ldi, i64 in_hs, CP w, int T, int heads, int N, int K, P stream);
 typedef int (*AttentionLatentFn)(P out, P part_o, P part_ml, CP q, CP pool, CP cu, CP ctx, CP bt, int bt_stride, int B, int T, int n_tiles,
-                                 int pages, int page_size, int nh, int kw, int dv, float scale, int nsplit, int window, CP sinks, P err,
-                                 P stream);
+                                 int pages, int page_size, int nh, int kw, int dv, float scale, int nsplit, int window, CP sinks, CP gate,
+                                 P err, P stream);
 typedef int (*EmbedPosFn)(P out, CP table, int tag, CP ids, CP pos_table, CP positions, int max_pos, int T, int H, int V, float scale, P err,
                           P stream);
 typedef int (*AttnPrepFn)(P q, CP qkv, i64 row_stride, CP q_w, CP k_w, int w_tag, float eps, int span, float temp_coef, int temp_every,
@@ -76,7 +77,12 @@ typedef int (*ActivationFn)(P h, CP u, i64 ld, int T, int n, int act, int tag, P
 
 typedef int (*RouteSoftmaxFn)(P idx, P wts, P gate, CP z, i64 ldz, CP bias, int b_tag, int T, int E, int top, float scale, int has_gate, P stream);
 typedef int (*ExpertsGatedRowwiseFn)(P out, P mid, P smid, CP y, i64 ldy, CP gu, CP down, CP sgu, CP sdown, CP idx, CP wts, CP gate, int T, int H,
-                                     int ff, int sff, int top, int E, int out_tag, int tag, P stream);
+                                     int ff, int sff, int top, int E, int gate_kind, float limit, float shared_limit, float slope, int out_tag, int tag,
+                                     P stream);
+typedef int (*RouteSoftmaxAllFn)(P idx, P wts, P gate, CP z, i64 ldz, CP bias, int b_tag, int T, int E, int top, int n_groups, int keep, float scale,
+                                 int has_gate, P stream);
+typedef int (*NormAddNormFn)(P x, CP delta, CP w_d, float eps_d, CP w, int w_tag, P y, CP rows, int n, int H, float eps, int act_tag, P stream);
+typedef int (*SoftCapFn)(P z, i64 n, float cap, P stream);
 typedef int (*GemmGatedFn)(P c, CP a, CP w, int M, int N, int K, i64 lda, i64 ldw, i64 ldc, int out_tag, int bn, int split_k, int gate_kind,
                            float limit, float slope, int w_is_static, P ws, P counters, P err, P stream);
 typedef int (*GemmGroupedGatedFn)(P c, CP a, CP w, int M, int N, int K, int groups, i64 lda, i64 ldw, i64 ldc, int out_tag, CP tile_group,
@@ -244,6 +250,24 @@ struct Run {
     // feed-forward read the same norm's output): regs.pending, the older, and pending2. They lie in the two output
     // slots, so before a third part writes, the older one goes into the stream.
     const void* pending2 = nullptr;
+    // the norm that the waiting result takes before it joins the stream (set only while one result waits)
+    const ResultNormParams* pending_norm = nullptr;
+    // for what is not a norm that takes both: the result is normed and added by a kernel of its own
+    void join_normed() {
+        if (!pending_norm) return;
+        const ResultNormParams& n = *pending_norm;
+        LAUNCH(fn<GatedNormAddFn>(FN_GATED_NORM_ADD)(regs.x, regs.pending, nullptr, nullptr, p.H, (int)act, nullptr, n.w, (int)n.w_dtype, nullptr, (int)s.T,
+                                                 (int)p.H, 1, (float)n.eps, (int)act, s.stream),
+               "gated_norm_add");
+        stream_in_y = false;
+        regs.pending = nullptr;
+        pending_norm = nullptr;
+    }
+    void result_norm(const ResultNormParams& n) {
+        if (dry && !regs.pending) return;       // the sizing walk calls no Python part: one before this record has left nothing
+        if (!regs.pending || pending2 || pending_norm) throw std::runtime_error("executor: a norm over a result without exactly one result before it");
+        pending_norm = &n;
+    }
     void add_older_now() {
         if (!regs.pending) return;
         LAUNCH(fn<ResidualAddFn>(FN_RESIDUAL_ADD)(regs.x, regs.pending, s.T * p.H, (int)act, s.stream), "residual_add");
@@ -253,6 +277,7 @@ struct Run {
     }
     // for what knows one addend only (a Python part, the stream's readers): the second joins the stream at once
     void one_addend() {
+        join_normed();
         if (!pending2) return;
         LAUNCH(fn<ResidualAddFn>(FN_RESIDUAL_ADD)(regs.x, pending2, s.T * p.H, (int)act, s.stream), "residual_add");
         stream_in_y = false;
@@ -282,8 +307,13 @@ struct Run {
         const bool rows = regs.phase == 2;
         arena.release();
         const i64 count = rows ? s.R : s.T;
+        if (pending_norm && (n.groups > 1 || pending_norm->w_dtype != n.dtype)) join_normed();
         void* y = arena.take(count * p.H * elt(act));
-        if (pending2)
+        if (pending_norm)
+            LAUNCH(fn<NormAddNormFn>(FN_NORM_ADD_NORM)(regs.x, regs.pending, pending_norm->w, (float)pending_norm->eps, n.w, (int)n.dtype, y,
+                                                   rows ? s.rows : nullptr, (int)count, (int)p.H, (float)n.eps, (int)act, s.stream),
+                   "norm_add_norm");
+        else if (pending2)
             LAUNCH(fn<Add2RmsnormFn>(FN_ADD2_RMSNORM)(regs.x, regs.pending, pending2, n.w, (int)n.dtype, y, rows ? s.rows : nullptr, (int)count,
                                                   (int)p.H, (int)std::max<i64>(n.groups, 1), (float)n.eps, (int)act, s.stream),
                    "add2_rmsnorm");
@@ -291,7 +321,7 @@ struct Run {
         LAUNCH(fn<AddRmsnormFn>(FN_ADD_RMSNORM)(regs.x, regs.pending, n.w, (int)n.dtype, y, rows ? s.rows : nullptr, (int)count, (int)p.H,
                                             (int)std::max<i64>(n.groups, 1), (float)n.eps, (int)act, s.stream),
            "add_rmsnorm");
-        if (!rows) regs.pending = pending2 = nullptr;      // with rows given the stream itself is not touched
+        if (!rows) regs.pending = pending2 = nullptr, pending_norm = nullptr;      // with rows given the stream itself is not touched
         regs.y = y;
         stream_in_y = false;
     }
@@ -299,6 +329,8 @@ struct Run {
         if (regs.phase != 2) throw std::runtime_error("executor: the output product belongs to the epilogue");
         if (h.w.dtype != act) throw std::runtime_error("executor: a head whose element type differs from the activations'");
         product(regs.logits, input(), h.w, s.R, p.H, EXEC_F32);
+        if (h.soft_cap > 0.0)
+            LAUNCH(fn<SoftCapFn>(FN_SOFT_CAP)(static_cast<float*>(regs.logits), s.R * p.V, (float)h.soft_cap, s.stream), "soft_cap");
     }
     void python(const PythonParams& py) {
         if (dry) {
@@ -339,7 +371,7 @@ struct Run {
     void gated_norm_add(const GatedNormAddParams& n) {
         if (!regs.pending) throw std::runtime_error("executor: a gate and norm without a sublayer's result before them");
         if (regs.phase != 1) throw std::runtime_error("executor: a gate and norm outside the layers");
-        if (pending2) throw std::runtime_error("executor: a gate and norm with two results before them");
+        if (pending2 || pending_norm) throw std::runtime_error("executor: a gate and norm with two results, or a normed one, before them");
         const i64 T = s.T, H = p.H;
         const void* g = nullptr;
         i64 g_ld = H, g_dtype = act;
@@ -416,8 +448,10 @@ struct Run {
             case OP_HEAD: head(*static_cast<const HeadParams*>(op.params)); break;
             case OP_PYTHON: python(*static_cast<const PythonParams*>(op.params)); break;
             case OP_READ_STREAM: read_stream(); break;
+            case OP_RESULT_NORM: result_norm(*static_cast<const ResultNormParams*>(op.params)); break;
             case OP_GATED_NORM_ADD: gated_norm_add(*static_cast<const GatedNormAddParams*>(op.params)); break;
             case OP_SHORT_CONV: case OP_ATTENTION: case OP_SWIGLU: case OP_MINGRU: case OP_LATENT_ATTENTION: case OP_GATED_MLP: case OP_ROUTED_MLP: {
+                join_normed();
                 if (regs.pending && pending2) add_older_now();      // both output slots are taken: the older addend's is written next
                 void* out = slot[turn];
                 produce(op, it, input(), out);
@@ -762,7 +796,14 @@ void Run::routed_mlp(const RoutedMlpParams& L, const void* x, void* out) {
     // the router's sums (and the shared expert's gate, one row more of the same matrix) as a product with 32-bit output
     void* z = linear(x, L.router, T, H, EXEC_F32);
     const i64 out_dtype = L.out32 ? (i64)EXEC_F32 : act;
-    if (L.softmax)
+    if (L.gate_kind && !L.gated) throw std::runtime_error("executor: a clamped gate belongs to gated experts");
+    const int gate_kind = (int)L.gate_kind;
+    const float limit = (float)L.limit, shared_limit = (float)L.shared_limit, slope = (float)L.slope;
+    if (L.softmax == 2)
+        LAUNCH(fn<RouteSoftmaxAllFn>(FN_ROUTE_SOFTMAX_ALL)(idx, wts, gate, z, L.router.N, L.correction, (int)L.c_dtype, (int)T, (int)L.experts, (int)L.top,
+                                                       (int)L.n_groups, (int)L.keep, (float)L.scale, L.shared_gate ? 1 : 0, s.stream),
+               "route_softmax_all");
+    else if (L.softmax)
         LAUNCH(fn<RouteSoftmaxFn>(FN_ROUTE_SOFTMAX)(idx, wts, gate, z, L.router.N, L.correction, (int)L.c_dtype, (int)T, (int)L.experts, (int)L.top,
                                                 (float)L.scale, L.shared_gate ? 1 : 0, s.stream),
                "route_softmax");
@@ -778,7 +819,7 @@ void Run::routed_mlp(const RoutedMlpParams& L, const void* x, void* out) {
         if (L.gated)
             LAUNCH(fn<ExpertsGatedRowwiseFn>(FN_EXPERTS_GATED_ROWWISE)(out, mid, smid, x, H, L.up.w, L.down.w, L.shared_up.w, L.shared_down.w, idx, wts,
                                                                    gate, (int)T, (int)H, (int)L.ff, (int)L.shared_ff, (int)L.top, (int)L.experts,
-                                                                   (int)out_dtype, (int)act, s.stream),
+                                                                   gate_kind, limit, shared_limit, slope, (int)out_dtype, (int)act, s.stream),
                    "experts_gated_rowwise");
         else
         LAUNCH(fn<ExpertsRowwiseFn>(FN_EXPERTS_ROWWISE)(out, mid, smid, x, H, L.up.w, L.down.w, L.shared_up.w, L.shared_down.w, idx, wts, gate,
@@ -798,8 +839,8 @@ void Run::routed_mlp(const RoutedMlpParams& L, const void* x, void* out) {
             plan_tiles(T, L.shared_up.N, H, p.sms, &bn, &split);
             if (bn == 64) bn = 128;
             else if (bn > 128 && bn < 256) bn = 256;
-            const Gate swiglu{0, 0.f, 0.f};
-            gemm_tc(h, x, L.shared_up, T, L.shared_up.N, H, act, bn, split, 1, -1, &swiglu);
+            const Gate shared_gate{gate_kind, shared_limit, slope};
+            gemm_tc(h, x, L.shared_up, T, L.shared_up.N, H, act, bn, split, 1, -1, &shared_gate);
         } else if (tc_ok(L.shared_up, H)) {        // the activation on the 32-bit sums in the product's epilogue
             LAUNCH(fn<GemmGroupedFn>(FN_GEMM_GROUPED)(h, x, L.shared_up.w, (int)T, (int)L.shared_ff, (int)H, 1, H, L.shared_up.ldw, L.shared_ff,
                                                   (int)EXEC_BF16, nullptr, (int)L.act, s.err, s.stream),
@@ -823,7 +864,7 @@ void Run::routed_mlp(const RoutedMlpParams& L, const void* x, void* out) {
         void* mid = arena.take(rows * L.ff * 2);
         if (L.gated)
             LAUNCH(fn<GemmGroupedGatedFn>(FN_GEMM_GROUPED_GATED)(mid, xs, L.up.w, (int)rows, (int)(2 * L.ff), (int)H, (int)L.experts, H, L.up.ldw, L.ff,
-                                                             (int)EXEC_BF16, tile_group, 0, 0.f, 0.f, s.err, s.stream),
+                                                             (int)EXEC_BF16, tile_group, gate_kind, limit, slope, s.err, s.stream),
                    "gemm_grouped_gated_tcgen05");
         else
         LAUNCH(fn<GemmGroupedFn>(FN_GEMM_GROUPED)(mid, xs, L.up.w, (int)rows, (int)L.ff, (int)H, (int)L.experts, H, L.up.ldw, L.ff, (int)EXEC_BF16,
@@ -855,18 +896,39 @@ void Run::mingru(const MinGruParams& L, const ExecItem& it, const void* x, void*
 }
 
 void Run::latent_attention(const LatentAttentionParams& L, const ExecItem& it, const void* x, void* out) {
-    const i64 T = s.T, H = p.H, nh = L.heads, kw = L.rank + L.rot_dim, e = elt(act);
+    const i64 T = s.T, H = p.H, nh = L.heads, qw = L.dim + L.rot_dim, kw = L.rank + L.rot_dim, e = elt(act);
     void* proj = linear(x, L.in_proj, T, H, act);
     if (L.extra) gate_at = static_cast<const char*>(proj) + (L.in_proj.N - L.extra) * e, gate_ld = L.in_proj.N, gate_dtype = act;
-    void* q_plain = arena.take(T * nh * L.dim * e);
+    const i64 down_col = L.q_rank ? L.q_rank : nh * qw, gate_col = L.gate ? down_col + kw : -1;
     void* q_full = arena.take(T * nh * kw * e);
-    LAUNCH(fn<LatentPrepFn>(FN_LATENT_PREP)(q_plain, q_full, proj, L.in_proj.N, (int)act, L.c_norm_w, (int)L.c_norm_dtype, (float)L.eps,
-                                        s.positions, s.seq_of_token, it.block_table, (int)it.bt_stride, it.writes ? it.k : nullptr,
-                                        (int)it.num_pages, (int)it.page_size, (int)T, (int)nh, (int)L.dim, (int)L.rot_dim, (int)L.rank,
-                                        (int)L.rot, (int)L.interleaved, L.inv_freq, (int)act, s.err, s.stream),
-           "latent_prep");
+    float* out_gate = L.gate ? static_cast<float*>(arena.take(T * nh * 4)) : nullptr;
+    enum { LATENT = 1, QUERY_NORM = 2, QUERIES = 4 };
+    auto prep = [&](int roles, void* q_plain, void* cq, float* gate_out, const void* q_rows, i64 q_ld) {
+        LAUNCH(fn<LatentPrepFn>(FN_LATENT_PREP)(q_plain, q_full, cq, gate_out, proj, L.in_proj.N, (int)act, q_rows, q_ld, (int)L.q_rank, L.q_norm_w,
+                                            (int)down_col, (int)gate_col, L.c_norm_w, (int)L.c_norm_dtype, (float)L.eps, s.positions,
+                                            s.seq_of_token, it.block_table, (int)it.bt_stride, it.writes ? it.k : nullptr, (int)it.num_pages,
+                                            (int)it.page_size, (int)T, (int)nh, (int)L.dim, (int)L.rot_dim, (int)L.rank, (int)L.rot,
+                                            (int)L.interleaved, L.inv_freq, (float)L.amplitude, roles, (int)act, s.err, s.stream),
+               "latent_prep");
+    };
+    // the queries' rows: columns of the first product, or a product of their own latent's norm
+    const void* q_rows = proj;
+    i64 q_ld = L.in_proj.N;
+    if (L.q_rank) {
+        void* cq = arena.take(T * L.q_rank * e);
+        prep(LATENT | QUERY_NORM, nullptr, cq, out_gate, nullptr, 0);
+        q_rows = linear(cq, L.q_up, T, L.q_rank, act);
+        q_ld = L.q_up.N;
+    }
+    // the per-head products read a head's unrotated part where it lies; rows that break the tensor cores' alignment are gathered first
+    const bool in_place = act == EXEC_F32 || (q_ld % 8 == 0 && qw % 8 == 0);
+    void* q_plain = in_place ? nullptr : arena.take(T * nh * L.dim * e);
+    const bool queries = q_plain || L.rot_dim || (L.gate && !L.q_rank);
+    if (!L.q_rank) prep(LATENT | (queries ? QUERIES : 0), q_plain, nullptr, out_gate, q_rows, q_ld);
+    else if (queries) prep(QUERIES, q_plain, nullptr, nullptr, q_rows, q_ld);
     // a head's query against the cached rows: [K_h^T q_h | rotated part]
-    head_products(q_full, nh * kw, kw, q_plain, nh * L.dim, L.dim, L.absorb_k, T, nh, L.rank, L.dim);
+    if (in_place) head_products(q_full, nh * kw, kw, q_rows, q_ld, qw, L.absorb_k, T, nh, L.rank, L.dim);
+    else head_products(q_full, nh * kw, kw, q_plain, nh * L.dim, L.dim, L.absorb_k, T, nh, L.rank, L.dim);
     // every head reads the same rows (one key/value head); a value is a row's first `rank` entries
     void* o_lat = arena.take(T * nh * L.rank * e);
     // bfloat16 and sizes the tensor-core kernel takes (multiples of 16, value columns that split over its warps, tiles
@@ -898,14 +960,14 @@ void Run::latent_attention(const LatentAttentionParams& L, const ExecItem& it, c
         LAUNCH(fn<AttentionLatentFn>(FN_ATTENTION_LATENT)(o_lat, part_o, part_ml, q_full, it.k, s.cu_seqlens, s.ctx_lens, it.block_table,
                                                       (int)it.bt_stride, (int)s.B, (int)T, (int)n_tiles, (int)it.num_pages,
                                                       (int)it.page_size, (int)nh, (int)kw, (int)L.rank, (float)L.scale, (int)nsplit,
-                                                      (int)L.window, L.sinks, s.err, s.stream),
+                                                      (int)L.window, L.sinks, out_gate, s.err, s.stream),
                "attention_latent");
         if (nsplit > 1) ++launches;                    // the merge of the pieces
-    } else if (L.window || L.sinks)
+    } else if (L.window || L.sinks || out_gate)
     LAUNCH(fn<AttentionPlainMaskedFn>(FN_ATTENTION_PLAIN_MASKED)(o_lat, q_full, it.k, it.k, s.positions, s.seq_of_token, it.block_table,
                                                              (int)it.bt_stride, (int)it.num_pages, (int)it.page_size, (int)T, (int)nh, 1,
                                                              (int)kw, (int)L.rank, (int)kw, (float)L.scale, (int)L.window, 0, L.sinks, 0.f, 0,
-                                                             nullptr, 0, (int)act, s.err, s.stream),
+                                                             out_gate, nh, (int)act, s.err, s.stream),
            "attention_plain_masked");
     else
     LAUNCH(fn<AttentionPlainFn>(FN_ATTENTION_PLAIN)(o_lat, q_full, it.k, it.k, s.positions, s.seq_of_token, it.block_table, (int)it.bt_stride,

@@ -54,7 +54,9 @@ enum OpKind : i64 {
     // a layer whose sublayers read the stream itself and whose results join it through a gate and a norm
     OP_READ_STREAM, OP_GATED_NORM_ADD, OP_MINGRU, OP_LATENT_ATTENTION, OP_GATED_MLP,
     // a feed-forward whose tokens each run a few of many small experts, chosen by a router
-    OP_ROUTED_MLP, OP_KINDS
+    OP_ROUTED_MLP,
+    // a norm over a sublayer's result before it joins the stream
+    OP_RESULT_NORM, OP_KINDS
 };
 
 struct ExecOp {
@@ -86,7 +88,7 @@ struct SwiGLUParams {
     ExecLinear gate_up, down;
     i64 ff, fused;      // fused: gate_up holds interleaved gate and up blocks for the product's SwiGLU epilogue
 };
-struct HeadParams { ExecLinear w; };                                   // logits = y . w^T in 32-bit
+struct HeadParams { ExecLinear w; double soft_cap; };                  // logits = y . w^T in 32-bit; soft_cap c > 0: c tanh(logits / c)
 struct PythonParams { i64 token; };                                    // the interpreter's name for the part
 struct LinearParams { ExecLinear w; i64 lda, out_dtype; };             // out [T, N] = in [T, K] (row pitch lda) . w^T
 // OP_ATTEND takes AttentionParams and reads only nh, nkv, hd, window and scale: out = attention of the queries `in`
@@ -99,13 +101,19 @@ struct ReadStreamParams { i64 reserved; };
 // gate.w null: no gate. y is the sublayer's input when the record starts.
 // stacked: the gate's rows lie behind the rows of the sublayer's own first product (its `extra`), which has formed the gate already.
 struct GatedNormAddParams { ExecLinear gate; const void* gate_bias; const void* w; i64 w_dtype, groups; double eps; i64 stacked; };
+// The waiting result of a sublayer is RMS-normed before it joins the stream: x += rms_norm(pending) * w. Nothing is launched
+// here: the next norm does it on its way (one kernel for both norms and the sum), or whatever else needs the stream first.
+struct ResultNormParams { const void* w; i64 w_dtype; double eps; };
 // minGRU: in_proj stacks the rows of z, candidate and output gate ([3 * width, H]); the state is the item's slot [width].
 // `extra` (here and below): rows stacked behind the part's own in its first matrix, whose products the part leaves for the
 // record after it (a gate over the same input).
 struct MinGruParams { ExecLinear in_proj, out_proj; const void* bz; const void* bx; i64 b_dtype, width, extra; };
 // Latent attention: in_proj stacks the queries' rows (heads * (dim + rot_dim)), the latent's (rank) and the shared
 // rotated key part's (rot_dim). absorb_k: [heads, rank, dim] (a head's key matrix transposed), expand_v: [heads, vdim,
-// rank]. The item's pages hold rows of rank + rot_dim values.
+// rank]. The item's pages hold rows of rank + rot_dim values. Two more forms:
+// q_rank > 0: queries through a latent of their own: in_proj's first rows are q_rank instead of the queries', q_up
+// [heads * (dim + rot_dim), q_rank] makes the queries from its norm. gate: `heads` rows behind the shared key part's; a
+// head's output is multiplied by the sigmoid of its row's product. (Rows of zeros may follow, then the `extra` ones.)
 struct LatentAttentionParams {
     ExecLinear in_proj, out_proj;
     const void* absorb_k; const void* expand_v;
@@ -116,6 +124,10 @@ struct LatentAttentionParams {
     i64 interleaved;            // the rotation's pairs: (2p, 2p + 1), or (p, p + rot / 2)
     i64 window;                 // 0: every earlier row; w: a token reads its last w rows
     const void* sinks;          // [heads] 32-bit: one more term exp(sink_h) in a head's denominator; null: none
+    double amplitude;           // factor of cos and sin
+    ExecLinear q_up;
+    const void* q_norm_w; i64 q_rank;   // of c_norm_w's element type, with its eps
+    i64 gate;
 };
 // down . (act(gate . y + bg) * (up . y + bu)) + bd; act 0 silu, 1 gelu (tanh form); the biases may be null.
 // act 2, the clamped gate (no biases): g' sigmoid(slope g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit).
@@ -130,8 +142,10 @@ struct GatedMlpParams {
 // up: [experts * ff, H] and down: [experts * H, ff], the experts' matrices one below the other. router: [experts (+ 1), H], the
 // last row the shared expert's gate when it has one. The choice: see routed.cu. act: 0 gelu (erf), 1 gelu (tanh), 2 silu, 3 relu.
 // gated: the experts are down_e (silu(gate_e y) * (up_e y)); `up` (and shared_up) holds gate and up in blocks of 64 rows,
-// [experts * 2 ff, H], ff (and shared_ff) a multiple of 64; act is not read. softmax: the router chooses by the largest sums
-// (+ correction, a bias; null: none) and weighs by the softmax over the chosen. out32: as above.
+// [experts * 2 ff, H], ff (and shared_ff) a multiple of 64; act is not read. gate_kind 1: the clamped gate in silu's place
+// (`limit`, the shared expert's `shared_limit`, `slope`). softmax 1: the router chooses by the largest sums (+ correction, a
+// bias; null: none) and weighs by the softmax over the chosen; 2: the scores are the softmax over all experts, a group's its
+// largest, and the chosen scores are divided by their sum. out32: as above.
 struct RoutedMlpParams {
     ExecLinear up, down, router;
     const void* correction; i64 c_dtype;
@@ -140,6 +154,7 @@ struct RoutedMlpParams {
     ExecLinear shared_up, shared_down;      // w null: no shared expert
     i64 shared_ff, shared_gate;
     i64 gated, softmax, out32;
+    i64 gate_kind; double limit, shared_limit, slope;
 };
 
 struct ExecOps { i64 n; const ExecOp* ops; };
@@ -163,7 +178,8 @@ enum ExecFn {
     FN_GATED_NORM_ADD, FN_STREAM_CAST, FN_MINGRU_SCAN, FN_LATENT_PREP, FN_HEAD_PRODUCT, FN_GATED_ACT, FN_BIAS_ADD, FN_ATTENTION_LATENT, FN_HEAD_PRODUCT_MMA,
     FN_EMBED_POS, FN_ATTN_PREP, FN_ATTENTION_PLAIN_WIDE, FN_ROUTE, FN_EXPERTS_ROWWISE, FN_ACTIVATION, FN_ADD2_RMSNORM,
     FN_MOE_SORT, FN_MOE_GATHER, FN_MOE_COMBINE, FN_GEMM_GROUPED, FN_ATTENTION_PLAIN_MASKED,
-    FN_ROUTE_SOFTMAX, FN_EXPERTS_GATED_ROWWISE, FN_MOE_COMBINE32, FN_GEMM_GATED, FN_GEMM_GROUPED_GATED, FN_CLAMPED_GATE, FN_COUNT
+    FN_ROUTE_SOFTMAX, FN_EXPERTS_GATED_ROWWISE, FN_MOE_COMBINE32, FN_GEMM_GATED, FN_GEMM_GROUPED_GATED, FN_CLAMPED_GATE,
+    FN_NORM_ADD_NORM, FN_SOFT_CAP, FN_ROUTE_SOFTMAX_ALL, FN_COUNT
 };
 
 struct ExecProgram {

@@ -31,7 +31,7 @@ _SIGNATURES = {
         "cellm_gated_norm_add": [P, P, P, P, L, I, P, P, I, P, I, I, I, F, I, P],
         "cellm_stream_cast": [P, P, L, I, P],
         "cellm_mingru_scan": [P, P, L, I, P, P, I, P, L, P, P, I, I, I, I, I, I, P, P],
-        "cellm_latent_prep": [P, P, P, L, I, P, I, F, P, P, P, I, P, I, I, I, I, I, I, I, I, I, P, I, P, P],
+        "cellm_latent_prep": [P, P, P, P, P, L, I, P, L, I, P, I, I, P, I, F, P, P, P, I, P, I, I, I, I, I, I, I, I, I, P, F, I, I, P, P],
         "cellm_head_product": [P, L, L, P, L, L, P, I, I, I, I, I, P],
         "cellm_gated_act": [P, P, L, P, P, I, I, I, I, I, I, P],
         "cellm_bias_add": [P, P, P, I, I, I, I, P],
@@ -69,7 +69,10 @@ _SIGNATURES = {
         "cellm_xielu": [P, P, L, I, I, P, I, P],
         "cellm_head_gate_mul": [P, P, L, I, I, I, I, P],
         "cellm_route_softmax": [P, P, P, P, L, P, I, I, I, I, F, I, P],
-        "cellm_experts_gated_rowwise": [P, P, P, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
+        "cellm_experts_gated_rowwise": [P, P, P, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, F, F, I, I, P],
+        "cellm_norm_add_norm": [P, P, P, F, P, I, P, P, I, I, F, I, P],
+        "cellm_soft_cap": [P, L, F, P],
+        "cellm_route_softmax_all": [P, P, P, P, L, P, I, I, I, I, I, I, F, I, P],
         "cellm_moe_combine32": [P, P, P, P, P, P, I, I, I, P],
         "cellm_clamped_gate_act": [P, P, L, I, I, F, F, I, P],
         "cellm_embed_norm": [P, P, I, P, P, I, I, I, F, F, P, P],
@@ -106,7 +109,7 @@ _SIGNATURES = {
         "cellm_decay_chunks_supports": [I, I],
     },
     "attention_latent": {
-        "cellm_attention_latent": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P, P, P],
+        "cellm_attention_latent": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P, P, P, P],
         "cellm_attention_latent_supports": [I, I],
         "cellm_head_product_mma": [P, L, L, P, L, L, P, I, I, I, I, P],
     },

@@ -264,6 +264,30 @@ def mingru_scan(proj: torch.Tensor, bz: Optional[torch.Tensor], bx: Optional[tor
     return out
 
 
+def norm_add_norm(x: torch.Tensor, delta: torch.Tensor, w_delta: torch.Tensor, eps_delta: float, w: torch.Tensor, eps: float,
+                  rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x [T, H] float32 += rms_norm(delta) * w_delta (in place; not with `rows`), then the RMS norm of the sum times w in
+    delta's element type, of all rows or of the given ones."""
+    require_cuda(x, delta, w_delta, w, rows)
+    T, H = x.shape
+    if x.dtype != torch.float32 or delta.shape != x.shape or w_delta.dtype != w.dtype:
+        raise ValueError("norm_add_norm: a float32 stream [T, H], an addend of its shape, weights of one element type")
+    n = T if rows is None else rows.numel()
+    y = torch.empty((n, H), dtype=delta.dtype, device=x.device)
+    check(fn(_LIB, "cellm_norm_add_norm")(ptr(x), ptr(delta), ptr(w_delta), float(eps_delta), ptr(w), tag(w), ptr(y), ptr(rows), n, H, float(eps),
+                                          tag(delta), stream_of(x)), "norm_add_norm")
+    return y
+
+
+def soft_cap_(z: torch.Tensor, cap: float) -> torch.Tensor:
+    """z = cap * tanh(z / cap), in place, float32."""
+    require_cuda(z)
+    if z.dtype != torch.float32 or not z.is_contiguous():
+        raise ValueError("soft_cap_: dense float32 values")
+    check(fn(_LIB, "cellm_soft_cap")(ptr(z), z.numel(), float(cap), stream_of(z)), "soft_cap")
+    return z
+
+
 def head_product(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """x [T, heads, K] (any row pitch, head pitch K or more) times per-head matrices w [heads, N, K] -> [T, heads, N];
     `out` may be a view with pitches of its own (last axis dense)."""
@@ -292,11 +316,13 @@ def gated_act(gu: torch.Tensor, bg: Optional[torch.Tensor], bu: Optional[torch.T
 
 def attention_latent(q: torch.Tensor, pool: torch.Tensor, cu_seqlens: torch.Tensor, ctx_lens: torch.Tensor,
                      block_table: torch.Tensor, q_lens, nh: int, dv: int, scale: float, nsplit: int,
-                     err: torch.Tensor, window: int = 0, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     err: torch.Tensor, window: int = 0, sinks: Optional[torch.Tensor] = None,
+                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The tensor-core attention over a latent cache by itself: q [T, nh * kw] bfloat16, pool [pages, 1, page_size, kw];
     every head reads the same rows, a value is a row's first dv entries. `q_lens`: the host's copy of the portions'
     lengths; `nsplit`: pieces the keys are cut into; `window`: 0, or how many of its last rows a token reads; `sinks` [nh]
-    float32: a sink per head in the denominator. Returns [T, nh * dv]."""
+    float32: a sink per head in the denominator; `gate` [T, nh] float32: a head's output times the sigmoid of its number.
+    Returns [T, nh * dv]."""
     require_cuda(q, pool, cu_seqlens, ctx_lens, block_table, err)
     pages, one, page_size, kw = pool.shape
     T = q.shape[0]
@@ -312,5 +338,5 @@ def attention_latent(q: torch.Tensor, pool: torch.Tensor, cu_seqlens: torch.Tens
     check(fn("attention_latent", "cellm_attention_latent")(
         ptr(out), ptr(part_o), ptr(part_ml), ptr(q), ptr(pool), ptr(cu_seqlens), ptr(ctx_lens), ptr(block_table),
         block_table.stride(0), len(q_lens), T, n_tiles, pages, page_size, nh, kw, dv, float(scale), int(nsplit), int(window), ptr(sinks),
-        ptr(err), stream_of(q)), "attention_latent")
+        ptr(gate), ptr(err), stream_of(q)), "attention_latent")
     return out

@@ -54,6 +54,58 @@ class ParallelBlock(Block):
 register_block("parallel", ParallelBlock)
 
 
+class SandwichNormBlock(Block):
+    """A layer with a norm before and a norm behind each sublayer: x += norm1b(mixer(norm1(x))), then
+    x += norm2b(feed_forward(norm2(x))). The layer may have no feed-forward (and then has neither norm2 nor norm2b). The
+    norms behind are RMS norms without groups, in 32-bit; each is formed together with the sum and the next norm.
+
+    params: hidden_size, eps (of the norms behind), feed_forward (default True). weights: mixer_result_norm,
+    feed_forward_result_norm [H]."""
+    graph_safe = True
+
+    @classmethod
+    def weight_specs(cls, params):
+        from .base import TensorSpec
+        H = int(params["hidden_size"])
+        specs = {"mixer_result_norm": TensorSpec((H,), "norm")}
+        if params.get("feed_forward", True):
+            specs["feed_forward_result_norm"] = TensorSpec((H,), "norm")
+        return specs
+
+    def __init__(self, mixer_norm, mixer, feed_forward_norm, feed_forward, params=None, weights=None, dtype=None):
+        from ..config.errors import ConfigError
+        self.mixer_norm, self.mixer = mixer_norm, mixer
+        self.feed_forward_norm, self.feed_forward = feed_forward_norm, feed_forward
+        self.eps, self.dtype = float(params["eps"]), dtype
+        if (feed_forward is None) != (feed_forward_norm is None) or (feed_forward is None) == bool(params.get("feed_forward", True)):
+            raise ConfigError("sandwich_norm: a feed-forward and its two norms come together")
+        self.w1 = weights["mixer_result_norm"].contiguous()
+        self.w2 = weights["feed_forward_result_norm"].contiguous() if feed_forward is not None else None
+
+    def _sublayers(self):
+        yield self.mixer_norm, self.mixer, self.w1
+        if self.feed_forward is not None:
+            yield self.feed_forward_norm, self.feed_forward, self.w2
+
+    def emit(self, emitter) -> None:
+        from ..ops._lib import tag
+        from ..runtime import records as R
+        for norm, part, w in self._sublayers():
+            norm.emit(emitter)
+            part.emit(emitter)
+            emitter.native(R.RESULT_NORM, R.ResultNormParams(w.data_ptr(), tag(w), self.eps), part=self)
+
+    def forward(self, residual: Residual, ctx: StepContext, cache: CacheBinding) -> None:
+        from .. import ops
+        for norm, part, w in self._sublayers():
+            h = norm.forward(residual)
+            m = part.forward(h, ctx, cache) if part is self.mixer else part.forward(h, ctx)
+            ops.gated_norm_add(residual.flush(), m.to(self.dtype).contiguous(), None, None, w, 1, self.eps, want_copy=False)
+
+
+register_block("sandwich_norm", SandwichNormBlock)
+
+
 class TwoNormParallelBlock(Block):
     """A layer whose mixer and feed-forward read the same stream through a norm each, and whose sum joins the stream
     times a constant:  x += mult * (mixer(norm1(x)) + feed_forward(norm2(x))). The layer may have no feed-forward.

@@ -90,7 +90,8 @@ class PairHashEmbedding(Embedding):
 class LinearHead(Head):
     graph_safe = True
 
-    """params: vocab_size, dim. weights: weight [vocab, dim] (the embedding's tensor when the two are tied)."""
+    """params: vocab_size, dim, soft_cap (default none; c: the logits become c tanh(logits / c)). weights: weight [vocab, dim]
+    (the embedding's tensor when the two are tied)."""
 
     @classmethod
     def weight_specs(cls, params):
@@ -99,15 +100,19 @@ class LinearHead(Head):
     def __init__(self, params: dict, weights: dict, dtype: torch.dtype):
         self.linear = Linear(weights["weight"], dtype)
         self.weight = self.linear.weight
+        self.soft_cap = float(params.get("soft_cap") or 0.0)
+        if self.soft_cap < 0.0:
+            raise ConfigError("linear head: soft_cap must be positive")
 
     def emit(self, emitter) -> None:
         from ..runtime import records as R
         if not emitter.fits(self.weight):
             return super().emit(emitter)
-        emitter.native(R.HEAD, R.HeadParams(R.linear(self.weight)), part=self)
+        emitter.native(R.HEAD, R.HeadParams(R.linear(self.weight), self.soft_cap), part=self)
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
-        return self.linear(x, out_dtype=torch.float32)
+        z = self.linear(x, out_dtype=torch.float32)
+        return ops.soft_cap_(z, self.soft_cap) if self.soft_cap else z
 
 
 register_embedding("lookup", TokenEmbedding)

@@ -10,8 +10,9 @@ the query of head h becomes [K_h^T q_h | rotated part], the weighted sum of the 
 and V_h turns it into the head's output. The rotation is a position part of its own (`position`), applied to the last
 rot_dim values of each query head and to the shared key part, in pairs that lie side by side or half a rotation apart.
 Optional: a sliding window (from position i the rows j with 0 <= i - j < window are visible; rows that no later token can read give
-their pages back) and a learned sink per head (one more term exp(sink_h) in the softmax's denominator, with no key and
-no value)."""
+their pages back); a learned sink per head (one more term exp(sink_h) in the softmax's denominator, with no key and
+no value); queries through a latent of their own (q = W_uq rms_norm(W_dq h) in W_q's place); an output gate (head h's output
+times sigmoid(W_g h)_h, formed with the first product and applied where the attention writes the head's sum)."""
 from __future__ import annotations
 
 import torch
@@ -28,18 +29,23 @@ class LatentAttentionMixer(Mixer):
 
     """params: hidden_size, heads, dim, rot_dim, vdim, kv_rank, scale, eps (of the latent's norm),
     position (PartSpec of a rotation over rot_dim values, or None), window (default 0: every earlier row), sinks (default
-    False), out_dtype32 (default False).
-    weights: q [heads*(dim+rot_dim), H], dkv [kv_rank+rot_dim, H], dkv_norm [kv_rank], uk [heads*dim, kv_rank],
-    uv [heads*vdim, kv_rank], o [H, heads*vdim]; sinks [heads]."""
+    False), q_rank (default 0: queries straight from the input), gate (default False).
+    weights: q [heads*(dim+rot_dim), H] (or dq [q_rank, H], dq_norm [q_rank], uq [heads*(dim+rot_dim), q_rank]), dkv [kv_rank+rot_dim, H], dkv_norm [kv_rank], uk [heads*dim, kv_rank],
+    uv [heads*vdim, kv_rank], o [H, heads*vdim]; sinks [heads]; g [heads, H]."""
 
     @classmethod
     def weight_specs(cls, params):
         H, nh, d, r, vd, rank = (params[k] for k in ("hidden_size", "heads", "dim", "rot_dim", "vdim", "kv_rank"))
-        specs = {"q": TensorSpec((nh * (d + r), H), "linear"), "dkv": TensorSpec((rank + r, H), "linear"),
+        qr = int(params.get("q_rank") or 0)
+        specs = {"dq": TensorSpec((qr, H), "linear"), "dq_norm": TensorSpec((qr,), "norm"),
+                 "uq": TensorSpec((nh * (d + r), qr), "linear")} if qr else {"q": TensorSpec((nh * (d + r), H), "linear")}
+        specs |= {"dkv": TensorSpec((rank + r, H), "linear"),
                  "dkv_norm": TensorSpec((rank,), "norm"), "uk": TensorSpec((nh * d, rank), "linear"),
                  "uv": TensorSpec((nh * vd, rank), "linear"), "o": TensorSpec((H, nh * vd), "linear")}
         if params.get("sinks"):
             specs["sinks"] = TensorSpec((nh,), "sink")
+        if params.get("gate"):
+            specs["g"] = TensorSpec((nh, H), "linear")
         return specs
 
     @classmethod
@@ -51,18 +57,26 @@ class LatentAttentionMixer(Mixer):
         self.nh, self.d, self.r = int(params["heads"]), int(params["dim"]), int(params["rot_dim"])
         self.vd, self.rank = int(params["vdim"]), int(params["kv_rank"])
         self.scale, self.eps = float(params["scale"]), float(params["eps"])
-        self.in_proj = Linear(stack_rows(weights["q"], weights["dkv"]), dtype)
+        self.q_rank, self.gate = int(params.get("q_rank") or 0), bool(params.get("gate"))
+        rows = [weights["dq"] if self.q_rank else weights["q"], weights["dkv"]] + ([weights["g"]] if self.gate else [])
+        fill = -sum(int(m.shape[0]) for m in rows) % 8
+        if self.gate and fill:          # the columns behind the gate stay on 16-byte borders
+            rows.append(torch.zeros((fill, self.H), dtype=rows[0].dtype, device=rows[0].device))
+        self.in_proj = Linear(stack_rows(*rows), dtype)
+        self.q_up = Linear(weights["uq"], dtype) if self.q_rank else None
         self.out_proj = Linear(weights["o"], dtype)
         self.c_norm_w = weights["dkv_norm"].contiguous()
+        self.q_norm_w = weights["dq_norm"].to(self.c_norm_w.dtype).contiguous() if self.q_rank else None
         # K_h transposed, [heads, kv_rank, dim]: turns a head's unrotated query into a query against the latent rows
         self.absorb_k = weights["uk"].reshape(self.nh, self.d, self.rank).transpose(1, 2).contiguous()
         self.expand_v = weights["uv"].reshape(self.nh, self.vd, self.rank).contiguous()
         pos: PartSpec | None = params.get("position")
         self.position = part_class("position", pos.kind)(pos.params, self.c_norm_w.device) if pos is not None else None
-        rot = self.position.rotation() if self.position is not None else (0, True, None)
+        rot = self.position.rotation(amplitude=True) if self.position is not None else (0, True, None)
         if rot is None or rot[0] > self.r:
             raise ConfigError("latent_attention: the position encoding must be a rotation over at most rot_dim values")
         self.rot, self.interleaved, self.inv_freq = int(rot[0]), bool(rot[1]), rot[2]
+        self.amplitude = float(getattr(self.position, "amplitude", 1.0)) if self.position is not None else 1.0
         self.window = int(params.get("window") or 0)
         self.sinks = weights["sinks"].to(torch.float32).contiguous() if params.get("sinks") else None
         self.extra = 0
@@ -81,7 +95,7 @@ class LatentAttentionMixer(Mixer):
     def record(self):
         from ..ops._lib import tag
         from ..runtime import records as R
-        ws = (self.in_proj.weight, self.out_proj.weight, self.absorb_k, self.expand_v)
+        ws = [self.in_proj.weight, self.out_proj.weight, self.absorb_k, self.expand_v] + ([self.q_up.weight] if self.q_rank else [])
         if self._record is None and all(w.dtype == self.dtype for w in ws):
             p = R.LatentAttentionParams()
             p.in_proj, p.out_proj = R.linear(self.in_proj.weight), R.linear(self.out_proj.weight)
@@ -90,7 +104,10 @@ class LatentAttentionMixer(Mixer):
             p.c_norm_w, p.c_norm_dtype, p.eps = self.c_norm_w.data_ptr(), tag(self.c_norm_w), self.eps
             p.rot, p.inv_freq, p.extra = self.rot, R.ptr(self.inv_freq), self.extra
             p.interleaved, p.window, p.sinks = int(self.interleaved), self.window, R.ptr(self.sinks)
-            self._record = R.Record(R.LATENT_ATTENTION, p, keep=[self.inv_freq, self.sinks], part=self)
+            p.amplitude, p.q_rank, p.gate = self.amplitude, self.q_rank, int(self.gate)
+            if self.q_rank:
+                p.q_up, p.q_norm_w = R.linear(self.q_up.weight), R.ptr(self.q_norm_w)
+            self._record = R.Record(R.LATENT_ATTENTION, p, keep=[self.inv_freq, self.sinks, self.q_norm_w], part=self)
         return self._record
 
     def emit(self, emitter) -> None:

@@ -8,7 +8,10 @@ that every token runs.
     out = sum_k weight_k * D_k act(U_k h)  +  sigmoid(g . h) * D_s act(U_s h)
 
 Two choices are parameters. `scores` "softmax": the `top` experts with the largest z + bias are chosen and weighed by the
-softmax over the chosen sums (no sigmoid, no groups). `gated`: an expert (the shared one too) is D (silu(G h) * (U h)).
+softmax over the chosen sums (no sigmoid, no groups); "softmax_all": s is the softmax over all experts, a run's score its
+largest, the weights as above. `gated`: an expert (the shared one too) is D (silu(G h) * (U h)), or with the activation
+"clamped" D (g' sigmoid(slope g') (u' + 1)) with g' = min(G h, limit), u' = clamp(U h, -limit, limit) (the shared expert has
+a limit of its own).
 
 The experts' matrices are kept one below the other, so that a kernel reaches expert e by an offset; gate and up rows of
 gated experts lie in blocks of 64, so that the grouped product's epilogue joins the two (widths are padded to multiples of
@@ -31,7 +34,8 @@ class RoutedExperts(FeedForward):
 
     """params: hidden_size, experts, top, ff_dim, activation ("gelu": the exact form), route_scale, groups (default 1),
     keep_groups (default groups), correction (default True), shared_ff (default 0: no shared expert), shared_gate
-    (default True), scores ("sigmoid", the default, or "softmax"), gated (default False), out_dtype32 (default False; gated
+    (default True), scores ("sigmoid", the default, "softmax" or "softmax_all"), limit, shared_limit (default none) and slope
+    (default 1) for gated experts with the activation "clamped", gated (default False), out_dtype32 (default False; gated
     experts only). weights: router [experts, H], correction [experts] (the router's bias under "softmax"), up_<e> [ff, H] and
     down_<e> [H, ff] for every expert e, shared_up [shared_ff, H], shared_down [H, shared_ff], shared_gate [1, H]; and, if
     gated, gate_<e> [ff, H], shared_gate_proj [shared_ff, H]."""
@@ -64,8 +68,14 @@ class RoutedExperts(FeedForward):
         self.keep = int(params.get("keep_groups", self.groups))
         self.route_scale = float(params.get("route_scale", 1.0))
         self.activation = params.get("activation", "gelu")
-        if self.activation not in ACTIVATIONS:
-            raise ConfigError(f"routed_experts: activation {self.activation!r}; known: {sorted(ACTIVATIONS)}")
+        self.clamped = self.activation == "clamped"
+        if self.activation not in ACTIVATIONS and not self.clamped:
+            raise ConfigError(f"routed_experts: activation {self.activation!r}; known: {sorted(ACTIVATIONS) + ['clamped']}")
+        if self.clamped and not params.get("gated"):
+            raise ConfigError("routed_experts: the clamped gate belongs to gated experts")
+        none_is_inf = lambda v: float("inf") if v is None else float(v)
+        self.limit, self.shared_limit = none_is_inf(params.get("limit")), none_is_inf(params.get("shared_limit"))
+        self.slope = float(params.get("slope", 1.0))
         if not 1 <= self.top <= self.E:
             raise ConfigError(f"routed_experts: top {self.top} of {self.E} experts")
         if self.groups < 1 or self.E % self.groups or not 1 <= self.keep <= self.groups:
@@ -74,10 +84,10 @@ class RoutedExperts(FeedForward):
             raise ConfigError(f"routed_experts: {self.keep} groups of {self.E // self.groups} experts cannot give {self.top} choices")
         self.gated, self.out32 = bool(params.get("gated")), bool(params.get("out_dtype32", False))
         scores = params.get("scores", "sigmoid")
-        if scores not in ("sigmoid", "softmax"):
-            raise ConfigError(f"routed_experts: scores {scores!r}; known: 'sigmoid', 'softmax'")
-        self.softmax = scores == "softmax"
-        if self.softmax and self.groups != 1:
+        if scores not in ("sigmoid", "softmax", "softmax_all"):
+            raise ConfigError(f"routed_experts: scores {scores!r}; known: 'sigmoid', 'softmax', 'softmax_all'")
+        self.softmax = ("sigmoid", "softmax", "softmax_all").index(scores)
+        if self.softmax == 1 and self.groups != 1:
             raise ConfigError("routed_experts: groups of experts under softmax scores are not built")
         if self.out32 and not self.gated:
             raise ConfigError("routed_experts: a 32-bit result is built for gated experts")
@@ -112,7 +122,8 @@ class RoutedExperts(FeedForward):
             p.up, p.down, p.router = R.linear(self.up), R.linear(self.down), R.linear(self.router)
             p.correction, p.c_dtype = self.correction.data_ptr(), tag(self.correction)
             p.experts, p.top, p.n_groups, p.keep, p.scale = self.E, self.top, self.groups, self.keep, self.route_scale
-            p.ff, p.act = self.ff, ACTIVATIONS[self.activation]
+            p.ff, p.act = self.ff, ACTIVATIONS.get(self.activation, 0)
+            p.gate_kind, p.limit, p.shared_limit, p.slope = int(self.clamped), self.limit, self.shared_limit, self.slope
             if self.shared_ff:
                 p.shared_up, p.shared_down = R.linear(self.shared_up), R.linear(self.shared_down)
             p.shared_ff, p.shared_gate = self.shared_ff, int(self.has_gate)

@@ -20,7 +20,7 @@ I64, F64, PTR = c_longlong, c_double, c_void_p
 
 # record kinds, in the order of the executor's OpKind
 (EMBED, RMS_NORM, SHORT_CONV, ATTENTION, SWIGLU, HEAD, PYTHON, LINEAR, ATTEND,
- READ_STREAM, GATED_NORM_ADD, MINGRU, LATENT_ATTENTION, GATED_MLP, ROUTED_MLP) = range(15)
+ READ_STREAM, GATED_NORM_ADD, MINGRU, LATENT_ATTENTION, GATED_MLP, ROUTED_MLP, RESULT_NORM) = range(16)
 
 
 class ExecLinear(Structure):
@@ -56,7 +56,7 @@ class SwiGLUParams(Structure):
 
 
 class HeadParams(Structure):
-    _fields_ = [("w", ExecLinear)]
+    _fields_ = [("w", ExecLinear), ("soft_cap", F64)]
 
 
 class PythonParams(Structure):
@@ -83,7 +83,8 @@ class LatentAttentionParams(Structure):
     _fields_ = [("in_proj", ExecLinear), ("out_proj", ExecLinear), ("absorb_k", PTR), ("expand_v", PTR),
                 ("heads", I64), ("dim", I64), ("rot_dim", I64), ("vdim", I64), ("rank", I64), ("scale", F64),
                 ("c_norm_w", PTR), ("c_norm_dtype", I64), ("eps", F64), ("rot", I64), ("inv_freq", PTR), ("extra", I64),
-                ("interleaved", I64), ("window", I64), ("sinks", PTR)]
+                ("interleaved", I64), ("window", I64), ("sinks", PTR), ("amplitude", F64), ("q_up", ExecLinear), ("q_norm_w", PTR),
+                ("q_rank", I64), ("gate", I64)]
 
 
 class GatedMlpParams(Structure):
@@ -95,7 +96,11 @@ class RoutedMlpParams(Structure):
     _fields_ = [("up", ExecLinear), ("down", ExecLinear), ("router", ExecLinear), ("correction", PTR), ("c_dtype", I64),
                 ("experts", I64), ("top", I64), ("n_groups", I64), ("keep", I64), ("scale", F64), ("ff", I64), ("act", I64),
                 ("shared_up", ExecLinear), ("shared_down", ExecLinear), ("shared_ff", I64), ("shared_gate", I64),
-                ("gated", I64), ("softmax", I64), ("out32", I64)]
+                ("gated", I64), ("softmax", I64), ("out32", I64), ("gate_kind", I64), ("limit", F64), ("shared_limit", F64), ("slope", F64)]
+
+
+class ResultNormParams(Structure):
+    _fields_ = [("w", PTR), ("w_dtype", I64), ("eps", F64)]
 
 
 class ExecOps(Structure):
@@ -127,7 +132,8 @@ ENTRY_POINTS = [("kernels_common", "cellm_embed"), ("kernels_common", "cellm_add
                 ("kernels_common", "cellm_attention_plain_masked"), ("kernels_common", "cellm_route_softmax"),
                 ("kernels_common", "cellm_experts_gated_rowwise"), ("kernels_common", "cellm_moe_combine32"),
                 ("gemm_tcgen05", "cellm_gemm_gated_tcgen05"), ("gemm_tcgen05", "cellm_gemm_grouped_gated_tcgen05"),
-                ("kernels_common", "cellm_clamped_gate_act")]
+                ("kernels_common", "cellm_clamped_gate_act"), ("kernels_common", "cellm_norm_add_norm"), ("kernels_common", "cellm_soft_cap"),
+                ("kernels_common", "cellm_route_softmax_all")]
 # libraries a model whose activations are 32-bit never calls into (they need not be compiled for it)
 BF16_ONLY_LIBRARIES = ("attention_decode", "attention_tc", "attention_flash", "gemm_tcgen05", "attention_latent")
 # libraries that only records of these kinds reach (a program without such a record need not have them compiled)
@@ -160,7 +166,7 @@ class ExecStep(Structure):
 # in the order cellm_exec_sizeof() numbers them
 LAYOUT_CHECKED = (ExecLinear, ExecOp, ExecProgram, ExecItem, ExecStep, ExecRegs, EmbedParams, RmsNormParams, ShortConvParams,
                   AttentionParams, SwiGLUParams, HeadParams, PythonParams, ExecOps, LinearParams, ReadStreamParams, GatedNormAddParams,
-                  MinGruParams, LatentAttentionParams, GatedMlpParams, RoutedMlpParams)
+                  MinGruParams, LatentAttentionParams, GatedMlpParams, RoutedMlpParams, ResultNormParams)
 
 
 def ptr(t: Optional[torch.Tensor]):
