@@ -249,7 +249,7 @@ def matrix_bytes(model) -> int:
                 scan(v, depth + 1)
         elif depth < 4 and hasattr(obj, "__dict__"):
             for k, v in vars(obj).items():
-                if k not in ("in_proj_tiled", "q_only", "_record", "_attend", "stacked_view"):
+                if k not in ("in_proj_tiled", "q_only", "_record", "_attend", "stacked_view", "kv_up"):
                     scan(v, depth + 1)
     for blk in model.blocks:
         scan(blk)

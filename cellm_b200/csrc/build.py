@@ -43,6 +43,7 @@ LIBRARIES: dict[str, tuple[str, list[str], list[str]]] = {
     "attention_decode": ("nvcc", ["kernels/attention_decode.cu"], []),
     "attention_tc": ("nvcc", ["kernels/attention_tc.cu"], []),
     "attention_latent": ("nvcc", ["kernels/attention_latent.cu"], []),
+    "attention_expanded": ("nvcc", ["kernels/attention_expanded.cu"], []),
     "decay_chunks": ("nvcc", ["kernels/decay_chunks.cu"], []),
 }
 

@@ -36,7 +36,7 @@ enum { LP_LATENT = 1, LP_QUERY_NORM = 2, LP_QUERIES = 4 };
 
 template <typename TP, typename TA, typename TW>
 __global__ void __launch_bounds__(128)
-latent_prep_kernel(TA* __restrict__ q_plain, TA* __restrict__ q_full, const TP* __restrict__ q_rows, long long q_ld,
+latent_prep_kernel(TA* __restrict__ q_plain, TA* __restrict__ q_turned, long long turned_hs, const TP* __restrict__ q_rows, long long q_ld,
                    TA* __restrict__ cq, const TP* __restrict__ cq_rows, int q_rank, const TW* __restrict__ cq_norm_w,
                    float* __restrict__ gate_out, const TP* __restrict__ gate_rows, const TP* __restrict__ down_rows, long long ld,
                    const TW* __restrict__ c_norm_w, float eps, const int* __restrict__ positions,
@@ -124,8 +124,7 @@ latent_prep_kernel(TA* __restrict__ q_plain, TA* __restrict__ q_full, const TP* 
         --role;
     }
     // the queries, a run of heads a block (so that a token's work is spread over several blocks when the tokens are few):
-    // the unrotated part head by head where a gathered copy is wanted; the rotated part turned, behind the kv_rank places
-    // of its head; the heads' gates
+    // the unrotated part head by head where a gathered copy is wanted; the rotated part turned; the heads' gates
     __syncthreads();
     pdl_wait();
     const TP* row = q_rows + (size_t)t * q_ld;
@@ -139,7 +138,7 @@ latent_prep_kernel(TA* __restrict__ q_plain, TA* __restrict__ q_full, const TP* 
         }
     for (int i = h_lo * rot_dim + threadIdx.x; i < h_hi * rot_dim; i += blockDim.x) {
         const int h = i / rot_dim, d = i - h * rot_dim;
-        q_full[((size_t)t * heads + h) * kw + rank + d] = from_float<TA>(turned(row + h * qw + dim, d));
+        q_turned[((size_t)t * heads + h) * turned_hs + d] = from_float<TA>(turned(row + h * qw + dim, d));
     }
     if (gate_out && !(roles & LP_QUERY_NORM))
         for (int h = h_lo + threadIdx.x; h < h_hi; h += blockDim.x) gate_out[(size_t)t * heads + h] = to_float(gate_rows[(size_t)t * ld + h]);
@@ -151,11 +150,11 @@ latent_prep_kernel(TA* __restrict__ q_plain, TA* __restrict__ q_full, const TP* 
 //   1  the latent normed and the key part turned into the cache (pool: one layer's rows; null: another's cache is read)
 //   2  the queries' latent normed into cq [T, q_rank] (with q_rank)
 //   4  of queries q_rows [T, q_ld] (heads of dim + rot_dim): the unrotated parts gathered into q_plain [T, heads * dim]
-//      (null: not wanted), the rotated parts turned into the last rot_dim values of each head of q_full [T, heads, rank + rot_dim]
+//      (null: not wanted), the rotated parts turned into q_turned [T, heads, rot_dim] whose heads lie turned_hs values apart
 // and the gates as 32-bit numbers into gate_out [T, heads] (by 2 where it is asked for, else by 4). rot: how many of the
 // rot_dim values turn (even), in pairs (2p, 2p + 1) if `interleaved`, else (p, p + rot / 2); inv_freq: [rot / 2] pairs of
 // floats (frequency, remainder); cos and sin are multiplied by `amplitude`.
-CELLM_API int cellm_latent_prep(void* q_plain, void* q_full, void* cq, float* gate_out, const void* proj, long long ld, int proj_dtype,
+CELLM_API int cellm_latent_prep(void* q_plain, void* q_turned, long long turned_hs, void* cq, float* gate_out, const void* proj, long long ld, int proj_dtype,
                                 const void* q_rows, long long q_ld, int q_rank, const void* cq_norm_w, int down_col, int gate_col,
                                 const void* c_norm_w, int w_dtype, float eps, const int* positions, const int* seq_of_token,
                                 const int* block_table, int bt_stride, void* pool, int num_pages, int page_size, int T, int heads, int dim,
@@ -166,7 +165,7 @@ CELLM_API int cellm_latent_prep(void* q_plain, void* q_full, void* cq, float* ga
     if (!(roles & 7) || (roles & ~7)) return CELLM_ERR_ARG;
     if ((roles & LP_LATENT) && (down_col < 0 || ld < (long long)down_col + rank + rot_dim || !c_norm_w)) return CELLM_ERR_SIZE;
     if ((roles & LP_QUERY_NORM) && (q_rank < 1 || ld < q_rank || !cq || !cq_norm_w)) return CELLM_ERR_SIZE;
-    if ((roles & LP_QUERIES) && (!q_rows || q_ld < (long long)heads * (dim + rot_dim))) return CELLM_ERR_SIZE;
+    if ((roles & LP_QUERIES) && (!q_rows || q_ld < (long long)heads * (dim + rot_dim) || (rot_dim && (!q_turned || turned_hs < rot_dim)))) return CELLM_ERR_SIZE;
     if (gate_out && (gate_col < 0 || ld < (long long)gate_col + heads)) return CELLM_ERR_SIZE;
     if (rot > 0 && !inv_freq) return CELLM_ERR_ARG;
     if (pool && (!block_table || page_size <= 0)) return CELLM_ERR_ARG;
@@ -175,7 +174,7 @@ CELLM_API int cellm_latent_prep(void* q_plain, void* q_full, void* cq, float* ga
     const int qblocks = !(roles & LP_QUERIES) ? 0 : (T >= 256 ? 1 : (heads < 8 ? heads : 8));
     const dim3 grid((unsigned)T, (unsigned)(qblocks + ((roles & LP_LATENT) ? 1 : 0) + ((roles & LP_QUERY_NORM) ? 1 : 0)));
 #define LAUNCH(TP, TA, TW)                                                                                              \
-    CELLM_RUN((latent_prep_kernel<TP, TA, TW>), grid, 128, smem, stream, (TA*)q_plain, (TA*)q_full, (const TP*)q_rows, q_ld, (TA*)cq,  \
+    CELLM_RUN((latent_prep_kernel<TP, TA, TW>), grid, 128, smem, stream, (TA*)q_plain, (TA*)q_turned, turned_hs, (const TP*)q_rows, q_ld, (TA*)cq, \
               (const TP*)proj, q_rank, (const TW*)cq_norm_w, gate_out, gate_col >= 0 ? (const TP*)proj + gate_col : nullptr,          \
               (const TP*)proj + down_col, ld, (const TW*)c_norm_w, eps, positions, seq_of_token, block_table, bt_stride, (TA*)pool,   \
               num_pages, page_size, heads, dim, rot_dim, rank, rot, interleaved, inv_freq, amplitude, roles, err)

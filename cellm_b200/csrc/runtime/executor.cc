@@ -45,13 +45,18 @@ typedef int (*GatedNormAddFn)(P x, CP m, CP m_bias, CP gate, i64 gate_ld, int ga
 typedef int (*StreamCastFn)(P y, CP x, i64 n, int act_tag, P stream);
 typedef int (*MinGruScanFn)(P out, CP proj, i64 ld, int proj_tag, CP bz, CP bx, int w_tag, P state, i64 slot_stride, CP slot_ids, CP cu,
                             int T, int B, int W, int n_slots, int max_q_len, int act_tag, P err, P stream);
-typedef int (*LatentPrepFn)(P q_plain, P q_full, P cq, P gate_out, CP proj, i64 ld, int proj_tag, CP q_rows, i64 q_ld, int q_rank, CP cq_norm_w,
+typedef int (*LatentPrepFn)(P q_plain, P q_turned, i64 turned_hs, P cq, P gate_out, CP proj, i64 ld, int proj_tag, CP q_rows, i64 q_ld, int q_rank, CP cq_norm_w,
                             int down_col, int gate_col, CP c_norm_w, int w_tag, float eps, CP positions, CP seq,
                             CP bt, int bt_stride, P pool, int pages, int page_size, int T, int heads, int dim, int rot_dim, int rank,
                             int rot, int interleaved, CP inv_freq, float amplitude, int roles, int act_tag, P err, P stream);
 typedef int (*AttentionPlainMaskedFn)(P out, CP q, CP kp, CP vp, CP positions, CP seq, CP bt, int bt_stride, int pages, int page_size,
                                       int T, int nh, int nkv, int hd, int hdv, int v_row, float scale, int window, int keep_first,
                                       CP sinks, float fixed_sink, int has_fixed_sink, CP gate, i64 gate_ld, int tag, P err, P stream);
+typedef int (*LatentRowsFn)(P rows, CP pool, CP cu, CP ctx, CP bt, int bt_stride, int B, int n_rows, int pages, int page_size, int window, int kw,
+                            P err, P stream);
+typedef int (*AttentionExpandedFn)(P out, CP q, i64 q_ld, CP q_rot, CP rows, CP kv, CP cu, CP ctx, int B, int T, int n_tiles, int n_rows, int heads,
+                                   int dim, int rot_dim, int vdim, int rank, float scale, int window, CP sinks, CP gate, P err, P stream);
+typedef int (*ExpandedSupportsFn)(int heads, int dim, int rot_dim, int vdim, int rank);
 typedef int (*HeadProductFn)(P out, i64 ldo, i64 out_hs, CP in, i64 ldi, i64 in_hs, CP w, int T, int heads, int N, int K, int tag, P stream);
 typedef int (*GatedActFn)(P h, CP gu, i64 ld, CP bg, CP bu, int w_tag, int T, int ff, int act, int tag, int gu_tag, P stream);
 typedef int (*BiasAddFn)(P out, CP in, CP b, int w_tag, int T, int N, int tag, P stream);
@@ -400,6 +405,7 @@ struct Run {
     void routed_mlp(const RoutedMlpParams& L, const void* x, void* out);
     void mingru(const MinGruParams& L, const ExecItem& it, const void* x, void* out);
     void latent_attention(const LatentAttentionParams& L, const ExecItem& it, const void* x, void* out);
+    i64 expanded_rows(const LatentAttentionParams& L, const ExecItem& it);
     void short_conv(const ShortConvParams& L, const ExecItem& it, const void* x, void* out);
     void attention(const AttentionParams& L, const ExecItem& it, const void* x, void* out);
     void* attend(const AttentionParams& L, const ExecItem& it, const void* q, void* o = nullptr);
@@ -895,16 +901,40 @@ void Run::mingru(const MinGruParams& L, const ExecItem& it, const void* x, void*
     product(out, y, L.out_proj, T, W, act);
 }
 
+// Whether the step's portions of a latent layer attend to expanded keys and values: the number of cached rows they can see
+// (0: no). bfloat16, sizes that the kernel takes, tokens that fill its tiles of 256, tiles enough for the SMs, and rows few
+// enough: a row costs rank * heads * (dim + vdim) multiply-adds on tcgen05, which some twenty tokens' scores and sums over
+// the row itself cost on the other path, and its expansion takes heads * (dim + vdim) values of the step's memory.
+i64 Run::expanded_rows(const LatentAttentionParams& L, const ExecItem& it) {
+    if (!p.latent_expand || act != EXEC_BF16 || !L.kv_up.w || !s.host_ctx_lens || !it.k || !(L.scale > 0)) return 0;
+    const i64 qw = L.dim + L.rot_dim, kw = L.rank + L.rot_dim, q_ld = L.q_rank ? L.q_up.N : L.in_proj.N;
+    if (q_ld % 8 || qw % 8 || kw % 8 || s.max_q_len < 2) return 0;
+    i64 tiles = 0, rows = 0;
+    for (i64 b = 0; b < s.B; ++b) {
+        if (s.q_lens[b] <= 0) continue;
+        tiles += ceil_div(s.q_lens[b], 256);
+        const i64 ctx = s.host_ctx_lens[b], first = L.window ? std::max<i64>(0, ctx - L.window + 1) : 0;
+        rows += ctx + s.q_lens[b] - first;
+    }
+    const i64 min_ctas = p.tc_min_ctas < 0 ? p.sms / 8 : p.tc_min_ctas;
+    if (tiles * L.heads < min_ctas || (double)s.T < p.tc_min_fill * (double)(tiles * 256) || rows > 16 * s.T) return 0;
+    if (rows * L.kv_up.N > (i64)1 << 30) return 0;
+    if (!reinterpret_cast<ExpandedSupportsFn>(p.fns[FN_EXPANDED_SUPPORTS])) return 0;
+    return reinterpret_cast<ExpandedSupportsFn>(p.fns[FN_EXPANDED_SUPPORTS])((int)L.heads, (int)L.dim, (int)L.rot_dim, (int)L.vdim, (int)L.rank) ? rows : 0;
+}
+
 void Run::latent_attention(const LatentAttentionParams& L, const ExecItem& it, const void* x, void* out) {
     const i64 T = s.T, H = p.H, nh = L.heads, qw = L.dim + L.rot_dim, kw = L.rank + L.rot_dim, e = elt(act);
     void* proj = linear(x, L.in_proj, T, H, act);
     if (L.extra) gate_at = static_cast<const char*>(proj) + (L.in_proj.N - L.extra) * e, gate_ld = L.in_proj.N, gate_dtype = act;
     const i64 down_col = L.q_rank ? L.q_rank : nh * qw, gate_col = L.gate ? down_col + kw : -1;
-    void* q_full = arena.take(T * nh * kw * e);
+    const i64 rows = expanded_rows(L, it);      // > 0: the portions attend to keys and values expanded from that many rows
+    void* q_full = rows ? nullptr : arena.take(T * nh * kw * e);
+    void* q_turned = rows ? (L.rot_dim ? arena.take(T * nh * L.rot_dim * e) : nullptr) : static_cast<char*>(q_full) + L.rank * e;
     float* out_gate = L.gate ? static_cast<float*>(arena.take(T * nh * 4)) : nullptr;
     enum { LATENT = 1, QUERY_NORM = 2, QUERIES = 4 };
     auto prep = [&](int roles, void* q_plain, void* cq, float* gate_out, const void* q_rows, i64 q_ld) {
-        LAUNCH(fn<LatentPrepFn>(FN_LATENT_PREP)(q_plain, q_full, cq, gate_out, proj, L.in_proj.N, (int)act, q_rows, q_ld, (int)L.q_rank, L.q_norm_w,
+        LAUNCH(fn<LatentPrepFn>(FN_LATENT_PREP)(q_plain, q_turned, rows ? L.rot_dim : kw, cq, gate_out, proj, L.in_proj.N, (int)act, q_rows, q_ld, (int)L.q_rank, L.q_norm_w,
                                             (int)down_col, (int)gate_col, L.c_norm_w, (int)L.c_norm_dtype, (float)L.eps, s.positions,
                                             s.seq_of_token, it.block_table, (int)it.bt_stride, it.writes ? it.k : nullptr, (int)it.num_pages,
                                             (int)it.page_size, (int)T, (int)nh, (int)L.dim, (int)L.rot_dim, (int)L.rank, (int)L.rot,
@@ -926,6 +956,23 @@ void Run::latent_attention(const LatentAttentionParams& L, const ExecItem& it, c
     const bool queries = q_plain || L.rot_dim || (L.gate && !L.q_rank);
     if (!L.q_rank) prep(LATENT | (queries ? QUERIES : 0), q_plain, nullptr, out_gate, q_rows, q_ld);
     else if (queries) prep(QUERIES, q_plain, nullptr, nullptr, q_rows, q_ld);
+    if (rows) {         // (in_place holds: expanded_rows asks for the alignment)
+        void* dense = arena.take(rows * kw * e);
+        LAUNCH(fn<LatentRowsFn>(FN_LATENT_ROWS)(dense, it.k, s.cu_seqlens, s.ctx_lens, it.block_table, (int)it.bt_stride, (int)s.B, (int)rows,
+                                            (int)it.num_pages, (int)it.page_size, (int)L.window, (int)kw, s.err, s.stream),
+               "latent_rows");
+        void* kv = arena.take(rows * L.kv_up.N * e);
+        product(kv, dense, L.kv_up, rows, kw, act);
+        i64 n_tiles = 0;
+        for (i64 b = 0; b < s.B; ++b) n_tiles += ceil_div(s.q_lens[b], 256);
+        void* o = arena.take(T * nh * L.vdim * e);
+        LAUNCH(fn<AttentionExpandedFn>(FN_ATTENTION_EXPANDED)(o, q_rows, q_ld, q_turned, dense, kv, s.cu_seqlens, s.ctx_lens, (int)s.B, (int)T, (int)n_tiles,
+                                                          (int)rows, (int)nh, (int)L.dim, (int)L.rot_dim, (int)L.vdim, (int)L.rank,
+                                                          (float)L.scale, (int)L.window, L.sinks, out_gate, s.err, s.stream),
+               "attention_expanded");
+        product(out, o, L.out_proj, T, nh * L.vdim, act);
+        return;
+    }
     // a head's query against the cached rows: [K_h^T q_h | rotated part]
     if (in_place) head_products(q_full, nh * kw, kw, q_rows, q_ld, qw, L.absorb_k, T, nh, L.rank, L.dim);
     else head_products(q_full, nh * kw, kw, q_plain, nh * L.dim, L.dim, L.absorb_k, T, nh, L.rank, L.dim);

@@ -128,6 +128,7 @@ struct LatentAttentionParams {
     ExecLinear q_up;
     const void* q_norm_w; i64 q_rank;   // of c_norm_w's element type, with its eps
     i64 gate;
+    ExecLinear kv_up;           // all heads' key matrices, then all heads' value matrices [heads * (dim + vdim), rank]; w null: never expanded
 };
 // down . (act(gate . y + bg) * (up . y + bu)) + bd; act 0 silu, 1 gelu (tanh form); the biases may be null.
 // act 2, the clamped gate (no biases): g' sigmoid(slope g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit).
@@ -179,7 +180,7 @@ enum ExecFn {
     FN_EMBED_POS, FN_ATTN_PREP, FN_ATTENTION_PLAIN_WIDE, FN_ROUTE, FN_EXPERTS_ROWWISE, FN_ACTIVATION, FN_ADD2_RMSNORM,
     FN_MOE_SORT, FN_MOE_GATHER, FN_MOE_COMBINE, FN_GEMM_GROUPED, FN_ATTENTION_PLAIN_MASKED,
     FN_ROUTE_SOFTMAX, FN_EXPERTS_GATED_ROWWISE, FN_MOE_COMBINE32, FN_GEMM_GATED, FN_GEMM_GROUPED_GATED, FN_CLAMPED_GATE,
-    FN_NORM_ADD_NORM, FN_SOFT_CAP, FN_ROUTE_SOFTMAX_ALL, FN_COUNT
+    FN_NORM_ADD_NORM, FN_SOFT_CAP, FN_ROUTE_SOFTMAX_ALL, FN_LATENT_ROWS, FN_ATTENTION_EXPANDED, FN_EXPANDED_SUPPORTS, FN_COUNT
 };
 
 struct ExecProgram {
@@ -187,6 +188,7 @@ struct ExecProgram {
     i64 sms, static_flag, max_counters;
     i64 fused_conv, fused_rope;     // decode steps: in_proj + convolution, q/k/v product + norm + rotation as one kernel each
     i64 latent_tc;                  // latent attention on the tensor cores where its sizes allow (0: the plain kernel always)
+    i64 latent_expand;              // prompt portions of latent layers over keys and values expanded once a step, where that pays
     i64 grouped_min_tokens;         // routed experts run as grouped tensor-core products from this many tokens (bfloat16)
     i64 tc_min_ctas;                // prompt attention on tcgen05 from this many CTAs (< 0: an eighth of the SMs)
     double tc_min_fill;             // and this share of its tiles' rows in use
@@ -208,6 +210,7 @@ struct ExecStep {
     i64 T, B, R, max_q_len, max_total_len, n_order;   // n_order: run only the first items (<= program's)
     const void *ids, *positions, *seq_of_token, *cu_seqlens, *ctx_lens, *slot_ids, *rows;
     const i64* q_lens;          // host copy, [B]
+    const i64* host_ctx_lens;   // host copy, [B] (null: not known; nothing is expanded then)
     const ExecItem* items;      // [n_order]
     void* arena; i64 arena_bytes;
     void* logits;               // [R, V] float, or null when R = 0

@@ -3,7 +3,7 @@ arguments, allocates its output with torch and launches on the current stream.""
 from .basic import (embed, embed_norm, add_rmsnorm, residual_add, swiglu, short_conv, qk_norm_rope,
                     attention_plain, argmax, sample, upload, take_pending_tokens, keep_last_tokens,
                     stream_cast, gated_norm_add, mingru_scan, head_product, gated_act, attention_latent,
-                    norm_add_norm, soft_cap_)
+                    norm_add_norm, soft_cap_, latent_rows, attention_expanded)
 from .gemm import gemm, gemm_act, gemm_plain
 from .recurrent import (embed_pairs, norm_pair, scaled_add2, pair_norm_mean, conv_state_update, sink_attn_prep, attention_plain_sink, attention_flash_sink,
                         hgrn2_scan, delta_prep, delta_scan, head_norm_gate, activation, attention_plain_masked, attention_flash_masked, gdelta_prep, gdelta_scan,
@@ -21,4 +21,4 @@ __all__ = ["embed", "add_rmsnorm", "residual_add", "swiglu", "short_conv", "qk_n
            "weighted_sum2", "xielu", "head_gate_mul", "post_norm", "embed_norm", "turned_attn_prep", "attention_plain_chunked", "attention_flash_chunked",
            "attention_tc_chunked", "rotate_heads", "decay_scan", "ssd_prep", "gated_group_norm", "head_norm_silu",
            "stream_cast", "gated_norm_add", "mingru_scan", "head_product", "gated_act", "attention_latent",
-           "norm_add_norm", "soft_cap_"]
+           "norm_add_norm", "soft_cap_", "latent_rows", "attention_expanded"]

@@ -31,7 +31,7 @@ _SIGNATURES = {
         "cellm_gated_norm_add": [P, P, P, P, L, I, P, P, I, P, I, I, I, F, I, P],
         "cellm_stream_cast": [P, P, L, I, P],
         "cellm_mingru_scan": [P, P, L, I, P, P, I, P, L, P, P, I, I, I, I, I, I, P, P],
-        "cellm_latent_prep": [P, P, P, P, P, L, I, P, L, I, P, I, I, P, I, F, P, P, P, I, P, I, I, I, I, I, I, I, I, I, P, F, I, I, P, P],
+        "cellm_latent_prep": [P, P, L, P, P, P, L, I, P, L, I, P, I, I, P, I, F, P, P, P, I, P, I, I, I, I, I, I, I, I, I, P, F, I, I, P, P],
         "cellm_head_product": [P, L, L, P, L, L, P, I, I, I, I, I, P],
         "cellm_gated_act": [P, P, L, P, P, I, I, I, I, I, I, P],
         "cellm_bias_add": [P, P, P, I, I, I, I, P],
@@ -107,6 +107,11 @@ _SIGNATURES = {
     "decay_chunks": {
         "cellm_decay_chunks": [P, P, L, I, P, L, P, L, P, L, P, L, P, L, P, P, I, I, I, I, I, I, I, P, P, P, P],
         "cellm_decay_chunks_supports": [I, I],
+    },
+    "attention_expanded": {
+        "cellm_latent_rows": [P, P, P, P, P, I, I, I, I, I, I, I, P, P],
+        "cellm_attention_expanded": [P, P, L, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, P, P, P],
+        "cellm_attention_expanded_supports": [I, I, I, I, I],
     },
     "attention_latent": {
         "cellm_attention_latent": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P, P, P, P],

@@ -264,6 +264,39 @@ def mingru_scan(proj: torch.Tensor, bz: Optional[torch.Tensor], bx: Optional[tor
     return out
 
 
+def latent_rows(pool: torch.Tensor, cu_seqlens: torch.Tensor, ctx_lens: torch.Tensor, block_table: torch.Tensor, n_rows: int, err: torch.Tensor,
+                window: int = 0) -> torch.Tensor:
+    """The cached rows [n_rows, kw] that the requests' new tokens can see, request after request, out of a pool [pages, 1, page_size,
+    kw] of bfloat16 rows: all ctx + new ones, or with a window those from max(0, ctx - window + 1) on."""
+    require_cuda(pool, cu_seqlens, ctx_lens, block_table, err)
+    pages, one, page_size, kw = pool.shape
+    if one != 1 or pool.dtype != torch.bfloat16:
+        raise ValueError("latent_rows: a bfloat16 pool [pages, 1, page_size, kw]")
+    rows = torch.empty((n_rows, kw), dtype=pool.dtype, device=pool.device)
+    check(fn("attention_expanded", "cellm_latent_rows")(ptr(rows), ptr(pool), ptr(cu_seqlens), ptr(ctx_lens), ptr(block_table), block_table.stride(0),
+                                                        ctx_lens.numel(), n_rows, pages, page_size, int(window), kw, ptr(err), stream_of(pool)),
+          "latent_rows")
+    return rows
+
+
+def attention_expanded(q: torch.Tensor, q_rot: Optional[torch.Tensor], rows: torch.Tensor, kv: torch.Tensor, cu_seqlens: torch.Tensor,
+                       ctx_lens: torch.Tensor, q_lens, heads: int, dim: int, rot_dim: int, vdim: int, scale: float, err: torch.Tensor,
+                       window: int = 0, sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The tcgen05 attention over expanded heads by itself: q [T, heads * (dim + rot_dim)] (its unrotated parts are read), q_rot [T,
+    heads * rot_dim], rows [n, rank + rot_dim] as `latent_rows` gives them, kv [n, heads * dim + heads * vdim]. `q_lens`: the
+    host's copy of the portions' lengths; `sinks` [heads], `gate` [T, heads] float32. Returns [T, heads * vdim]."""
+    require_cuda(q, q_rot, rows, kv, cu_seqlens, ctx_lens, err)
+    T = q.shape[0]
+    if any(t is not None and t.dtype != torch.bfloat16 for t in (q, q_rot, rows, kv)) or kv.shape != (rows.shape[0], heads * (dim + vdim)):
+        raise ValueError("attention_expanded: bfloat16 operands, kv [rows, heads * (dim + vdim)]")
+    out = torch.empty((T, heads * vdim), dtype=q.dtype, device=q.device)
+    n_tiles = sum((int(n) + 255) // 256 for n in q_lens)
+    check(fn("attention_expanded", "cellm_attention_expanded")(
+        ptr(out), ptr(q), q.stride(0), ptr(q_rot), ptr(rows), ptr(kv), ptr(cu_seqlens), ptr(ctx_lens), len(q_lens), T, n_tiles, rows.shape[0], heads,
+        dim, rot_dim, vdim, rows.shape[1] - rot_dim, float(scale), int(window), ptr(sinks), ptr(gate), ptr(err), stream_of(q)), "attention_expanded")
+    return out
+
+
 def norm_add_norm(x: torch.Tensor, delta: torch.Tensor, w_delta: torch.Tensor, eps_delta: float, w: torch.Tensor, eps: float,
                   rows: Optional[torch.Tensor] = None) -> torch.Tensor:
     """x [T, H] float32 += rms_norm(delta) * w_delta (in place; not with `rows`), then the RMS norm of the sum times w in

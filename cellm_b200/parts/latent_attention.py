@@ -7,7 +7,8 @@ row is cached.
 
 Since q_h . (K_h c) = (K_h^T q_h) . c, the attention runs over the cached rows themselves with one key/value "head":
 the query of head h becomes [K_h^T q_h | rotated part], the weighted sum of the rows' first kv_rank values is formed,
-and V_h turns it into the head's output. The rotation is a position part of its own (`position`), applied to the last
+and V_h turns it into the head's output. Portions of many tokens take the equations as they stand instead: keys and values
+of all heads are made from the rows that the portion sees, once a step. The rotation is a position part of its own (`position`), applied to the last
 rot_dim values of each query head and to the shared key part, in pairs that lie side by side or half a rotation apart.
 Optional: a sliding window (from position i the rows j with 0 <= i - j < window are visible; rows that no later token can read give
 their pages back); a learned sink per head (one more term exp(sink_h) in the softmax's denominator, with no key and
@@ -70,6 +71,8 @@ class LatentAttentionMixer(Mixer):
         # K_h transposed, [heads, kv_rank, dim]: turns a head's unrotated query into a query against the latent rows
         self.absorb_k = weights["uk"].reshape(self.nh, self.d, self.rank).transpose(1, 2).contiguous()
         self.expand_v = weights["uv"].reshape(self.nh, self.vd, self.rank).contiguous()
+        # both as one matrix, for prompt portions whose keys and values are expanded once a step
+        self.kv_up = stack_rows(weights["uk"], weights["uv"]) if dtype == torch.bfloat16 and weights["uk"].dtype == weights["uv"].dtype == dtype else None
         pos: PartSpec | None = params.get("position")
         self.position = part_class("position", pos.kind)(pos.params, self.c_norm_w.device) if pos is not None else None
         rot = self.position.rotation(amplitude=True) if self.position is not None else (0, True, None)
@@ -105,6 +108,8 @@ class LatentAttentionMixer(Mixer):
             p.rot, p.inv_freq, p.extra = self.rot, R.ptr(self.inv_freq), self.extra
             p.interleaved, p.window, p.sinks = int(self.interleaved), self.window, R.ptr(self.sinks)
             p.amplitude, p.q_rank, p.gate = self.amplitude, self.q_rank, int(self.gate)
+            if self.kv_up is not None:
+                p.kv_up = R.linear(self.kv_up)
             if self.q_rank:
                 p.q_up, p.q_norm_w = R.linear(self.q_up.weight), R.ptr(self.q_norm_w)
             self._record = R.Record(R.LATENT_ATTENTION, p, keep=[self.inv_freq, self.sinks, self.q_norm_w], part=self)

@@ -29,9 +29,10 @@ from . import records as R
 # and the q/k/v product + head norms + rotation + cache write, as one kernel each. attention_tc_*: prompt attention
 # goes to the tcgen05 kernel from this many CTAs (None: an eighth of the SMs) and this share of its tiles' rows in use.
 # latent_tc: latent attention runs on the tensor cores where its sizes allow (off: the plain kernel, as in 32-bit).
+# latent_expand: prompt portions of latent layers attend to keys and values expanded once a step (tcgen05) where that pays.
 # grouped_experts_min_tokens: routed experts run as grouped tensor-core products from this many tokens of a step (fewer
 # tokens walk their experts row by row).
-OPTIONS = {"fused_conv": True, "fused_rope": True, "attention_tc_min_ctas": None, "attention_tc_min_fill": 0.5, "latent_tc": True,
+OPTIONS = {"fused_conv": True, "fused_rope": True, "attention_tc_min_ctas": None, "attention_tc_min_fill": 0.5, "latent_tc": True, "latent_expand": True,
            "grouped_experts_min_tokens": 17}
 
 _bound = False
@@ -185,7 +186,7 @@ class Program:
     def _options(self) -> None:
         p = self.program
         p.fused_conv, p.fused_rope = int(OPTIONS["fused_conv"]), int(OPTIONS["fused_rope"])
-        p.latent_tc = int(OPTIONS["latent_tc"])
+        p.latent_tc, p.latent_expand = int(OPTIONS["latent_tc"]), int(OPTIONS["latent_expand"])
         p.grouped_min_tokens = int(OPTIONS["grouped_experts_min_tokens"])
         p.tc_min_ctas = -1 if OPTIONS["attention_tc_min_ctas"] is None else int(OPTIONS["attention_tc_min_ctas"])
         p.tc_min_fill = float(OPTIONS["attention_tc_min_fill"])
@@ -207,11 +208,14 @@ class Program:
         s.cu_seqlens, s.ctx_lens, s.slot_ids = ctx.cu_seqlens.data_ptr(), ctx.ctx_lens.data_ptr(), ctx.slot_ids.data_ptr()
         s.rows = logit_rows.data_ptr() if nrows else None
         q_lens = (R.I64 * ctx.B)(*ctx.q_lens)
+        ctx_lens = (R.I64 * ctx.B)(*ctx.ctx_lens_host) if ctx.ctx_lens_host else None
         s.q_lens, s.items = q_lens, items
+        if ctx_lens is not None:
+            s.host_ctx_lens = ctx_lens
         s.err = ctx.err.data_ptr()
         s.stream = klib.stream_of(ctx.err) if stream is None else stream
         s.counters = counters(self.device).data_ptr()
-        return s, (items, q_lens)
+        return s, (items, q_lens, ctx_lens)
 
     def _buffers(self, s, need) -> torch.Tensor:
         arena = self._grow("_arena", need[0] + 256, torch.uint8)

@@ -84,7 +84,7 @@ class LatentAttentionParams(Structure):
                 ("heads", I64), ("dim", I64), ("rot_dim", I64), ("vdim", I64), ("rank", I64), ("scale", F64),
                 ("c_norm_w", PTR), ("c_norm_dtype", I64), ("eps", F64), ("rot", I64), ("inv_freq", PTR), ("extra", I64),
                 ("interleaved", I64), ("window", I64), ("sinks", PTR), ("amplitude", F64), ("q_up", ExecLinear), ("q_norm_w", PTR),
-                ("q_rank", I64), ("gate", I64)]
+                ("q_rank", I64), ("gate", I64), ("kv_up", ExecLinear)]
 
 
 class GatedMlpParams(Structure):
@@ -133,18 +133,19 @@ ENTRY_POINTS = [("kernels_common", "cellm_embed"), ("kernels_common", "cellm_add
                 ("kernels_common", "cellm_experts_gated_rowwise"), ("kernels_common", "cellm_moe_combine32"),
                 ("gemm_tcgen05", "cellm_gemm_gated_tcgen05"), ("gemm_tcgen05", "cellm_gemm_grouped_gated_tcgen05"),
                 ("kernels_common", "cellm_clamped_gate_act"), ("kernels_common", "cellm_norm_add_norm"), ("kernels_common", "cellm_soft_cap"),
-                ("kernels_common", "cellm_route_softmax_all")]
+                ("kernels_common", "cellm_route_softmax_all"), ("attention_expanded", "cellm_latent_rows"),
+                ("attention_expanded", "cellm_attention_expanded"), ("attention_expanded", "cellm_attention_expanded_supports")]
 # libraries a model whose activations are 32-bit never calls into (they need not be compiled for it)
-BF16_ONLY_LIBRARIES = ("attention_decode", "attention_tc", "attention_flash", "gemm_tcgen05", "attention_latent")
+BF16_ONLY_LIBRARIES = ("attention_decode", "attention_tc", "attention_flash", "gemm_tcgen05", "attention_latent", "attention_expanded")
 # libraries that only records of these kinds reach (a program without such a record need not have them compiled)
 LIBRARY_USERS = {"attention_decode": (ATTENTION, ATTEND), "attention_tc": (ATTENTION, ATTEND), "attention_flash": (ATTENTION, ATTEND),
-                 "attention_latent": (LATENT_ATTENTION,)}
+                 "attention_latent": (LATENT_ATTENTION,), "attention_expanded": (LATENT_ATTENTION,)}
 
 
 class ExecProgram(Structure):
     _fields_ = [("n_layers", I64), ("n_order", I64), ("H", I64), ("V", I64), ("act_dtype", I64),
                 ("sms", I64), ("static_flag", I64), ("max_counters", I64), ("fused_conv", I64), ("fused_rope", I64),
-                ("latent_tc", I64), ("grouped_min_tokens", I64), ("tc_min_ctas", I64), ("tc_min_fill", F64),
+                ("latent_tc", I64), ("latent_expand", I64), ("grouped_min_tokens", I64), ("tc_min_ctas", I64), ("tc_min_fill", F64),
                 ("prologue", ExecOps), ("epilogue", ExecOps), ("layers", POINTER(ExecOps)), ("order", POINTER(I64)),
                 ("python", PythonOpFn), ("fns", PTR * len(ENTRY_POINTS))]
 
@@ -157,7 +158,7 @@ class ExecItem(Structure):
 class ExecStep(Structure):
     _fields_ = [("T", I64), ("B", I64), ("R", I64), ("max_q_len", I64), ("max_total_len", I64), ("n_order", I64),
                 ("ids", PTR), ("positions", PTR), ("seq_of_token", PTR), ("cu_seqlens", PTR), ("ctx_lens", PTR),
-                ("slot_ids", PTR), ("rows", PTR), ("q_lens", POINTER(I64)), ("items", POINTER(ExecItem)),
+                ("slot_ids", PTR), ("rows", PTR), ("q_lens", POINTER(I64)), ("host_ctx_lens", POINTER(I64)), ("items", POINTER(ExecItem)),
                 ("arena", PTR), ("arena_bytes", I64), ("logits", PTR), ("err", PTR), ("stream", PTR),
                 ("gemm_ws", PTR), ("gemm_ws_floats", I64), ("attn_ws", PTR), ("attn_ws_floats", I64), ("counters", PTR),
                 ("launches", I64), ("calls", I64 * len(ENTRY_POINTS))]

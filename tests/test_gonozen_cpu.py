@@ -119,9 +119,9 @@ def test_kernels_of_a_decode_step(monkeypatch):
         "norm_add_norm", "gemm_tcgen05", "soft_cap"]
     assert model.program.all_native
     p0, p1 = rec.of("cellm_latent_prep")
-    assert p0[0] is None and p0[2] is None and p0[3] is not None and p0[32] == 1 | 4 and p0[9] == 0             # no copy, no query latent, gates, latent and queries
-    assert (p0[11], p0[12], p0[5]) == (4 * 48, 4 * 48 + 80, 280) and abs(p0[31] - 1.0693147) < 1e-6            # where the latent and the gates lie; cos and sin
-    assert p1[32] == 1 | 2 and (p1[9], p1[11], p1[12]) == (56, 56, -1) and p1[2] is not None and p1[3] is None
+    assert p0[0] is None and p0[3] is None and p0[4] is not None and p0[33] == 1 | 4 and p0[10] == 0            # no copy, no query latent, gates, latent and queries
+    assert (p0[12], p0[13], p0[6]) == (4 * 48, 4 * 48 + 80, 280) and abs(p0[32] - 1.0693147) < 1e-6            # where the latent and the gates lie; cos and sin
+    assert p1[33] == 1 | 2 and (p1[10], p1[12], p1[13]) == (56, 56, -1) and p1[3] is not None and p1[4] is None
     a0, a1 = rec.of("cellm_attention_latent")
     assert a0[19] == 0 and a0[20] is None and a0[21] is not None and a1[19] == 9 and a1[20] is not None and a1[21] is None    # window, sinks, gate
     assert [h[4:6] for h in rec.of("cellm_head_product")[:1]] == [(280, 48)]                                    # queries read where the product left them
@@ -194,3 +194,28 @@ def test_parts_refuse_what_they_cannot_run():
         SandwichNormBlock(norm(), None, norm(), None, {"eps": 1e-5}, {"mixer_result_norm": torch.ones(4)}, torch.bfloat16)
     with pytest.raises(ConfigError, match="soft_cap"):
         LinearHead({"soft_cap": -1.0}, {"weight": z(4, 8)}, torch.float32)
+
+
+def test_a_long_portion_expands_its_keys_once(monkeypatch):
+    """Tokens that fill the tiles: the rows out of their pages, one product for all heads' keys and values, the attention over
+    them, and none of the per-head products; the windowed layer takes only the rows that its first new token can see. Short
+    portions, single tokens, and portions with far more rows than tokens stay on the rows themselves."""
+    rec = Recorder(monkeypatch, hooks={"cellm_attention_expanded_supports": lambda *a: 1})
+    cfg, plan, model = zero_model(config())
+    run_step(model, plan, [2000, 600, 30], [100, 0, 64])
+    names = names_of(rec)
+    assert not {"attention_latent", "head_product", "head_product_mma"} & set(names)
+    rows = rec.of("cellm_latent_rows")
+    assert [r[7] for r in rows] == [2100 + 600 + 94, 2000 + 8 + 600 + 30 + 8] and [r[10] for r in rows] == [0, 9]
+    a0, a1 = rec.of("cellm_attention_expanded")
+    assert (a0[8], a0[9], a0[10], a0[11]) == (3, 2630, 8 + 3 + 1, 2794) and a0[12:17] == (4, 32, 16, 24, 64) and a0[20] is not None and a0[19] is None
+    assert a1[12:17] == (2, 48, 0, 40, 64) and a1[18] == 9 and a1[19] is not None and a1[20] is None
+    kv = [g for g in rec.of("cellm_gemm_tcgen05") if (g[3], g[4], g[5]) == (2794, 4 * 56, 64)]
+    assert len(kv) == 1 and kv[0][6] == 80                                  # the rows' first 64 columns, 80 apart
+    prep = rec.of("cellm_latent_prep")[0]
+    assert prep[2] == 16 and prep[1] is not None                            # turned query parts by themselves, head behind head
+    for q_lens, ctx_lens in (([100], [0]), ([1] * 8, [500] * 8), ([2300], [40000])):
+        rec.calls.clear()
+        cfg, plan, model = zero_model(config())
+        run_step(model, plan, q_lens, ctx_lens)
+        assert len(rec.of("cellm_attention_expanded")) == (1 if ctx_lens == [40000] else 0), (q_lens, ctx_lens)      # the window leaves few rows

@@ -594,6 +594,109 @@ def test_latent_kernel_with_gates_and_sinks(nh, kw, dv, page, window):
     assert int(ctx.err.item()) == 0
 
 
+EXPANDED = [  # heads, dim, rot_dim, vdim, rank
+    (4, 128, 64, 128, 512), (2, 64, 0, 64, 64), (3, 16, 16, 16, 24), (2, 48, 32, 80, 40), (1, 96, 64, 112, 128), (2, 192, 64, 128, 64), (5, 32, 0, 32, 96),
+    (2, 128, 0, 48, 72), (1, 64, 96, 96, 16),
+]
+
+
+@pytest.mark.parametrize("window", [0, 1, 50, 128, 129, 300])
+@pytest.mark.parametrize("heads,dim,rot,vdim,rank", EXPANDED)
+def test_expanded_attention_alone(heads, dim, rot, vdim, rank, window):
+    """The tcgen05 attention over keys and values that were expanded from the rows: portions of several requests (one with a single
+    token, one with none) at contexts that end inside a block of keys, at its edge and inside a page; tiles that start inside a
+    block and blocks that only one of a pair of tiles reads; sinks and gates. Against 64-bit torch over the same rounded
+    inputs. The rows themselves come out of pages in an order of their own, those behind the window taken away."""
+    from cellm_b200 import ops
+    g = torch.Generator().manual_seed(heads * 1000 + dim + vdim)
+    q_lens, ctx_lens, page = [300, 1, 129, 0, 256, 7, 520], [0, 40, 131, 20, 128, 500, 255], 16
+    T, kw = sum(q_lens), rank + rot
+    rnd = lambda *s: (torch.randn(*s, generator=g) * 0.7).to(torch.bfloat16)
+    cache, table = paged([c + n for c, n in zip(ctx_lens, q_lens)], kw, page, torch.bfloat16, g)
+    pool = rnd(*cache.k.shape)
+    first = [max(0, c - window + 1) if window else 0 for c in ctx_lens]
+    bt = cache.block_table.clone()
+    for b, f in enumerate(first):
+        bt[b, :f // page] = -1
+    ctx = step_ctx(q_lens, ctx_lens)
+    keep = [range(f, c + n) if n else [] for f, c, n in zip(first, ctx_lens, q_lens)]
+    n_rows = sum(len(k) for k in keep)
+    rows = ops.latent_rows(pool.to(DEV), ctx.cu_seqlens, ctx.ctx_lens, bt, n_rows, ctx.err, window)
+    want_rows = torch.cat([torch.stack([pool[table[b, j // page], 0, j % page] for j in k]) for b, k in enumerate(keep) if len(k)])
+    assert torch.equal(rows.cpu(), want_rows)
+    qw = dim + rot
+    q, q_rot, kv = rnd(T, heads * qw + 8), rnd(T, heads * rot) if rot else None, rnd(n_rows, heads * (dim + vdim))
+    sinks, gate = torch.linspace(-2.0, 3.0, heads), torch.randn(T, heads, generator=g) * 2
+    scale = 1.5 * qw ** -0.5
+    for with_extras in (True, False):
+        want, t, at = torch.zeros(T, heads, vdim, dtype=torch.float64), 0, 0
+        for b, n in enumerate(q_lens):
+            m = len(keep[b])
+            if not n:
+                continue
+            k = kv[at:at + m, :heads * dim].double().view(m, heads, dim)
+            v = kv[at:at + m, heads * dim:].double().view(m, heads, vdim)
+            qq = q[t:t + n, :heads * qw].double().view(n, heads, qw)[..., :dim]
+            s = torch.einsum("ihd,jhd->hij", qq, k)
+            if rot:
+                s = s + torch.einsum("ihd,jd->hij", q_rot[t:t + n].double().view(n, heads, rot), rows[at:at + m, rank:].cpu().double())
+            back = (ctx_lens[b] + torch.arange(n))[:, None] - (first[b] + torch.arange(m))[None, :]
+            sees = (back >= 0) & ((back < window) if window else (back >= 0))
+            pr = plain.weights_of_scores(s * scale, sees, sinks.double() if with_extras else None)
+            want[t:t + n] = torch.einsum("hij,jhd->ihd", pr, v)
+            t, at = t + n, at + m
+        if with_extras:
+            want = want * torch.sigmoid(gate.double())[:, :, None]
+        out = ops.attention_expanded(q.to(DEV), q_rot.to(DEV) if rot else None, rows, kv.to(DEV), ctx.cu_seqlens, ctx.ctx_lens, q_lens, heads, dim, rot, vdim,
+                                     scale, ctx.err, window, sinks.to(DEV) if with_extras else None, gate.to(DEV) if with_extras else None)
+        assert int(ctx.err.item()) == 0
+        torch.testing.assert_close(out.cpu().double().view(T, heads, vdim), want, rtol=2e-2, atol=1e-2)
+
+
+def test_expanded_attention_refuses_what_it_does_not_take():
+    from cellm_b200.ops import _lib
+    supports = _lib.fn("attention_expanded", "cellm_attention_expanded_supports")
+    assert all(supports(*s) for s in EXPANDED)
+    assert not any(supports(*s) for s in [(2, 24, 0, 16, 16), (2, 16, 8, 16, 16), (2, 16, 0, 20, 16), (2, 16, 0, 144, 16), (2, 16, 0, 16, 12), (2, 320, 0, 64, 64), (0, 16, 0, 16, 16)])
+
+
+@pytest.mark.parametrize("windows", [(0, 90), (40, 0)])
+def test_expanded_portions_against_the_rows_themselves(tmp_path, windows):
+    """Whole models whose prompt portions take the expanded form, against the plain model and against the same engine with the form
+    switched off: prompts of several tiles, portions that start inside a block, portions beside single tokens, requests that
+    share a step."""
+    from cellm_b200.runtime import program
+    config = model_config(200, 128, [lat2(4, 32, 48, 64, 64, window=windows[0], mlp=moe(4, 2, 64, 1.0, (2, 1), (64, 1.5))),
+                                     lat(2, 64, 32, 64, 128, rot=(1000.0, 32, yarn(2.0, 128))), lat2(2, 48, 32, 96, 40, window=windows[1])])
+    folder = write_model(tmp_path / "m", config, 6)
+    cfg, w = load_plain(folder)
+    rng = np.random.default_rng(5)
+    reqs = {"x": rng.integers(0, 200, 700).tolist(), "y": rng.integers(0, 200, 333).tolist(), "z": rng.integers(0, 200, 40).tolist()}
+    ref = {rid: Ref(t, cfg, w) for rid, t in reqs.items()}
+    assert min(r.margin for r in ref.values()) > 0.1
+    both = [{"step": 0, "entries": [{"id": r, "tokens": t[:n], "want": list(range(n))} for (r, t), n in zip(reqs.items(), (300, 200, 39))], "end": []},
+            {"step": 1, "entries": [{"id": r, "tokens": t[a:b], "want": list(range(b - a))} for (r, t), a, b in zip(reqs.items(), (300, 200, 39), (699, 333, 40))],
+             "end": ["y", "z"]},
+            {"step": 2, "entries": [{"id": "x", "tokens": reqs["x"][699:], "want": [0]}], "end": ["x"]}]
+    old = dict(program.OPTIONS)
+    outs = {}
+    try:
+        program.OPTIONS["attention_tc_min_ctas"] = 1
+        for on in (True, False):
+            program.OPTIONS["latent_expand"] = on
+            before = program.CALLS["cellm_attention_expanded"]
+            outs[on] = {"whole": run_trace(folder, "bfloat16", traces.whole(reqs), 16),
+                        "portions": run_trace(folder, "bfloat16", traces.portions(reqs, (300, 130, 2, 190)), 8), "both": run_trace(folder, "bfloat16", both, 16)}
+            assert (program.CALLS["cellm_attention_expanded"] > before) == on
+    finally:
+        program.OPTIONS.update(old)
+    for fam in outs[True]:
+        for rid, t in reqs.items():
+            got = traces.as_matrix(outs[True][fam][rid], len(t))
+            against_plain(got, ref[rid], "bfloat16", f"expanded {fam} {rid}")
+            check_close(got, traces.as_matrix(outs[False][fam][rid], len(t)), "bfloat16", f"expanded vs rows, {fam} {rid}", k=K_SELF["bfloat16"])
+
+
 @pytest.mark.parametrize("window,page", [(0, 8), (1, 4), (16, 8), (21, 8), (33, 16), (130, 32), (400, 16)])
 @pytest.mark.parametrize("kw,dv", [(24, 8), (32, 16), (80, 64)])
 def test_a_window_sees_exactly_its_rows(window, page, kw, dv):

@@ -99,7 +99,7 @@ def test_decode_step_kernels(monkeypatch):
         "gated_norm_add",                                                        # (its bias is added by the gate-and-norm kernel)
         "add_rmsnorm", "gemm_tcgen05"]
     prep = rec.of("cellm_latent_prep")[0]
-    assert prep[23:29] == (3, 4, 32, 16, 64, 16) and prep[20] is not None                    # tokens, heads, dim, rot_dim, rank, rot; a cache to write
+    assert prep[24:30] == (3, 4, 32, 16, 64, 16) and prep[21] is not None                    # tokens, heads, dim, rot_dim, rank, rot; a cache to write
     att = rec.of("cellm_attention_latent")[0]
     assert (att[9], att[10], att[14], att[15], att[16]) == (3, 3, 4, 80, 64)                 # requests, tokens, heads, row width, value width
     norm = rec.of("cellm_gated_norm_add")[0]
