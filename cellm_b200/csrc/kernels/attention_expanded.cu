@@ -16,8 +16,8 @@
 //               bytes, 128-byte swizzle) through one ring of 16-KB slots: a block's key chunks (unrotated, rotated), then
 //               its value chunks, then the next block's;
 //   warp 1      MMA: per tile S = Q.K^T (M 128, N 128, K = dim, then rot_dim) and O += P.V (M 128, N up to 64 a chunk, K
-//               128). P takes the place of the scores in tensor memory, so a tile's next scores are issued when its P.V is
-//               done; while one tile's softmax runs, the tensor cores work on the other tile;
+//               128). P takes the place of the scores in tensor memory, so a tile's next scores are issued behind its P.V;
+//               while one tile's softmax runs, the tensor cores work on the other tile;
 //   warps 2..5  softmax of the first tile, warps 6..9 of the second, one row per thread, as in attention_tc.cu: scores into
 //               registers, mask, running maximum and sum in 32-bit, P = 2^(s*c - m) rounded to bfloat16 into tensor memory;
 //               the output accumulator is rescaled only when a row's maximum has grown by more than 2^8.
@@ -146,14 +146,16 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
         kb0 = lo_blk[0];
         nblk = (hi_blk[1] > 0 ? hi_blk[1] : hi_blk[0]) - kb0;
     }
-    auto active = [&](int t, int j) { return kb0 + j >= lo_blk[t] && kb0 + j < hi_blk[t]; };
+    auto active = [&](int t, int j) { return kb0 + j >= (t ? lo_blk[1] : lo_blk[0]) && kb0 + j < (t ? hi_blk[1] : hi_blk[0]); };
     const int per_block = kc + sh.vc;                                 // chunks of a block
 
     if (warp == 0) {
         if (live && lane == 0) {
             const int tiles = hi_blk[1] > 0 ? 2 : 1, qw = sh.dim + sh.rot;
             mbar_expect_tx(&sm.q_full, (uint32_t)(tiles * kc * CHUNK));
-            for (int t = 0; t < tiles; ++t) {
+#pragma unroll
+            for (int t = 0; t < 2; ++t) {
+                if (t >= tiles) break;
                 for (int c = 0; c < sh.kc_plain; ++c) tma_load_2d(q_s + (t * kc + c) * CHUNK, &map_q, head * qw + c * 64, t_base + tok0[t], &sm.q_full);
                 for (int c = 0; c < sh.kc_rot; ++c)
                     tma_load_2d(q_s + (t * kc + sh.kc_plain + c) * CHUNK, &map_q_rot, head * sh.rot + c * 64, t_base + tok0[t], &sm.q_full);
@@ -179,89 +181,96 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
     } else if (warp == 1) {
         if (live && lane == 0) {
             const uint32_t idesc_s = umma_idesc(TM, TN, false);       // S[128 x 128] = Q (K-major) . K^T (K-major)
-            int n_pv[2] = {0, 0};                                     // P.V products issued so far, per tile
+            const uint32_t idesc_v0 = umma_idesc(TM, min(sh.vdim, 64), true), idesc_v1 = umma_idesc(TM, max(sh.vdim - 64, 16), true);
+            const uint64_t dq0 = umma_desc(smem_u32(q_s)), dr0 = umma_desc(smem_u32(ring));
+            bool started[2] = {false, false};                         // a tile's output accumulator holds something
+            uint32_t p_phase[2] = {0, 0};
             bool ok = mbar_wait(&sm.q_full, 0, abort_flag);
-            // chunk c of block j lies in slot (j * per_block + c) % slots, filled for the ((j * per_block + c) / slots)th time
-            auto wait_chunks = [&](int j, int c0, int c1) -> bool {
-                for (int c = c0; c < c1; ++c) {
-                    const int n = j * per_block + c;
-                    if (!mbar_wait(&sm.slot_full[n % sh.slots], (uint32_t)(n / sh.slots) & 1u, abort_flag)) return false;
-                }
+            // The chunks go through the ring in order: a cursor is a slot and its fill's parity.
+            struct Cursor { int slot; uint32_t phase; };
+            auto advance = [&](Cursor c, int n) { c.slot += n; if (c.slot >= sh.slots) { c.slot -= sh.slots; c.phase ^= 1u; } return c; };
+            auto wait_chunks = [&](Cursor c, int n) -> bool {
+                for (int i = 0; i < n; ++i, c = advance(c, 1))
+                    if (!mbar_wait(&sm.slot_full[c.slot], c.phase, abort_flag)) return false;
                 return true;
             };
-            auto release_chunks = [&](int j, int c0, int c1) {
-                for (int c = c0; c < c1; ++c) umma_commit(&sm.slot_empty[(j * per_block + c) % sh.slots]);
+            auto release_chunks = [&](Cursor c, int n) {
+                for (int i = 0; i < n; ++i, c = advance(c, 1)) umma_commit(&sm.slot_empty[c.slot]);
             };
-            // scores of block j for tile t: its P.V before must be done, P lies where the scores go
-            auto issue_s = [&](int t, int j) -> bool {
-                if (n_pv[t] > 0 && !mbar_wait(&sm.pv_done[t], (uint32_t)(n_pv[t] - 1) & 1u, abort_flag)) return false;
-                tc_fence_after();
+            // scores of a block whose key chunks begin at c, for tile t. They take the place of the tile's P, which the P.V
+            // issued before them reads: one thread's products run in the order in which it issues them.
+            auto issue_s = [&](int t, Cursor c) {
+                uint64_t dq = dq0 + (uint64_t)(t * kc * (CHUNK / 16));
                 uint32_t acc = 0u;
-                for (int c = 0; c < kc; ++c) {
-                    const int width = c < sh.kc_plain ? sh.dim - c * 64 : sh.rot - (c - sh.kc_plain) * 64;
-                    const int steps = min(width, 64) / 16;
-                    const uint64_t dq = umma_desc(smem_u32(q_s + (t * kc + c) * CHUNK));
-                    const uint64_t dk = umma_desc(smem_u32(ring + ((j * per_block + c) % sh.slots) * CHUNK));
-                    for (int ks = 0; ks < steps; ++ks) {
-                        umma_bf16(tmem + (uint32_t)(t * TN), dq + (uint64_t)(ks * 2), dk + (uint64_t)(ks * 2), idesc_s, acc);
-                        acc = 1u;
+                for (int part = 0; part < 2; ++part) {
+                    int steps = (part ? sh.rot : sh.dim) / 16;
+                    while (steps > 0) {
+                        const uint64_t dk = dr0 + (uint64_t)(c.slot * (CHUNK / 16));
+#pragma unroll
+                        for (int ks = 0; ks < 4; ++ks) {
+                            if (ks < steps) umma_bf16(tmem + (uint32_t)(t * TN), dq + (uint64_t)(ks * 2), dk + (uint64_t)(ks * 2), idesc_s, acc);
+                            acc = 1u;
+                        }
+                        steps -= 4;
+                        dq += (uint64_t)(CHUNK / 16);
+                        c = advance(c, 1);
                     }
                 }
                 umma_commit(&sm.s_full[t]);
-                return true;
             };
-            auto issue_pv = [&](int t, int j) -> bool {
-                if (!mbar_wait(&sm.p_full[t], (uint32_t)n_pv[t] & 1u, abort_flag)) return false;
+            auto issue_pv = [&](int t, Cursor c) -> bool {
+                if (!mbar_wait(&sm.p_full[t], p_phase[t], abort_flag)) return false;
+                p_phase[t] ^= 1u;
                 tc_fence_after();
-                for (int c = 0; c < sh.vc; ++c) {
-                    const uint32_t idesc_o = umma_idesc(TM, min(sh.vdim - c * 64, 64), true);      // O[128 x 64] += P (K-major) . V (MN-major)
-                    const uint64_t dv = umma_desc(smem_u32(ring + ((j * per_block + kc + c) % sh.slots) * CHUNK));
+                for (int v = 0; v < sh.vc; ++v, c = advance(c, 1)) {
+                    const uint64_t dv = dr0 + (uint64_t)(c.slot * (CHUNK / 16));
 #pragma unroll
-                    for (int ks = 0; ks < TN / 16; ++ks) {
-                        const uint32_t pa = tmem + (uint32_t)(t * TN + ks * 8);                    // 16 keys = 8 columns of P
-                        umma_bf16_ts(tmem + (uint32_t)(O_COL + t * TN + c * 64), pa, dv + (uint64_t)(ks * 16 * 128 / 16), idesc_o,
-                                     (n_pv[t] | ks) != 0 ? 1u : 0u);
-                    }
+                    for (int ks = 0; ks < TN / 16; ++ks)               // 16 keys = 8 columns of P = 16 rows of V
+                        umma_bf16_ts(tmem + (uint32_t)(O_COL + t * TN + v * 64), tmem + (uint32_t)(t * TN + ks * 8), dv + (uint64_t)(ks * 16 * 128 / 16),
+                                     v ? idesc_v1 : idesc_v0, started[t] || ks != 0 ? 1u : 0u);
                 }
-                umma_commit(&sm.pv_done[t]);
-                ++n_pv[t];
+                started[t] = true;
                 return true;
             };
+            Cursor keys{0, 0u};
             if (ok && nblk > 0) {
-                ok = wait_chunks(0, 0, kc);
-                for (int t = 0; ok && t < 2; ++t)
-                    if (active(t, 0)) ok = issue_s(t, 0);
-                if (ok) release_chunks(0, 0, kc);
+                ok = wait_chunks(keys, kc);
+                if (ok) {
+                    tc_fence_after();
+#pragma unroll
+                    for (int t = 0; t < 2; ++t)
+                        if (active(t, 0)) issue_s(t, keys);
+                    release_chunks(keys, kc);
+                }
             }
             for (int j = 0; ok && j < nblk; ++j) {
-                ok = wait_chunks(j, kc, per_block);
-                bool next_here = false;                                // the next block's keys are in the ring
-                for (int t = 0; ok && t < 2; ++t) {
-                    if (active(t, j)) ok = issue_pv(t, j);
-                    if (ok && j + 1 < nblk && active(t, j + 1)) {
-                        if (!next_here) ok = wait_chunks(j + 1, 0, kc), next_here = true;
-                        if (ok) ok = issue_s(t, j + 1);
-                    }
-                }
+                const Cursor vals = advance(keys, kc), next = advance(vals, sh.vc);
+                const bool more = j + 1 < nblk;
+                ok = wait_chunks(vals, sh.vc) && (!more || wait_chunks(next, kc));
                 if (!ok) break;
-                release_chunks(j, kc, per_block);
-                if (j + 1 < nblk) {
-                    if (!next_here) ok = wait_chunks(j + 1, 0, kc);    // (a block neither tile reads: not reached by the ranges above)
-                    if (ok) release_chunks(j + 1, 0, kc);
+#pragma unroll
+                for (int t = 0; t < 2; ++t) {
+                    if (ok && active(t, j)) ok = issue_pv(t, vals);
+                    if (ok && active(t, j) && !active(t, j + 1)) umma_commit(&sm.pv_done[t]);       // the tile's last
+                    if (t == 1 && ok) release_chunks(vals, sh.vc);
+                    if (ok && more && active(t, j + 1)) { tc_fence_after(); issue_s(t, next); }
                 }
+                if (ok && more) release_chunks(next, kc);
+                keys = next;
             }
             if (!ok) { *abort_flag = 1; atomicOr(err, CELLM_DEV_WAIT_TIMEOUT); }
         }
-    } else if (live && hi_blk[(warp - 2) >> 2] > 0) {
+    } else if (live && (warp >= 6 ? hi_blk[1] : hi_blk[0]) > 0) {
         const int t = (warp - 2) >> 2;                                // which tile
+        const int lo_t = t ? lo_blk[1] : lo_blk[0], hi_t = t ? hi_blk[1] : hi_blk[0];
         const int qt = warp & 3;                                      // quarter of the tile's rows = of tensor memory's lanes
-        const int tok = tok0[t] + qt * 32 + lane;                     // token within the portion
+        const int tok = (t ? tok0[1] : tok0[0]) + qt * 32 + lane;                     // token within the portion
         const bool row_ok = tok < q_len;
         const int pos = row_ok ? ctx + tok : -1;
         const int lo = window > 0 ? pos - window + 1 : 0;
         const uint32_t lane_base = tmem + ((uint32_t)(qt * 32) << 16);
         const uint32_t s_col = (uint32_t)(t * TN), o_col = (uint32_t)(O_COL + t * TN);
-        const int n_blocks = hi_blk[t] - lo_blk[t];
+        const int n_blocks = hi_t - lo_t;
         const int o_cols = (sh.vdim + 31) / 32 * 32;
         float m = -INFINITY, l = 0.f;
         bool ok = true;
@@ -274,7 +283,7 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
 #pragma unroll
             for (int c = 0; c < TN / 32; ++c) tmem_ld32_nowait(lane_base + s_col + (uint32_t)(c * 32), s + c * 32);
             tmem_ld_wait();
-            const int jbase = (lo_blk[t] + it) * TN;
+            const int jbase = (lo_t + it) * TN;
             const bool open_block = row_ok && jbase + TN - 1 <= pos && jbase >= lo;
             if (!open_block) {
 #pragma unroll
@@ -326,7 +335,7 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
             tc_fence_before();
             mbar_arrive(&sm.p_full[t]);
         }
-        if (ok && n_blocks > 0) ok = mbar_wait(&sm.pv_done[t], (uint32_t)(n_blocks - 1) & 1u, abort_flag);
+        if (ok && n_blocks > 0) ok = mbar_wait(&sm.pv_done[t], 0, abort_flag);
         if (!ok && lane == 0) { *abort_flag = 1; atomicOr(err, CELLM_DEV_WAIT_TIMEOUT); }
         if (ok) {
             tc_fence_after();
