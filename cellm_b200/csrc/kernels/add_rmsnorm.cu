@@ -164,7 +164,7 @@ CELLM_API int cellm_add2_rmsnorm(float* x, const void* delta, const void* delta2
 
 // ---- an addend that is normed before it joins the stream -------------------------------------------------------------
 template <typename TA, typename TW>
-__global__ void norm_add_norm_kernel(float* __restrict__ x, const TA* __restrict__ delta, const TW* __restrict__ w_d, float eps_d,
+__global__ void norm_add_norm_kernel(float* x, const TA* delta, const TW* __restrict__ w_d, float eps_d,
                                      const TW* __restrict__ w, TA* __restrict__ y, const int* __restrict__ rows, int H, float eps) {
     extern __shared__ float vals[];      // [H]
     __shared__ float scratch[32];

@@ -25,7 +25,7 @@ latent_flash_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
                     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ pool,
                     const int* __restrict__ cu_seqlens, const int* __restrict__ ctx_lens, const int* __restrict__ block_table,
                     int bt_stride, int B, int T, int num_pages, int page_size, int nh, int kw, int dv, float scale_log2e,
-                    int nsplit, int window, const float* __restrict__ sinks, const float* __restrict__ gate, int* __restrict__ err) {
+                    int nsplit, int window, const float* __restrict__ sinks, const float* gate, int* __restrict__ err) {
     constexpr int NT = DVW / 8;
     extern __shared__ __align__(128) uint8_t smem_raw[];
     const int stride = kw + 8;                                   // elements per row in shared memory (16 bytes of padding)
@@ -233,9 +233,8 @@ latent_flash_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
 }
 
 // The pieces of a row merged in their order: out = sum_s 2^(m_s - M) o_s / sum_s 2^(m_s - M) l_s.
-__global__ void latent_merge_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ part_o,
-                                    const float* __restrict__ part_ml, size_t n_rows, int dv, int nsplit,
-                                    const float* __restrict__ sinks, const float* __restrict__ gate, int nh) {
+__global__ void latent_merge_kernel(__nv_bfloat16* __restrict__ out, const float* part_o, const float* part_ml, size_t n_rows, int dv, int nsplit,
+                                    const float* __restrict__ sinks, const float* gate, int nh) {
     extern __shared__ float ml[];        // [nsplit][2]: maximum and sum of each piece, then its weight in [s][0]
     pdl_trigger();
     pdl_wait();

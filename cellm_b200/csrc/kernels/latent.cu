@@ -31,14 +31,15 @@ __device__ __forceinline__ void split_angle(int pos, float hi, float lo, float* 
     *s_out = s * ce + c * se;
 }
 
+// (The products' rows are not declared __restrict__ in the kernel: their loads stay behind the wait on the kernel before.)
 // What a launch of the preparation does; a block's role follows from blockIdx.y (in this order, the roles asked for).
 enum { LP_LATENT = 1, LP_QUERY_NORM = 2, LP_QUERIES = 4 };
 
 template <typename TP, typename TA, typename TW>
 __global__ void __launch_bounds__(128)
-latent_prep_kernel(TA* __restrict__ q_plain, TA* __restrict__ q_turned, long long turned_hs, const TP* __restrict__ q_rows, long long q_ld,
-                   TA* __restrict__ cq, const TP* __restrict__ cq_rows, int q_rank, const TW* __restrict__ cq_norm_w,
-                   float* __restrict__ gate_out, const TP* __restrict__ gate_rows, const TP* __restrict__ down_rows, long long ld,
+latent_prep_kernel(TA* __restrict__ q_plain, TA* __restrict__ q_turned, long long turned_hs, const TP* q_rows, long long q_ld,
+                   TA* __restrict__ cq, const TP* cq_rows, int q_rank, const TW* __restrict__ cq_norm_w,
+                   float* __restrict__ gate_out, const TP* gate_rows, const TP* down_rows, long long ld,
                    const TW* __restrict__ c_norm_w, float eps, const int* __restrict__ positions,
                    const int* __restrict__ seq_of_token, const int* __restrict__ block_table, int bt_stride,
                    TA* __restrict__ pool, int num_pages, int page_size, int heads, int dim, int rot_dim, int rank,
